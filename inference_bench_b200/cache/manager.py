@@ -1,7 +1,7 @@
 """The cache manager: pages of keys and values with a block table per request, in groups of layers
 with the same needs, and beside them slots of fixed-size per-request state.
 
-Executions of the schedule whose mixers ask for the same `PagedKV(kv_heads, head_dim, window)` form a
+Executions of the schedule whose mixers ask for the same `PagedKV(kv_heads, head_dim, window, keep_first)` form a
 group. A group has its own page pool, its own device tensor
 [executions, pages, 2 (K, V), kv_heads, page_size, head_dim] and its own block table per request
 (`PagedRows(width, window)`, one row per token, is the same with one plane and one head:
@@ -9,7 +9,7 @@ group. A group has its own page pool, its own device tensor
 page therefore holds `page_size` positions of every execution in the group, and one table serves
 them all (block-major, like the reference: docs/specrt-scheduler.md:11, 20-22). A group with a window
 gives a page back as soon as every position in it has fallen out of the window of the request's
-next token; a request's end gives everything back. Mixers that ask for `FixedState(shape, dtype)`
+next token, except the pages that hold its first `keep_first` positions; a request's end gives everything back. Mixers that ask for `FixedState(shape, dtype)`
 get a tensor [slots, *shape], zeroed for a slot when a request is admitted to it
 (reference: crates/specrt/src/statepool.rs:7-80, crates/specrt/src/runtime/step.rs:133-135).
 
@@ -127,7 +127,8 @@ class CacheManager:
                     raise TypeError(f"schedule entry {i} asks the cache for {n!r}, which it does not know")
         self._lib = native.load()
         windows = (C.c_int * max(1, len(self.groups)))(*[int(g.need.window or 0) for g in self.groups])
-        self._core = self._lib.ibh_cache_new(len(self.groups), windows, page_size, num_pages, max_requests, max_tokens_per_request)
+        keeps = (C.c_int * max(1, len(self.groups)))(*[int(getattr(g.need, "keep_first", 0) or 0) for g in self.groups])
+        self._core = self._lib.ibh_cache_new(len(self.groups), windows, keeps, page_size, num_pages, max_requests, max_tokens_per_request)
         if not self._core:
             raise ValueError(native.last_error())
         for gi, g in enumerate(self.groups):

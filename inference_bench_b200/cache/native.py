@@ -12,7 +12,7 @@ _SIGNATURES = {
     "ibh_pool_new": (_p, [_i]), "ibh_pool_free": (None, [_p]), "ibh_pool_num_pages": (_i, [_p]), "ibh_pool_free_pages": (_i, [_p]),
     "ibh_pool_allocate": (_i, [_p]), "ibh_pool_share": (_i, [_p, _i]), "ibh_pool_release": (_i, [_p, _i]), "ibh_pool_refcount": (_i, [_p, _i]),
     "ibh_pool_check": (_i, [_p]),
-    "ibh_cache_new": (_p, [_i, C.POINTER(_i), _i, _i, _i, _i]), "ibh_cache_free": (None, [_p]), "ibh_cache_pool": (_p, [_p, _i]),
+    "ibh_cache_new": (_p, [_i, C.POINTER(_i), C.POINTER(_i), _i, _i, _i, _i]), "ibh_cache_free": (None, [_p]), "ibh_cache_pool": (_p, [_p, _i]),
     "ibh_cache_tables": (C.POINTER(_i), [_p]), "ibh_cache_table_width": (_i, [_p]), "ibh_cache_free_slots": (_i, [_p]),
     "ibh_cache_admit": (_i, [_p]), "ibh_cache_length": (_i, [_p, _i]), "ibh_cache_pages_missing": (None, [_p, _i, _i, _i, C.POINTER(_i)]),
     "ibh_cache_extend": (_i, [_p, _i, _i]), "ibh_cache_shrink_to_committed": (_i, [_p, _i]), "ibh_cache_commit": (_i, [_p, _i, _i]),

@@ -27,9 +27,21 @@ constexpr int kKS = kKeysPerWarp / 16;           // 16-key MMA steps per warp
 // tiles_per_slice > 0: slices of that many tiles at fixed absolute positions. 0: the token's own visible
 // tiles in max_slices equal parts of at least kMinTiles tiles, so that every token gives about as many
 // units of work, of about equal size, whatever its length.
+// keep > 0 (with a window): the positions before `keep` are seen as well. Tiles of kept keys that lie before the window's first tile
+// are then numbered right before it (the slices cut one run of tiles): tile number n < win_tile stands for tile n - pre_shift, and the
+// slices start at the first kept tile's number whatever tiles_per_slice is. Without kept keys pre_shift is 0 and win_tile 0.
 constexpr int kMinTiles = 2;
-__device__ __forceinline__ void slice_plan(int pos, int window, int max_slices, int tiles_per_slice, int& lo, int& tile_lo, int& tps) {
+__device__ __forceinline__ void slice_plan(int pos, int window, int keep, int max_slices, int tiles_per_slice, int& lo, int& tile_lo, int& tps, int& win_tile, int& pre_shift) {
   lo = ib::first_visible(pos, window);
+  win_tile = 0, pre_shift = 0;
+  if (keep > 0) {
+    win_tile = lo / kTile;
+    const int n_pre = min((keep + kTile - 1) / kTile, win_tile);
+    tile_lo = pre_shift = win_tile - n_pre;
+    const int tiles = pos / kTile - tile_lo + 1;
+    tps = tiles_per_slice > 0 ? tiles_per_slice : max(kMinTiles, (tiles + max_slices - 1) / max_slices);
+    return;
+  }
   if (tiles_per_slice > 0) {
     tile_lo = 0;
     tps = tiles_per_slice;
@@ -45,8 +57,9 @@ __global__ void __launch_bounds__(kWarps * 32)
     decode_split_kernel(const __nv_bfloat16* __restrict__ q, IbKvView kv, const int* __restrict__ dec_tokens,
                         const int* __restrict__ positions, const int* __restrict__ seg_of_token, int window, float scale_log2e,
                         float* __restrict__ part_o, float* __restrict__ part_ml, int heads, int max_slices, int tiles_per_slice,
-                        unsigned* __restrict__ status, float cap_pre) {
+                        unsigned* __restrict__ status, float cap_pre, int keep) {
   // cap_pre != 0: a raw product s counts as tanh(s * cap_pre) (the caller's scale_log2e is then cap * log2 e)
+  // keep > 0: see slice_plan; `tile` and `key` below are the numbers of tiles and keys, real_key() the position a key number stands for
   constexpr int CPR = HD / 8;              // 16-byte chunks per row
   constexpr int TILE = kTile * HD * 2;     // bytes of one K (or V) tile
   extern __shared__ __align__(1024) uint8_t smem[];
@@ -64,10 +77,17 @@ __global__ void __launch_bounds__(kWarps * 32)
   const int kvh = blockIdx.x, item = blockIdx.y, slice = blockIdx.z;
   const int t = dec_tokens[item];
   const int pos = positions[t], seg = seg_of_token[t];
-  const int lo = ib::first_visible(pos, window);
-  const int slice_keys = tiles_per_slice * kTile;
-  const int k_begin = max(lo, slice * slice_keys), k_end = min(pos + 1, (slice + 1) * slice_keys);
+  int lo, tile_lo, tps, win_tile, pre_shift;
+  slice_plan(pos, window, keep, gridDim.z, tiles_per_slice, lo, tile_lo, tps, win_tile, pre_shift);
+  const int k_begin = max(keep > 0 ? 0 : lo, (tile_lo + slice * tps) * kTile), k_end = min(pos + 1, (tile_lo + (slice + 1) * tps) * kTile);
   if (k_begin >= k_end) return;
+  auto real_key = [&](int tile, int key) { return tile < win_tile ? key - pre_shift * kTile : key; };
+  auto seen = [&](int tile, int key) {   // whether the token sees the key with this number (of this slice)
+    if (key < k_begin || key >= k_end) return false;
+    if (keep <= 0) return true;
+    const int r = real_key(tile, key);
+    return r >= lo || r < keep;
+  };
   const int tile_begin = k_begin / kTile, tile_end = (k_end - 1) / kTile + 1;
   const int group = heads / kv.kv_heads;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -80,7 +100,7 @@ __global__ void __launch_bounds__(kWarps * 32)
     long long* o = offs + stage * kTile;
     if (tid < kTile) {
       int key = tile * kTile + tid;
-      long long off = (key >= k_begin && key < k_end) ? ib::kv_offset(kv, seg, key, kvh) : -2;
+      long long off = seen(tile, key) ? ib::kv_offset(kv, seg, real_key(tile, key), kvh) : -2;
       if (off == -1) atomicOr(status, IB_ERR_BAD_PAGE);
       o[tid] = off;
     }
@@ -173,7 +193,7 @@ __global__ void __launch_bounds__(kWarps * 32)
 #pragma unroll
       for (int e = 0; e < 4; e++) {
         int key = tile * kTile + wkey + 8 * j + 2 * tq + (e & 1);
-        float v = (key >= k_begin && key < k_end) ? (cap_pre != 0.f ? ib::tanh_fast(s[j][e] * cap_pre) : s[j][e]) * scale_log2e : -INFINITY;
+        float v = seen(tile, key) ? (cap_pre != 0.f ? ib::tanh_fast(s[j][e] * cap_pre) : s[j][e]) * scale_log2e : -INFINITY;
         s[j][e] = v;
         mn[e >> 1] = fmaxf(mn[e >> 1], v);
       }
@@ -270,7 +290,7 @@ template <int HD>
 __global__ void __launch_bounds__(kCombineThreads)
     decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const int* __restrict__ dec_tokens,
                           const int* __restrict__ positions, int window, __nv_bfloat16* __restrict__ out, int heads, int max_slices,
-                          int tiles_per_slice, unsigned* __restrict__ status, int sink, IbAttnTail tail) {
+                          int tiles_per_slice, unsigned* __restrict__ status, int sink, IbAttnTail tail, int keep) {
   // sink: one more term of score 0 (or tail.sink_values[head]) and no value in the denominator; tail: factors on the output and its row length
   constexpr int DQ = HD / 4;
   constexpr int SG = kCombineThreads / DQ;
@@ -280,9 +300,9 @@ __global__ void __launch_bounds__(kCombineThreads)
   const int h = blockIdx.x, item = blockIdx.y;
   const int t = dec_tokens[item];
   const int pos = positions[t];
-  int lo, tile_lo, tps;
-  slice_plan(pos, window, max_slices, tiles_per_slice, lo, tile_lo, tps);
-  const int s_begin = (lo / kTile - tile_lo) / tps;
+  int lo, tile_lo, tps, win_tile, pre_shift;
+  slice_plan(pos, window, keep, max_slices, tiles_per_slice, lo, tile_lo, tps, win_tile, pre_shift);
+  const int s_begin = keep > 0 ? 0 : (lo / kTile - tile_lo) / tps;
   int s_end = (pos / kTile - tile_lo) / tps + 1;
   if (s_end > max_slices) {   // the caller's max_slices does not cover this position: nothing beyond the scratch is read, and the status says so
     if (threadIdx.x == 0) atomicOr(status, IB_ERR_INTERNAL);
@@ -388,7 +408,7 @@ __global__ void __launch_bounds__((kWarps + 1) * 32, 2)
                          const int* __restrict__ seg_of_token, int window, float scale_log2e, float* __restrict__ part_o,
                          float* __restrict__ part_ml, int heads, int n_dec, int max_slices, int tiles_per_slice, int merge_cols,
                          const __grid_constant__ CUtensorMap kv_map, long long view_row0, unsigned long long wait_ns, unsigned* __restrict__ status,
-                         float cap_pre) {
+                         float cap_pre, int keep) {
   constexpr int CPR = HD / 8;
   constexpr int TILE = kTile * HD * 2;
   constexpr int HB = HD / 64;
@@ -435,6 +455,7 @@ __global__ void __launch_bounds__((kWarps + 1) * 32, 2)
   __syncthreads();
   // unit -> what it covers; false when it holds no visible key
   int kvh, item, slice, t, pos, seg, k_begin, k_end;
+  int lo = 0, win_tile = 0, pre_shift = 0;   // keep > 0: see slice_plan (tile, key and box below are numbers; these turn them into positions)
   bool has_own = false;   // fused form: the unit's slice holds the token's own position
   auto open_unit = [&](int u) {
     kvh = u % kv.kv_heads;
@@ -450,9 +471,9 @@ __global__ void __launch_bounds__((kWarps + 1) * 32, 2)
       pos = positions[t];
       seg = seg_of_token[t];
     }
-    int lo, tile_lo, tps;
-    slice_plan(pos, window, max_slices, tiles_per_slice, lo, tile_lo, tps);
-    k_begin = max(lo, (tile_lo + slice * tps) * kTile);
+    int tile_lo, tps;
+    slice_plan(pos, window, keep, max_slices, tiles_per_slice, lo, tile_lo, tps, win_tile, pre_shift);
+    k_begin = max(keep > 0 ? 0 : lo, (tile_lo + slice * tps) * kTile);
     k_end = min(pos + 1, (tile_lo + (slice + 1) * tps) * kTile);
     if constexpr (FUSED) {   // the own position comes from the projection, not from the cache
       has_own = k_begin < k_end && k_end == pos + 1;
@@ -492,10 +513,15 @@ __global__ void __launch_bounds__((kWarps + 1) * 32, 2)
       for (int tile = tile_begin; tile < tile_end; tile++, n++) {
         const int rel = (tile - tile_begin) * ppt;
         if ((rel & 31) == 0) {
-          const int box = tile_begin * ppt + rel + lane;
-          const int key0 = box * box_rows;
+          int box = tile_begin * ppt + rel + lane;
+          int key0 = box * box_rows;
           held_row = -1;
-          if (key0 < k_end && key0 + box_rows > k_begin) {
+          bool want = key0 < k_end && key0 + box_rows > k_begin;
+          if (keep > 0) {
+            if (key0 < win_tile * kTile) box -= pre_shift * ppt, key0 -= pre_shift * kTile;
+            want = want && (key0 + box_rows > lo || key0 < keep);
+          }
+          if (want) {
             const int col = boxes_per_page == 1 ? box : box / boxes_per_page;
             const int page = col < kv.table_stride ? kv.block_table[(size_t)seg * kv.table_stride + col] : -1;
             if (page >= 0 && page < kv.num_pages)
@@ -736,7 +762,12 @@ __global__ void __launch_bounds__((kWarps + 1) * 32, 2)
 #pragma unroll
         for (int e = 0; e < 4; e++) {
           const int key = tile * kTile + wkey + 8 * j + 2 * tq + (e & 1);
-          const float v = (key >= k_begin && key < k_end) ? (cap_pre != 0.f ? ib::tanh_fast(s[j][e] * cap_pre) : s[j][e]) * scale_log2e : -INFINITY;
+          bool seen = key >= k_begin && key < k_end;
+          if (keep > 0) {
+            const int r = tile < win_tile ? key - pre_shift * kTile : key;
+            seen = seen && (r >= lo || r < keep);
+          }
+          const float v = seen ? (cap_pre != 0.f ? ib::tanh_fast(s[j][e] * cap_pre) : s[j][e]) * scale_log2e : -INFINITY;
           s[j][e] = v;
           mn[e >> 1] = fmaxf(mn[e >> 1], v);
         }
@@ -846,7 +877,7 @@ template <int HD, bool FUSED>
 int launch_stream(const void* q, const RawQkv* raw, const IbKvView* kv, const int* dec_tokens, int n_dec, const int* positions, const int* seg_of_token,
                   int window, float scale, float* part_o, float* part_ml, void* out, int heads, int max_slices, int tiles_per_slice,
                   const CUtensorMap* kv_map, long long view_row0, unsigned* status, cudaStream_t stream, float softcap = 0.f, int sink = 0,
-                  const IbAttnTail& tail = IbAttnTail{}) {
+                  const IbAttnTail& tail = IbAttnTail{}, int keep = 0) {
   const float scale_log2e = (softcap > 0.f ? softcap : scale) * 1.4426950408889634f, cap_pre = softcap > 0.f ? scale / softcap : 0.f;
   const int group = heads / kv->kv_heads;
   const int merge_cols = stream_merge_cols(group, HD);
@@ -869,10 +900,10 @@ int launch_stream(const void* q, const RawQkv* raw, const IbKvView* kv, const in
   const RawQkv none = {};
   ib::launch(decode_stream_kernel<HD, FUSED>, grid, (kWarps + 1) * 32, smem, stream, (const __nv_bfloat16*)q, raw ? *raw : none, *kv, dec_tokens,
              positions, seg_of_token, window, scale_log2e, part_o, part_ml, heads, n_dec, max_slices, tiles_per_slice, merge_cols,
-             *kv_map, view_row0, ib_wait_limit_ns(), status, cap_pre);
+             *kv_map, view_row0, ib_wait_limit_ns(), status, cap_pre, keep);
   IB_CHECK_LAUNCH("attention_decode_stream split");
   ib::launch(decode_combine_kernel<HD>, dim3(heads, n_dec), kCombineThreads, 0, stream, part_o, part_ml, dec_tokens, positions, window, (__nv_bfloat16*)out, heads,
-             max_slices, tiles_per_slice, status, sink, tail);
+             max_slices, tiles_per_slice, status, sink, tail, keep);
   IB_CHECK_LAUNCH("attention_decode_stream combine");
   return 0;
 }
@@ -880,7 +911,7 @@ int launch_stream(const void* q, const RawQkv* raw, const IbKvView* kv, const in
 template <int HD>
 int launch(const void* q, const IbKvView* kv, const int* dec_tokens, int n_dec, const int* positions, const int* seg_of_token, int window,
            float scale, float* part_o, float* part_ml, void* out, int heads, int max_slices, int tiles_per_slice, unsigned* status,
-           cudaStream_t stream, float softcap = 0.f, int sink = 0, const IbAttnTail& tail = IbAttnTail{}) {
+           cudaStream_t stream, float softcap = 0.f, int sink = 0, const IbAttnTail& tail = IbAttnTail{}, int keep = 0) {
   const float scale_log2e = (softcap > 0.f ? softcap : scale) * 1.4426950408889634f, cap_pre = softcap > 0.f ? scale / softcap : 0.f;
   constexpr int smem = 16 * HD * 2 + 4 * kTile * HD * 2 + 2 * kTile * 8;   // Q, two stages of K and V, key offsets
   static_assert(kWarps * 16 * HD * 4 <= 4 * kTile * HD * 2, "the merge buffer must fit in the tiles");
@@ -892,10 +923,10 @@ int launch(const void* q, const IbKvView* kv, const int* dec_tokens, int n_dec, 
   }
   dim3 grid(kv->kv_heads, n_dec, max_slices);
   ib::launch(decode_split_kernel<HD>, grid, kWarps * 32, smem, stream, (const __nv_bfloat16*)q, *kv, dec_tokens, positions, seg_of_token, window,
-             scale_log2e, part_o, part_ml, heads, max_slices, tiles_per_slice, status, cap_pre);
+             scale_log2e, part_o, part_ml, heads, max_slices, tiles_per_slice, status, cap_pre, keep);
   IB_CHECK_LAUNCH("attention_decode split");
   ib::launch(decode_combine_kernel<HD>, dim3(heads, n_dec), kCombineThreads, 0, stream, part_o, part_ml, dec_tokens, positions, window, (__nv_bfloat16*)out, heads,
-             max_slices, tiles_per_slice, status, sink, tail);
+             max_slices, tiles_per_slice, status, sink, tail, keep);
   IB_CHECK_LAUNCH("attention_decode combine");
   return 0;
 }
@@ -946,12 +977,14 @@ bool read_tail(const char* who, const IbAttnTail* in, int sink, int heads, const
 
 // softcap > 0: scores become softcap * tanh(score / softcap) after the scale; sink: the softmax's denominator has one added (or
 // exp(tail->sink_values[head])). window < 0: a position sees the earlier positions of its own block of -window positions. tail (may be
-// null): the sink's scores, a gate and a constant on the output, the output's row length (IbAttnTail).
+// null): the sink's scores, a gate and a constant on the output, the output's row length (IbAttnTail). keep (with a window): the first
+// positions of the request that are seen beside the window.
 extern "C" int ib_attention_decode_capped(const void* q, const IbKvView* kv, const int* dec_tokens, int n_dec, const int* positions,
                                           const int* seg_of_token, int window, float scale, float* part_o, float* part_ml, void* out, int heads,
-                                          int max_slices, int tiles_per_slice, float softcap, int sink, const IbAttnTail* tail_in, unsigned* status,
+                                          int max_slices, int tiles_per_slice, float softcap, int sink, const IbAttnTail* tail_in, int keep, unsigned* status,
                                           cudaStream_t stream) {
   if (n_dec == 0) return 0;
+  IB_CHECK_ARG(keep >= 0 && (keep == 0 || window > 0), "attention_decode: %d kept positions need a window", keep);
   IbAttnTail tail;
   if (!read_tail("attention_decode", tail_in, sink, heads, kv, tail)) return 1;
   IB_CHECK_ARG(kv && kv->base && kv->block_table, "attention_decode: the cache view has a null pointer");
@@ -962,10 +995,10 @@ extern "C" int ib_attention_decode_capped(const void* q, const IbKvView* kv, con
   IB_CHECK_ARG(n_dec > 0 && n_dec <= 65535 && max_slices > 0 && max_slices <= 65535, "attention_decode: bad sizes n=%d slices=%d", n_dec, max_slices);
   if (kv->head_dim == 128)
     return launch<128>(q, kv, dec_tokens, n_dec, positions, seg_of_token, window, scale, part_o, part_ml, out, heads, max_slices, tiles_per_slice,
-                       status, stream, softcap, sink, tail);
+                       status, stream, softcap, sink, tail, keep);
   if (kv->head_dim == 64)
     return launch<64>(q, kv, dec_tokens, n_dec, positions, seg_of_token, window, scale, part_o, part_ml, out, heads, max_slices, tiles_per_slice,
-                      status, stream, softcap, sink, tail);
+                      status, stream, softcap, sink, tail, keep);
   return ib_set_error("attention_decode: head_dim %d has no tensor-core kernel (64 and 128 have)", kv->head_dim);
 }
 
@@ -973,15 +1006,16 @@ extern "C" int ib_attention_decode(const void* q, const IbKvView* kv, const int*
                                    const int* seg_of_token, int window, float scale, float* part_o, float* part_ml, void* out, int heads,
                                    int max_slices, int tiles_per_slice, unsigned* status, cudaStream_t stream) {
   return ib_attention_decode_capped(q, kv, dec_tokens, n_dec, positions, seg_of_token, window, scale, part_o, part_ml, out, heads, max_slices, tiles_per_slice, 0.f, 0,
-                                    nullptr, status, stream);
+                                    nullptr, 0, status, stream);
 }
 
 namespace {
 int stream_entry(const void* q, const RawQkv* raw, const IbKvView* kv, const int* dec_tokens, int n_dec, const int* positions, const int* seg_of_token,
                  int window, float scale, float* part_o, float* part_ml, void* out, int heads, int max_slices, int tiles_per_slice,
                  const void* kv_map, long long view_row0, unsigned* status, cudaStream_t stream, float softcap = 0.f, int sink = 0,
-                 const IbAttnTail* tail_in = nullptr) {
+                 const IbAttnTail* tail_in = nullptr, int keep = 0) {
   if (n_dec == 0) return 0;
+  IB_CHECK_ARG(keep >= 0 && (keep == 0 || (window > 0 && !raw)), "attention_decode_stream: %d kept positions need a window and finished queries", keep);
   IbAttnTail tail;
   if (!read_tail("attention_decode_stream", tail_in, sink, heads, kv, tail)) return 1;
   IB_CHECK_ARG(kv && kv->base && kv->block_table && kv_map, "attention_decode_stream: the cache view or the tensor map is a null pointer");
@@ -998,13 +1032,13 @@ int stream_entry(const void* q, const RawQkv* raw, const IbKvView* kv, const int
     if (raw) return launch_stream<128, true>(q, raw, kv, dec_tokens, n_dec, positions, seg_of_token, window, scale, part_o, part_ml, out, heads, max_slices,
                                              tiles_per_slice, map, view_row0, status, stream, softcap, sink, tail);
     return launch_stream<128, false>(q, raw, kv, dec_tokens, n_dec, positions, seg_of_token, window, scale, part_o, part_ml, out, heads, max_slices,
-                                     tiles_per_slice, map, view_row0, status, stream, softcap, sink, tail);
+                                     tiles_per_slice, map, view_row0, status, stream, softcap, sink, tail, keep);
   }
   if (kv->head_dim == 64) {
     if (raw) return launch_stream<64, true>(q, raw, kv, dec_tokens, n_dec, positions, seg_of_token, window, scale, part_o, part_ml, out, heads, max_slices,
                                             tiles_per_slice, map, view_row0, status, stream, softcap, sink, tail);
     return launch_stream<64, false>(q, raw, kv, dec_tokens, n_dec, positions, seg_of_token, window, scale, part_o, part_ml, out, heads, max_slices,
-                                    tiles_per_slice, map, view_row0, status, stream, softcap, sink, tail);
+                                    tiles_per_slice, map, view_row0, status, stream, softcap, sink, tail, keep);
   }
   return ib_set_error("attention_decode_stream: head_dim %d has no tensor-core kernel (64 and 128 have)", kv->head_dim);
 }
@@ -1023,14 +1057,14 @@ extern "C" int ib_attention_decode_stream(const void* q, const IbKvView* kv, con
 }
 
 // The same with capped scores (softcap > 0: softcap * tanh(score / softcap)) and, with sink, one added to the softmax's denominator;
-// window < 0 and tail as for ib_attention_decode_capped.
+// window < 0, tail and keep as for ib_attention_decode_capped.
 extern "C" int ib_attention_decode_stream_capped(const void* q, const IbKvView* kv, const int* dec_tokens, int n_dec, const int* positions,
                                                  const int* seg_of_token, int window, float scale, float* part_o, float* part_ml, void* out,
                                                  int heads, int max_slices, int tiles_per_slice, const void* kv_map, long long view_row0,
-                                                 float softcap, int sink, const IbAttnTail* tail, unsigned* status, cudaStream_t stream) {
+                                                 float softcap, int sink, const IbAttnTail* tail, int keep, unsigned* status, cudaStream_t stream) {
   IB_CHECK_ARG(q || n_dec == 0, "attention_decode_stream: q is a null pointer");
   return stream_entry(q, nullptr, kv, dec_tokens, n_dec, positions, seg_of_token, window, scale, part_o, part_ml, out, heads, max_slices,
-                      tiles_per_slice, kv_map, view_row0, status, stream, softcap, sink, tail);
+                      tiles_per_slice, kv_map, view_row0, status, stream, softcap, sink, tail, keep);
 }
 
 // The same from the output of the q/k/v projection (float32 partial sums qkv [P][T][(heads + 2 kv_heads) * head_dim],

@@ -218,7 +218,8 @@ __global__ void attention_generic_kernel(const A* __restrict__ q, IbKvView kv, c
                                          const int* __restrict__ seg_of_token, int window, float scale, A* __restrict__ out, int T,
                                          int heads, unsigned* __restrict__ status, int qk_dim, int v_dim, float softcap, int sink, int chunk,
                                          const float* __restrict__ sink_values, const float* __restrict__ gate, int gate_P, size_t gate_stride, int gate_row,
-                                         float out_scale, int out_row) {
+                                         float out_scale, int out_row, int keep) {
+  // keep > 0 (with a window): the first `keep` positions are seen as well, whatever the window.
   // qk_dim, v_dim: a query/key head's and a value head's size (at most the cache's row). softcap > 0: s <- softcap * tanh(s / softcap).
   // sink: the softmax has one more term whose score is 0 and which has no value (its denominator is 1 + sum exp(s)); with sink_values
   // the term's score is sink_values[head] instead (not scaled). chunk > 0: a position sees the earlier positions of its own block of
@@ -245,11 +246,13 @@ __global__ void attention_generic_kernel(const A* __restrict__ q, IbKvView kv, c
   float m = sink ? (sink_values ? sink_values[h] : 0.f) : -INFINITY, l = sink ? 1.f : 0.f;   // the sink is a key of its own score: it starts the running maximum and sum
   (void)row;
   const C* base = (const C*)kv.base;
-  for (int k0 = lo; k0 <= pos; k0 += 32) {
-    int key = k0 + lane;
+  // the keys that are kept and lie before the window come first, then the window; `base_key` turns a place in that row into a position
+  const int kept = min(keep, lo), base_key = lo - kept, n_keys = kept + pos - lo + 1;
+  for (int k0 = 0; k0 < n_keys; k0 += 32) {
+    const int key = k0 + lane < kept ? k0 + lane : base_key + k0 + lane;
     long long off = -1;
     float s = -INFINITY;
-    if (key <= pos) {
+    if (k0 + lane < n_keys) {
       off = ib::kv_offset(kv, seg, key, kvhead);
       if (off < 0) {
         atomicOr(status, IB_ERR_BAD_PAGE);
@@ -268,7 +271,7 @@ __global__ void attention_generic_kernel(const A* __restrict__ q, IbKvView kv, c
     l = l * corr + ib::warp_sum(p);
 #pragma unroll
     for (int r = 0; r < kMaxHeadDim / 32; r++) acc[r] *= corr;
-    int n = min(32, pos - k0 + 1);
+    int n = min(32, n_keys - k0);
     for (int jj = 0; jj < n; jj++) {
       float pj = __shfl_sync(0xffffffffu, p, jj);
       long long oj = __shfl_sync(0xffffffffu, off, jj);
@@ -370,8 +373,8 @@ extern "C" int ib_qk_norm_rope_kv(const float* qkv, int P, long long stride_p, c
 extern "C" int ib_attention_generic(const void* q, int act_dtype, const IbKvView* kv, const int* positions, const int* seg_of_token,
                                     int window, float scale, void* out, int T, int heads, unsigned* status, int qk_dim, int v_dim, float softcap, int sink,
                                     int chunk, const float* sink_values, const float* gate, int gate_P, long long gate_stride, int gate_row, float out_scale,
-                                    int out_row, cudaStream_t stream) {
-  // chunk, sink_values, gate, out_scale, out_row: see the kernel; out_row = 0 stands for heads * v_dim, gate = null for no gate.
+                                    int out_row, int keep, cudaStream_t stream) {
+  // keep: the first positions that are seen beside the window. chunk, sink_values, gate, out_scale, out_row: see the kernel; out_row = 0 stands for heads * v_dim, gate = null for no gate.
   // qk_dim, v_dim: 0 = the cache's row size; softcap: 0 = scores as they are; sink: 1 = one added to the softmax's denominator.
   if (T == 0) return 0;
   if (check_view("attention_generic", kv, heads)) return 1;
@@ -381,17 +384,18 @@ extern "C" int ib_attention_generic(const void* q, int act_dtype, const IbKvView
   IB_CHECK_ARG((act_dtype == IB_F32 && kv->dtype == IB_F32) || (act_dtype == IB_BF16 && kv->dtype == IB_BF16),
                "attention_generic: activation dtype %d and cache dtype %d must match", act_dtype, kv->dtype);
   if (out_row <= 0) out_row = heads * v_dim;
+  IB_CHECK_ARG(keep >= 0 && (keep == 0 || window > 0), "attention_generic: %d kept positions need a window", keep);
   IB_CHECK_ARG(out_row >= heads * v_dim && chunk >= 0 && (!sink_values || sink), "attention_generic: bad output row %d, chunk %d or sink values without a sink", out_row, chunk);
   long long items = (long long)T * heads;
   unsigned blocks = (unsigned)((items + kWarps - 1) / kWarps);
   if (act_dtype == IB_F32)
     ib::launch(attention_generic_kernel<float, float>, blocks, kWarps * 32, 0, stream, (const float*)q, *kv, positions, seg_of_token, window, scale,
                                                                               (float*)out, T, heads, status, qk_dim, v_dim, softcap, sink, chunk, sink_values, gate,
-                                                                              gate_P, (size_t)gate_stride, gate_row, out_scale, out_row);
+                                                                              gate_P, (size_t)gate_stride, gate_row, out_scale, out_row, keep);
   else
     ib::launch(attention_generic_kernel<__nv_bfloat16, __nv_bfloat16>, blocks, kWarps * 32, 0, stream, 
         (const __nv_bfloat16*)q, *kv, positions, seg_of_token, window, scale, (__nv_bfloat16*)out, T, heads, status, qk_dim, v_dim, softcap, sink, chunk,
-        sink_values, gate, gate_P, (size_t)gate_stride, gate_row, out_scale, out_row);
+        sink_values, gate, gate_P, (size_t)gate_stride, gate_row, out_scale, out_row, keep);
   IB_CHECK_LAUNCH("attention_generic");
   return 0;
 }

@@ -86,9 +86,10 @@ __global__ void __launch_bounds__(kThreads, 2)
     prefill_ws_kernel(const __nv_bfloat16* __restrict__ q, IbKvView kv, const int* __restrict__ tile_seg, const int* __restrict__ tile_row0,
                       const int* __restrict__ seg_start, const int* __restrict__ seg_pos0, int window, float scale_log2e,
                       __nv_bfloat16* __restrict__ out, int heads, const __grid_constant__ CUtensorMap kv_map, long long view_row0,
-                      unsigned long long wait_ns, unsigned* __restrict__ status, float cap_pre, int sink, IbAttnTail tail) {
+                      unsigned long long wait_ns, unsigned* __restrict__ status, float cap_pre, int sink, IbAttnTail tail, int keep) {
   // cap_pre != 0: a raw product s counts as tanh(s * cap_pre) (scale_log2e is then cap * log2 e); sink: the softmax has one more term
-  // of score 0 (or tail.sink_values[head]) that carries no value; window < 0: blocks of -window positions (ib::first_visible)
+  // of score 0 (or tail.sink_values[head]) that carries no value; window < 0: blocks of -window positions (ib::first_visible);
+  // keep > 0 (with a window): every row also sees the positions before `keep`: their key tiles come first
   using SM = Smem<HD>;
   constexpr int CPR = HD / 8, HB = HD / 64;
   constexpr int kTmemCols = 256;            // S0 [0,64) | S1 [64,128) | O [128, 128+HD); P_j lies over the first 32 columns of S_j
@@ -139,7 +140,9 @@ __global__ void __launch_bounds__(kThreads, 2)
   const int key_lo = ib::first_visible(pos_first, window);   // of the tile's rows, the first sees the earliest key
   const int lo_last = ib::first_visible(pos_last, window);   // a tile of keys from here on is seen by every row whose position has come
   const int kt_begin = key_lo / BN, kt_end = pos_last / BN + 1;
-  const int n_kt = kt_end - kt_begin;
+  const int n_pre = min((keep + BN - 1) / BN, kt_begin);   // tiles of kept keys before the window's first tile
+  const int n_kt = n_pre + kt_end - kt_begin;
+  auto key_tile = [&](int j) { return j < n_pre ? j : kt_begin + j - n_pre; };   // the j-th tile of keys that this CTA walks
   // a wait that ran out: say so once, and from then on nobody waits (the results are void, the status says so)
   auto wait = [&](uint64_t* bar, uint32_t parity) {
     if (sm100::mbar_try_wait(bar, parity) || *gave_up) return;
@@ -173,10 +176,10 @@ __global__ void __launch_bounds__(kThreads, 2)
     for (int j = 0; j < n_kt; j++) {
       const int rel = j * ppt;
       if ((rel & 31) == 0) {   // the pages of the next 32 boxes, one per lane
-        const int box = kt_begin * ppt + rel + lane;
+        const int box = rel + lane < n_pre * ppt ? rel + lane : (kt_begin - n_pre) * ppt + rel + lane;
         const int key0 = box * box_rows;
         held_row = -1;
-        if (key0 <= pos_last && key0 + box_rows > key_lo) {
+        if (key0 <= pos_last && (key0 + box_rows > key_lo || key0 < keep)) {
           const int col = boxes_per_page == 1 ? box : box / boxes_per_page;
           const int page = col < kv.table_stride ? kv.block_table[(size_t)seg * kv.table_stride + col] : -1;
           if (page >= 0 && page < kv.num_pages)
@@ -270,7 +273,7 @@ __global__ void __launch_bounds__(kThreads, 2)
 
     float m_ref = -INFINITY, l = 0.f;
     for (int j = 0; j < n_kt; j++) {
-      const int kt = kt_begin + j;
+      const int kt = key_tile(j);
       wait(&s_full[j & 1], (j >> 1) & 1);
       sm100::tc_fence_after();
       uint32_t sr[BN];
@@ -287,7 +290,7 @@ __global__ void __launch_bounds__(kThreads, 2)
 #pragma unroll
         for (int c = 0; c < BN; c++) {
           const int key = key0 + c;
-          const bool live = key <= my_pos && key >= my_lo;
+          const bool live = key <= my_pos && (key >= my_lo || key < keep);
           if (!live) sr[c] = 0xff800000u;  // -inf
         }
       }
@@ -389,7 +392,7 @@ __global__ void __launch_bounds__(kThreads, 2)
 template <int HD>
 int launch(const void* q, const IbKvView* kv, const int* tile_seg, const int* tile_row0, int n_tiles, const int* seg_start, const int* seg_pos0,
            int window, float scale, void* out, int heads, const CUtensorMap* kv_map, long long view_row0, unsigned* status, cudaStream_t stream,
-           float softcap, int sink, const IbAttnTail& tail) {
+           float softcap, int sink, const IbAttnTail& tail, int keep) {
   const float scale_log2e = (softcap > 0.f ? softcap : scale) * 1.4426950408889634f, cap_pre = softcap > 0.f ? scale / softcap : 0.f;
   static bool configured = false;
   if (!configured) {
@@ -398,7 +401,7 @@ int launch(const void* q, const IbKvView* kv, const int* tile_seg, const int* ti
     configured = true;
   }
   ib::launch(prefill_ws_kernel<HD>, dim3(heads, n_tiles), kThreads, Smem<HD>::kBytes, stream, (const __nv_bfloat16*)q, *kv, tile_seg, tile_row0,
-             seg_start, seg_pos0, window, scale_log2e, (__nv_bfloat16*)out, heads, *kv_map, view_row0, ib_wait_limit_ns(), status, cap_pre, sink, tail);
+             seg_start, seg_pos0, window, scale_log2e, (__nv_bfloat16*)out, heads, *kv_map, view_row0, ib_wait_limit_ns(), status, cap_pre, sink, tail, keep);
   IB_CHECK_LAUNCH("attention_prefill_ws");
   return 0;
 }
@@ -409,13 +412,15 @@ int launch(const void* q, const IbKvView* kv, const int* tile_seg, const int* ti
 // tiles that see the most keys first. kv_map: the tensor map of the view's pool (ib_make_kv_map), view_row0
 // the pool row where this view's keys of page 0, head 0 start.
 // softcap > 0: scores become softcap * tanh(score / softcap) after the scale; sink: the softmax's denominator has one added (or
-// exp(tail->sink_values[head])). window < 0: a position sees the earlier positions of its own block of -window positions. tail (may be
+// exp(tail->sink_values[head])). window < 0: a position sees the earlier positions of its own block of -window positions. keep (with a
+// window): the first positions of the request that are seen beside the window. tail (may be
 // null): the sink's scores, a gate and a constant on the output, the output's row length (IbAttnTail).
 extern "C" int ib_attention_prefill_ws_capped(const void* q, const IbKvView* kv, const int* tile_seg, const int* tile_row0, int n_tiles,
                                               const int* seg_start, const int* seg_pos0, int window, float scale, void* out, int heads,
-                                              const void* kv_map, long long view_row0, float softcap, int sink, const IbAttnTail* tail_in,
+                                              const void* kv_map, long long view_row0, float softcap, int sink, const IbAttnTail* tail_in, int keep,
                                               unsigned* status, cudaStream_t stream) {
   if (n_tiles == 0) return 0;
+  IB_CHECK_ARG(keep >= 0 && (keep == 0 || window > 0), "attention_prefill_ws: %d kept positions need a window", keep);
   const IbAttnTail tail = tail_in ? *tail_in : IbAttnTail{};
   IB_CHECK_ARG((!tail.sink_values || sink) && (tail.out_row == 0 || (tail.out_row >= heads * (kv ? kv->head_dim : 0) && tail.out_row % 8 == 0)) &&
                    (!tail.gate || (tail.gate_parts >= 1 && tail.gate_row >= heads)),
@@ -431,16 +436,16 @@ extern "C" int ib_attention_prefill_ws_capped(const void* q, const IbKvView* kv,
   IB_CHECK_ARG(kv->page_stride % kv->head_dim == 0 && kv->v_offset % kv->head_dim == 0, "attention_prefill_ws: strides are not whole rows");
   if (kv->head_dim == 128)
     return launch<128>(q, kv, tile_seg, tile_row0, n_tiles, seg_start, seg_pos0, window, scale, out, heads, (const CUtensorMap*)kv_map, view_row0,
-                       status, stream, softcap, sink, tail);
+                       status, stream, softcap, sink, tail, keep);
   if (kv->head_dim == 64)
     return launch<64>(q, kv, tile_seg, tile_row0, n_tiles, seg_start, seg_pos0, window, scale, out, heads, (const CUtensorMap*)kv_map, view_row0,
-                      status, stream, softcap, sink, tail);
+                      status, stream, softcap, sink, tail, keep);
   return ib_set_error("attention_prefill_ws: head_dim %d has no tensor-core kernel (64 and 128 have)", kv->head_dim);
 }
 
 extern "C" int ib_attention_prefill_ws(const void* q, const IbKvView* kv, const int* tile_seg, const int* tile_row0, int n_tiles,
                                        const int* seg_start, const int* seg_pos0, int window, float scale, void* out, int heads,
                                        const void* kv_map, long long view_row0, unsigned* status, cudaStream_t stream) {
-  return ib_attention_prefill_ws_capped(q, kv, tile_seg, tile_row0, n_tiles, seg_start, seg_pos0, window, scale, out, heads, kv_map, view_row0, 0.f, 0, nullptr,
+  return ib_attention_prefill_ws_capped(q, kv, tile_seg, tile_row0, n_tiles, seg_start, seg_pos0, window, scale, out, heads, kv_map, view_row0, 0.f, 0, nullptr, 0,
                                         status, stream);
 }

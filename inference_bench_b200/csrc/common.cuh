@@ -91,6 +91,11 @@ __device__ __forceinline__ float xielu(float z, float ap, float an) {
   return z > 0.f ? __fmaf_rn(ap * z, z, 0.5f * z) : __fmaf_rn(an, expm1f(z) - z, 0.5f * z);
 }
 
+__device__ __forceinline__ float relu2(float z) {   // the square of max(z, 0)
+  const float r = fmaxf(z, 0.f);
+  return r * r;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

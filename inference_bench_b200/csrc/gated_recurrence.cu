@@ -13,6 +13,11 @@
 //    chunks in order (S_in of the next = decay * S_in + the chunk's closing state, elementwise, ending in the request's state) and
 //    `chunk_apply` adds (q_t * decay)^T S_in to every output. The three give what the walk over the whole segment gives, up to
 //    rounding, with as many CTAs as the segment has chunks; which path a segment takes depends on its own length only.
+//  * Other forms of the same walk: a fixed decay per head with a key (form 1: q, k, v behind a SiLU; form 2: q and k turned by the token's
+//    angles, the key scaled, v as it is), and a decay per channel and token with a bonus for the current token (form 3:
+//    o = (S + diag(u) k v^T)^T r before S <- diag(w) S + k v^T).
+//  * decay_rows: the decays of form 3, exp(-exp(w0 + W2 tanh(low))), from the float32 sums of the low-rank projection.
+//  * head_norm_gate: out[t, a, :] = w * o / sqrt(mean(o^2) + eps) * silu(gate), the weight (optional) and the gate per channel of all heads.
 //  * head_rmsnorm: out[t, a, :] = w * o[t, a, :] / sqrt(mean(o^2) + eps), into the activation dtype.
 #include <type_traits>
 
@@ -23,14 +28,27 @@ namespace {
 constexpr int kChunk = 16;   // tokens prepared at a time
 
 // RPT: rows of S a thread holds (for each of its two columns); kCols: value columns per CTA (32, or 16 where a thread holds sixteen rows)
-template <int RPT, int kCols>
-__global__ void __launch_bounds__(kCols * 16) gated_recurrence_kernel(const float* __restrict__ proj, int P, size_t stride_p, int R, const float* __restrict__ f_bias,
+// BONUS: form 3
+struct RecurrenceExtras {
+  const float* cos_t;   // form 2: float32 [T][rot_half], the angles of the first 2 * rot_half entries of q and k (entry i with i + rot_half), or null
+  const float* sin_t;
+  int rot_half;
+  float k_scale;        // form 2: factor on the key after the rotation
+  const float* decay;   // form 3: float32 [T][heads * D]
+};
+
+template <int RPT, int kCols, bool BONUS>
+__global__ void __launch_bounds__(kCols * 16) gated_recurrence_kernel(const float* __restrict__ q_src, const float* __restrict__ f_src, const float* __restrict__ v_src,
+                                        int P, size_t stride_p, int R, const float* __restrict__ f_bias,
                                         const float* __restrict__ lower, float* __restrict__ state, size_t slot_stride, const int* __restrict__ seg_start,
                                         const int* __restrict__ seg_slot, float* __restrict__ o_out, int heads, int D, int V, int DS,
                                         const int* __restrict__ seg_list, const int* __restrict__ chunks, float* __restrict__ chunk_state,
-                                        float* __restrict__ chunk_decay, float* __restrict__ qa_out, int form, int q_col, int f_col, int v_col) {
-  // form 0: the gated form above (columns [q | f | v] at q_col, f_col, v_col of a row of R). form 1: a fixed decay per head and a key:
-  // S <- lower[a] S + k v^T with q, k, v = silu of the columns at q_col, f_col, v_col (f_bias is not read; lower holds one decay a head).
+                                        float* __restrict__ chunk_decay, float* __restrict__ qa_out, int form, RecurrenceExtras ex) {
+  // q_src, f_src, v_src: float32 partial sums of the three parts, rows of R entries, P of them stride_p apart.
+  // form 0: the gated form above (q, z_f, v). form 1: a fixed decay per head and a key:
+  // S <- lower[a] S + k v^T with q, k, v = silu of q_src, f_src, v_src (f_bias is not read; lower holds one decay a head).
+  // form 2: the same with q and k turned by ex's angles, k times ex.k_scale, and no SiLU anywhere.
+  // form 3 (BONUS): r, k, v as they are, decays ex.decay, lower = u [heads * D]: o = (S + diag(u) k v^T)^T r, then S <- diag(decay) S + k v^T.
   // seg_list: the segments this launch walks (null: all). chunks != null: blockIdx.x is a chunk (first row, rows) that starts from a zero
   // state and leaves its closing state in chunk_state[chunk][head], its decay in chunk_decay[chunk][head] and q * decay in qa_out[row][head].
   extern __shared__ float sm[];   // q[kChunk][D], f[kChunk][D], g[kChunk][D], v[kChunk][kCols], running decay [D]
@@ -64,15 +82,48 @@ __global__ void __launch_bounds__(kCols * 16) gated_recurrence_kernel(const floa
     st[r][0] = (!chunks && d < D && j < V) ? S[(size_t)d * V + j] : 0.f;
     st[r][1] = (!chunks && d < D && j + 1 < V) ? S[(size_t)d * V + j + 1] : 0.f;
   }
-  const int q_off = q_col + a * D, f_off = f_col + a * D, v_off = v_col + a * V + j0;
+  const int q_off = a * D, v_off = a * V + j0;
+  float u[BONUS ? RPT : 1];
+  if constexpr (BONUS) {
+#pragma unroll
+    for (int r = 0; r < RPT; r++) u[r] = d0 + r < D ? lower[a * D + d0 + r] : 0.f;
+  }
   for (int c0 = t0; c0 < t1; c0 += kChunk) {
     const int n = min(kChunk, t1 - c0);
     __syncthreads();
+    if (!BONUS && form == 2) {   // a thread takes a pair of entries that are turned together, or one that is not
+      const int half = ex.rot_half, per = D - half;
+      for (int i = tid; i < n * per; i += blockDim.x) {
+        const int tt = i / per, w = i % per;
+        const size_t row = (size_t)(c0 + tt) * R + q_off;
+        const int d = w < half ? w : w + half, d2 = w + half;
+        float zq = q_src[row + d], zk = f_src[row + d];
+        for (int p = 1; p < P; p++) zq += q_src[p * stride_p + row + d], zk += f_src[p * stride_p + row + d];
+        if (w < half) {
+          float yq = q_src[row + d2], yk = f_src[row + d2];
+          for (int p = 1; p < P; p++) yq += q_src[p * stride_p + row + d2], yk += f_src[p * stride_p + row + d2];
+          const float c = ex.cos_t[(size_t)(c0 + tt) * half + w], s = ex.sin_t[(size_t)(c0 + tt) * half + w];
+          sq[tt * D + d2] = yq * c + zq * s;
+          sg[tt * D + d2] = (yk * c + zk * s) * ex.k_scale;
+          sf[tt * D + d2] = lower[a];
+          zq = zq * c - yq * s, zk = zk * c - yk * s;
+        }
+        sq[tt * D + d] = zq;
+        sg[tt * D + d] = zk * ex.k_scale;
+        sf[tt * D + d] = lower[a];
+      }
+    } else
     for (int i = tid; i < n * D; i += blockDim.x) {
       const int tt = i / D, d = i % D;
-      const float* src = proj + (size_t)(c0 + tt) * R;
-      float zq = src[q_off + d], zf = src[f_off + d];
-      for (int p = 1; p < P; p++) zq += src[p * stride_p + q_off + d], zf += src[p * stride_p + f_off + d];
+      const size_t row = (size_t)(c0 + tt) * R + q_off + d;
+      float zq = q_src[row], zf = f_src[row];
+      for (int p = 1; p < P; p++) zq += q_src[p * stride_p + row], zf += f_src[p * stride_p + row];
+      if constexpr (BONUS) {
+        sq[i] = zq;
+        sg[i] = zf;
+        sf[i] = ex.decay[(size_t)(c0 + tt) * heads * D + q_off + d];
+        continue;
+      }
       sq[i] = zq / (1.f + expf(-zq));
       if (form == 1) {
         sf[i] = lower[a];
@@ -90,7 +141,7 @@ __global__ void __launch_bounds__(kCols * 16) gated_recurrence_kernel(const floa
       const int tt = i / kCols, c = i % kCols;
       float z = 0.f;
       if (j0 + c < V) {
-        const float* src = proj + (size_t)(c0 + tt) * R + v_off + c;
+        const float* src = v_src + (size_t)(c0 + tt) * R + v_off + c;
         z = src[0];
         for (int p = 1; p < P; p++) z += src[p * stride_p];
         if (form == 1) z = z / (1.f + expf(-z));
@@ -102,8 +153,9 @@ __global__ void __launch_bounds__(kCols * 16) gated_recurrence_kernel(const floa
       for (int d = tid; d < D; d += blockDim.x) {
         float r = run[d];
         for (int tt = 0; tt < n; tt++) {
-          r *= sf[tt * D + d];
+          if (!BONUS) r *= sf[tt * D + d];
           qa_out[((size_t)(c0 + tt) * heads + a) * D + d] = sq[tt * D + d] * r;
+          if (BONUS) r *= sf[tt * D + d];   // the current token's decay comes after its output
         }
         run[d] = r;
       }
@@ -128,6 +180,19 @@ __global__ void __launch_bounds__(kCols * 16) gated_recurrence_kernel(const floa
         }
       }
       float acc0 = 0.f, acc1 = 0.f;
+      if constexpr (BONUS) {
+        float own = 0.f;   // this thread's rows of r . (u k)
+#pragma unroll
+        for (int r = 0; r < RPT; r++) {
+          own = __fmaf_rn(q[r], u[r] * g[r], own);
+          acc0 = __fmaf_rn(st[r][0], q[r], acc0);
+          acc1 = __fmaf_rn(st[r][1], q[r], acc1);
+          st[r][0] = __fmaf_rn(f[r], st[r][0], g[r] * v0);
+          st[r][1] = __fmaf_rn(f[r], st[r][1], g[r] * v1);
+        }
+        acc0 = __fmaf_rn(own, v0, acc0);
+        acc1 = __fmaf_rn(own, v1, acc1);
+      } else
 #pragma unroll
       for (int r = 0; r < RPT; r++) {   // rows beyond D have f = g = q = 0: their state stays zero
         st[r][0] = __fmaf_rn(f[r], st[r][0], g[r] * v0);
@@ -248,12 +313,117 @@ __global__ void head_rmsnorm_kernel(const float* __restrict__ o, const float* __
   for (int i = lane; i < V; i += 32) out[item * V + i] = ib::from_f32<O>(w[i] * (src[i] * inv));
 }
 
+// dec[t][c] = exp(-exp(w0[c] + sum_j w2[j][c] tanh(low[t][j]))): TT tokens and 256 channels a CTA; the tanh values are made once per CTA.
+template <int TT>
+__global__ void __launch_bounds__(256) decay_rows_kernel(const float* __restrict__ low, int P, size_t stride_p, int rank, const float* __restrict__ w2,
+                                                         const float* __restrict__ w0, float* __restrict__ dec, int T, int C) {
+  extern __shared__ float th[];   // [rank][TT]
+  ib::pdl_launch_dependents();
+  ib::pdl_wait();
+  const int t0 = blockIdx.y * TT, n = min(TT, T - t0);
+  for (int i = threadIdx.x; i < rank * TT; i += blockDim.x) {
+    const int tt = i / rank, j = i % rank;
+    float z = 0.f;
+    if (tt < n) {
+      const float* src = low + (size_t)(t0 + tt) * rank + j;
+      z = src[0];
+      for (int p = 1; p < P; p++) z += src[p * stride_p];
+    }
+    th[j * TT + tt] = tanhf(z);
+  }
+  __syncthreads();
+  const int c = blockIdx.x * 256 + threadIdx.x;
+  if (c >= C) return;
+  float acc[TT];
+#pragma unroll
+  for (int tt = 0; tt < TT; tt++) acc[tt] = 0.f;
+#pragma unroll 4
+  for (int j = 0; j < rank; j++) {
+    const float w = w2[(size_t)j * C + c];
+#pragma unroll
+    for (int tt = 0; tt < TT; tt++) acc[tt] = __fmaf_rn(w, th[j * TT + tt], acc[tt]);
+  }
+  const float b = w0[c];
+#pragma unroll
+  for (int tt = 0; tt < TT; tt++)
+    if (tt < n) dec[(size_t)(t0 + tt) * C + c] = expf(-expf(acc[tt] + b));
+}
+
+// A warp per (token, head): the head's norm, a weight per channel (or none), the gate's SiLU from its float32 partial sums.
+template <typename O>
+__global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, float eps, const float* __restrict__ gate, int gate_P, size_t gate_stride,
+                                      int gate_row, O* __restrict__ out, long long items, int heads, int V) {
+  ib::pdl_launch_dependents();
+  ib::pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + warp;
+  if (item >= items) return;
+  const long long t = item / heads;
+  const int a = (int)(item - t * heads);
+  const float* src = o + item * V;
+  const float* gr = gate + t * gate_row + a * V;
+  float ss = 0.f;
+  for (int i = lane; i < V; i += 32) ss = __fmaf_rn(src[i], src[i], ss);
+  const float inv = 1.f / sqrtf(ib::warp_sum(ss) / (float)V + eps);
+  for (int i = lane; i < V; i += 32) {
+    float g = gr[i];
+    for (int p = 1; p < gate_P; p++) g += gr[p * gate_stride + i];
+    const float y = w ? w[a * V + i] * (src[i] * inv) : src[i] * inv;
+    out[item * V + i] = ib::from_f32<O>(y * (g / (1.f + expf(-g))));
+  }
+}
+
 }  // namespace
 
 // seg_list: int32 [n_segments] of the segments to walk (null: segments 0 .. n_segments - 1).
 // chunks: null, or int32 [n_segments][2] = (first row, rows <= 64) of chunks that each start from a zero state (n_segments then counts
 // chunks); chunk_state float32 [chunks][heads][D][V], chunk_decay float32 [chunks][heads][D] and qa float32 [T][heads][D] receive what
 // ib_recurrence_chunks_finish needs.
+namespace {
+int launch_recurrence(const float* q_src, const float* f_src, const float* v_src, int P, long long stride_p, int R, const float* f_bias, const float* lower, float* state,
+                      long long slot_stride, const int* seg_start, const int* seg_slot, int n_segments, float* o_out, int heads, int D, int V, const int* seg_list,
+                      const int* chunks, float* chunk_state, float* chunk_decay, float* qa, int form, const RecurrenceExtras& ex, cudaStream_t stream) {
+  if (n_segments == 0) return 0;
+  IB_CHECK_ARG(!chunks || (chunk_state && chunk_decay && qa), "recurrence: chunks need their state, decay and query buffers");
+  IB_CHECK_ARG(n_segments > 0 && P >= 1 && heads > 0 && D > 0 && V > 0, "recurrence: bad sizes segments=%d P=%d heads=%d D=%d V=%d", n_segments, P, heads, D, V);
+  IB_CHECK_ARG(D <= 512, "recurrence: a head's key size %d is above 512", D);
+  IB_CHECK_ARG(R >= heads * D && R >= heads * V, "recurrence: rows of %d entries do not hold %d heads of %d and %d", R, heads, D, V);
+  const int rpt = D <= 256 ? 8 : 16, kCols = D <= 256 ? 32 : 16;
+  IB_CHECK_ARG(heads <= 65535 && (V + kCols - 1) / kCols <= 65535, "recurrence: the grid is too large");
+  int DS = 1;
+  while (DS * rpt < D) DS *= 2;
+  if (DS < 2) DS = 2;   // a CTA is a whole warp at least (kCols / 2 column pairs x DS)
+  const size_t smem = ((size_t)kChunk * (3 * D + kCols) + D) * sizeof(float);
+  const dim3 grid((unsigned)n_segments, (unsigned)heads, (unsigned)((V + kCols - 1) / kCols));
+  auto go = [&](auto kernel) {
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    ib::launch(kernel, grid, kCols / 2 * DS, smem, stream, q_src, f_src, v_src, P, (size_t)stride_p, R, f_bias, lower, state, (size_t)slot_stride, seg_start, seg_slot, o_out,
+               heads, D, V, DS, seg_list, chunks, chunk_state, chunk_decay, qa, form, ex);
+  };
+  if (rpt == 8 && form == 3) go(gated_recurrence_kernel<8, 32, true>);
+  else if (rpt == 8) go(gated_recurrence_kernel<8, 32, false>);
+  else if (form == 3) go(gated_recurrence_kernel<16, 16, true>);
+  else go(gated_recurrence_kernel<16, 16, false>);
+  IB_CHECK_LAUNCH("recurrence");
+  return 0;
+}
+}  // namespace
+
+// The forms with parts of their own (2: turned queries and keys with a fixed decay per head; 3: a decay per channel and token, a bonus for the
+// current token): q, k, v float32 partial sums [P][T][row] each, stride_p elements apart. The other arguments as for ib_gated_recurrence.
+extern "C" int ib_recurrence_parts(const float* q, const float* k, const float* v, int P, long long stride_p, int row, const float* head_param, float* state,
+                                   long long slot_stride, const int* seg_start, const int* seg_slot, int n_segments, float* o_out, int heads, int D, int V,
+                                   const int* seg_list, const int* chunks, float* chunk_state, float* chunk_decay, float* qa, int form, const float* cos_t,
+                                   const float* sin_t, int rot_half, float k_scale, const float* decay, cudaStream_t stream) {
+  if (n_segments == 0) return 0;
+  IB_CHECK_ARG(form == 2 || form == 3, "recurrence_parts: form %d is not 2 or 3", form);
+  IB_CHECK_ARG(q && k && v && head_param && (form != 3 || decay), "recurrence_parts: a part, the decays or the bonus is missing");
+  IB_CHECK_ARG(rot_half >= 0 && 2 * rot_half <= D && (rot_half == 0 || (cos_t && sin_t)), "recurrence_parts: a rotation of %d entries of %d", 2 * rot_half, D);
+  RecurrenceExtras ex = {cos_t, sin_t, rot_half, k_scale, decay};
+  return launch_recurrence(q, k, v, P, stride_p, row, nullptr, head_param, state, slot_stride, seg_start, seg_slot, n_segments, o_out, heads, D, V, seg_list, chunks, chunk_state,
+                           chunk_decay, qa, form, ex, stream);
+}
+
 extern "C" int ib_gated_recurrence(const float* proj, int P, long long stride_p, const float* f_bias, const float* lower, float* state, long long slot_stride,
                                    const int* seg_start, const int* seg_slot, int n_segments, float* o_out, int heads, int D, int V, const int* seg_list,
                                    const int* chunks, float* chunk_state, float* chunk_decay, float* qa, int form, int row, int q_col, int f_col, int v_col,
@@ -261,30 +431,13 @@ extern "C" int ib_gated_recurrence(const float* proj, int P, long long stride_p,
   // form, row, q_col, f_col, v_col: see the kernel; row <= 0 stands for the gated form's own row [q | f | v] with its columns.
   if (n_segments == 0) return 0;
   IB_CHECK_ARG(form == 0 || form == 1, "gated_recurrence: form %d is not known (0: gated, 1: fixed decay with a key)", form);
-  IB_CHECK_ARG(!chunks || (chunk_state && chunk_decay && qa), "gated_recurrence: chunks need their state, decay and query buffers");
-  IB_CHECK_ARG(n_segments > 0 && P >= 1 && heads > 0 && D > 0 && V > 0, "gated_recurrence: bad sizes segments=%d P=%d heads=%d D=%d V=%d", n_segments, P, heads, D, V);
-  IB_CHECK_ARG(D <= 512, "gated_recurrence: a head's key size %d is above 512", D);
-  const int rpt = D <= 256 ? 8 : 16, kCols = D <= 256 ? 32 : 16;
-  IB_CHECK_ARG(heads <= 65535 && (V + kCols - 1) / kCols <= 65535, "gated_recurrence: the grid is too large");
-  int DS = 1;
-  while (DS * rpt < D) DS *= 2;
-  if (DS < 2) DS = 2;   // a CTA is a whole warp at least (kCols / 2 column pairs x DS)
   int R = 2 * heads * D + heads * V;
   if (row <= 0) q_col = 0, f_col = heads * D, v_col = 2 * heads * D;
   else R = row;
   IB_CHECK_ARG(q_col >= 0 && f_col >= 0 && v_col >= 0 && q_col + heads * D <= R && f_col + heads * D <= R && v_col + heads * V <= R,
                "gated_recurrence: the columns %d, %d, %d do not fit a row of %d", q_col, f_col, v_col, R);
-  const size_t smem = ((size_t)kChunk * (3 * D + kCols) + D) * sizeof(float);
-  const dim3 grid((unsigned)n_segments, (unsigned)heads, (unsigned)((V + kCols - 1) / kCols));
-  auto go = [&](auto kernel) {
-    if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    ib::launch(kernel, grid, kCols / 2 * DS, smem, stream, proj, P, (size_t)stride_p, R, f_bias, lower, state, (size_t)slot_stride, seg_start, seg_slot, o_out, heads, D, V, DS,
-               seg_list, chunks, chunk_state, chunk_decay, qa, form, q_col, f_col, v_col);
-  };
-  if (rpt == 8) go(gated_recurrence_kernel<8, 32>);
-  else go(gated_recurrence_kernel<16, 16>);
-  IB_CHECK_LAUNCH("gated_recurrence");
-  return 0;
+  return launch_recurrence(proj + q_col, proj + f_col, proj + v_col, P, stride_p, R, f_bias, lower, state, slot_stride, seg_start, seg_slot, n_segments, o_out, heads, D, V,
+                           seg_list, chunks, chunk_state, chunk_decay, qa, form, RecurrenceExtras{}, stream);
 }
 
 // After ib_gated_recurrence on chunks: long_segs int32 [n_long][3] = (segment, its first chunk, its chunks), chunks as above (n_chunks of them).
@@ -308,5 +461,35 @@ extern "C" int ib_head_rmsnorm(const float* o, const float* w, float eps, void* 
   else if (out_dtype == IB_BF16) ib::launch(head_rmsnorm_kernel<__nv_bfloat16>, grid, 128, 0, stream, o, w, eps, (__nv_bfloat16*)out, items, V);
   else return ib_set_error("head_rmsnorm: unknown output dtype %d", out_dtype);
   IB_CHECK_LAUNCH("head_rmsnorm");
+  return 0;
+}
+
+extern "C" int ib_decay_rows(const float* low, int P, long long stride_p, int rank, const float* w2, const float* w0, float* dec, int T, int C, cudaStream_t stream) {
+  if (T == 0) return 0;
+  IB_CHECK_ARG(T > 0 && C > 0 && rank > 0 && P >= 1, "decay_rows: bad sizes T=%d channels=%d rank=%d P=%d", T, C, rank, P);
+  auto go = [&](auto kernel, int tt) {
+    const size_t smem = (size_t)rank * tt * sizeof(float);
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    ib::launch(kernel, dim3((unsigned)((C + 255) / 256), (unsigned)((T + tt - 1) / tt)), 256, smem, stream, low, P, (size_t)stride_p, rank, w2, w0, dec, T, C);
+  };
+  IB_CHECK_ARG(rank <= 3072 && T <= 65535, "decay_rows: rank %d (at most 3072) or T=%d rows are too large", rank, T);
+  if (T >= 256) go(decay_rows_kernel<16>, 16);   // (a channel's sum runs over the rank in the same order in both forms)
+  else go(decay_rows_kernel<1>, 1);
+  IB_CHECK_LAUNCH("decay_rows");
+  return 0;
+}
+
+// gate: float32 partial sums [gate_P][T][gate_row], offset to the first head's first column.
+extern "C" int ib_head_norm_gate(const float* o, const float* w, float eps, const float* gate, int gate_P, long long gate_stride, int gate_row, void* out, int out_dtype,
+                                 int T, int heads, int V, cudaStream_t stream) {
+  if (T == 0) return 0;
+  IB_CHECK_ARG(T > 0 && heads > 0 && V > 0 && gate && gate_P >= 1 && gate_row >= heads * V, "head_norm_gate: bad sizes T=%d heads=%d V=%d gate rows of %d", T, heads, V, gate_row);
+  const long long items = (long long)T * heads;
+  const unsigned grid = (unsigned)((items + 3) / 4);
+  if (out_dtype == IB_F32) ib::launch(head_norm_gate_kernel<float>, grid, 128, 0, stream, o, w, eps, gate, gate_P, (size_t)gate_stride, gate_row, (float*)out, items, heads, V);
+  else if (out_dtype == IB_BF16)
+    ib::launch(head_norm_gate_kernel<__nv_bfloat16>, grid, 128, 0, stream, o, w, eps, gate, gate_P, (size_t)gate_stride, gate_row, (__nv_bfloat16*)out, items, heads, V);
+  else return ib_set_error("head_norm_gate: unknown output dtype %d", out_dtype);
+  IB_CHECK_LAUNCH("head_norm_gate");
   return 0;
 }

@@ -36,6 +36,7 @@ struct RowsArgs {
   const float* gate;
   int gate_P, gate_row;
   long long gate_stride;
+  int relu2;     // grouped mode without a gate half: the output is the square of max(product, 0)
 };
 
 template <bool GATED, typename O>
@@ -177,6 +178,7 @@ __global__ void __launch_bounds__(128) gemm_rows_mma_kernel(RowsArgs p) {
           if (n >= N) continue;
           float v = acc[m][nt][2 * h + c];
           if constexpr (GATED) v = (v / (1.f + expf(-v))) * acu[m][nt][2 * h + c];
+          else if (p.relu2) v = ib::relu2(v);
           dst[n] = ib::from_f32<O>(v * f);
         }
     }
@@ -203,12 +205,15 @@ int launch_rows(const RowsArgs& a, dim3 grid, int gated, int out_dtype, cudaStre
 }  // namespace
 
 extern "C" int ib_gemm_grouped_mma(const void* x, const int* src_row, const void* w, void* out, int out_dtype, const int* offsets, const int* tile_start, int R, int E,
-                                   int N, int K, int gated, cudaStream_t stream) {
+                                   int N, int K, int act, cudaStream_t stream) {
+  // act: 0 the product, 1 silu(gate) * up (w holds gate rows, then up rows), 2 the square of max(product, 0)
   if (R == 0 || N == 0) return 0;
+  IB_CHECK_ARG(act >= 0 && act <= 2, "gemm_grouped_mma: activation %d is not known", act);
+  const int gated = act == 1;
   IB_CHECK_ARG(R > 0 && E > 0 && N > 0 && K > 0, "gemm_grouped_mma: bad sizes rows=%d experts=%d N=%d K=%d", R, E, N, K);
   RowsArgs a = {};
   a.x = (const __nv_bfloat16*)x, a.w = (const __nv_bfloat16*)w, a.out = out, a.src_row = src_row, a.offsets = offsets, a.tile_start = tile_start;
-  a.n_groups = E, a.N = N, a.K = K, a.grouped = 1;
+  a.n_groups = E, a.N = N, a.K = K, a.grouped = 1, a.relu2 = act == 2;
   return launch_rows(a, dim3((N + TN - 1) / TN, R / TM + E, 1), gated, out_dtype, stream, "gemm_grouped_mma");
 }
 

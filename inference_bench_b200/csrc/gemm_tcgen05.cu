@@ -29,6 +29,7 @@ constexpr int kThreads = 192;
 constexpr int EPI_STORE = 0;   // float32 partial products
 constexpr int EPI_SWIGLU = 1;  // accumulator 0 = gate, accumulator 1 = up -> bfloat16 silu(gate) * up
 constexpr int EPI_XIELU = 3;   // one or two accumulators of plain rows -> bfloat16 xielu(product) with the two numbers of act_pq
+constexpr int EPI_RELU2 = 4;   // the same with the square of max(product, 0)
 constexpr int EPI_SWIGLU_HALF = 2;  // one accumulator: rows 0-63 = 64 gate rows, rows 64-127 = the matching 64 up rows -> bfloat16 silu(gate) * up
 // (for a handful of tokens: as many CTAs as the plain product has, I / 64, so the weights stream as fast, and neither the
 // float32 [T, 2I] intermediate nor the SiLU-mul kernel exists)
@@ -185,7 +186,7 @@ __global__ void __launch_bounds__(kThreads, 1)
     ok = __all_sync(0xffffffffu, ok);
     constexpr int CH = BN < 32 ? 16 : 32;
     const uint32_t lane_addr = tmem + ((uint32_t)(q * 32) << 16);
-    if (ok && (EPI == EPI_STORE || EPI == EPI_XIELU)) {
+    if (ok && (EPI == EPI_STORE || EPI == EPI_XIELU || EPI == EPI_RELU2)) {
       float* dst = (float*)out_ + (size_t)split * T * N;
       __nv_bfloat16* dst_act = (__nv_bfloat16*)out_;   // EPI_XIELU: the whole k-range is this CTA's, the activation is applied here
       float ap = 0.f, an = 0.f;
@@ -213,6 +214,8 @@ __global__ void __launch_bounds__(kThreads, 1)
               if (t < t_end) {
                 if constexpr (EPI == EPI_XIELU)
                   dst_act[(size_t)t * N + n] = __float2bfloat16_rn(ib::xielu(__uint_as_float(r[c]), ap, an));
+                else if constexpr (EPI == EPI_RELU2)
+                  dst_act[(size_t)t * N + n] = __float2bfloat16_rn(ib::relu2(__uint_as_float(r[c])));
                 else
                   dst[(size_t)t * N + n] = __uint_as_float(r[c]);
               }
@@ -414,6 +417,32 @@ extern "C" int ib_gemm_xielu_tcgen05(const void* x, const void* w, void* act, in
   }
 }
 
+// x [T, K], w [N, K] bfloat16 -> act [T, N] bfloat16 = max(x w^T, 0)^2: the product with the activation in its epilogue. bn, wide: as for
+// ib_gemm_tcgen05; the k-range is not split.
+extern "C" int ib_gemm_relu2_tcgen05(const void* x, const void* w, void* act, int T, int N, int K, int bn, int wide, unsigned* status, cudaStream_t stream) {
+  if (T == 0 || N == 0) return 0;
+  if (check_common("gemm_relu2_tcgen05", x, w, T, N, K, bn)) return 1;
+  const int total_kt = (K + BK - 1) / BK;
+  CUtensorMap tw, tx;
+  if (make_tmap(&tw, w, N, K, BM)) return 1;
+  if (make_tmap(&tx, x, T, K, bn)) return 1;
+  if (wide) {
+    switch (bn) {
+      case 128: return launch<128, 2, EPI_RELU2>(tw, tx, act, T, N, K, 1, total_kt, BM, status, stream);
+      case 256: return launch<256, 2, EPI_RELU2>(tw, tx, act, T, N, K, 1, total_kt, BM, status, stream);
+      default: return ib_set_error("gemm_relu2_tcgen05: 256 rows of w per CTA go with token tiles of 128 or 256, not %d", bn);
+    }
+  }
+  switch (bn) {
+    case 16: return launch<16, 1, EPI_RELU2>(tw, tx, act, T, N, K, 1, total_kt, 0, status, stream);
+    case 32: return launch<32, 1, EPI_RELU2>(tw, tx, act, T, N, K, 1, total_kt, 0, status, stream);
+    case 64: return launch<64, 1, EPI_RELU2>(tw, tx, act, T, N, K, 1, total_kt, 0, status, stream);
+    case 128: return launch<128, 1, EPI_RELU2>(tw, tx, act, T, N, K, 1, total_kt, 0, status, stream);
+    case 256: return launch<256, 1, EPI_RELU2>(tw, tx, act, T, N, K, 1, total_kt, 0, status, stream);
+    default: return ib_set_error("gemm_relu2_tcgen05: token tile %d is not one of 16, 32, 64, 128, 256", bn);
+  }
+}
+
 // SwiGLU front half in one kernel: w [2*I, K] = gate rows then up rows; act [T, I] bfloat16 =
 // silu(x gate^T) * (x up^T). bn: 16 or 32 tokens per CTA, or 64 with half != 0 (64 gate rows and their 64 up rows in one
 // accumulator: I must be a multiple of 64), or 64, 128 or 256 (128 gate rows and 128 up rows in two accumulators).
@@ -461,6 +490,28 @@ extern "C" int ib_gemm_grouped_tcgen05(const void* x, const void* w, float* out,
     case 128: return launch<128, 1, EPI_STORE>(tw, tx, out, R, N, K, 1, total_kt, 0, status, stream, 0, g);
     case 256: return launch<256, 1, EPI_STORE>(tw, tx, out, R, N, K, 1, total_kt, 0, status, stream, 0, g);
     default: return ib_set_error("gemm_grouped_tcgen05: token tile %d is not one of 16, 32, 64, 128, 256", bn);
+  }
+}
+
+// The same with act [R, N] bfloat16 = max(x w[e]^T, 0)^2 (experts without a gate).
+extern "C" int ib_gemm_grouped_relu2_tcgen05(const void* x, const void* w, void* act, int R, int N, int K, int bn, const int* offsets, const int* tiles, int E,
+                                             unsigned* status, cudaStream_t stream) {
+  if (R == 0 || N == 0) return 0;
+  if (check_common("gemm_grouped_relu2_tcgen05", x, w, R, N, K, bn)) return 1;
+  IB_CHECK_ARG(E > 0 && offsets && tiles, "gemm_grouped_relu2_tcgen05: the groups' tables are missing");
+  const int total_kt = (K + BK - 1) / BK;
+  CUtensorMap tw, tx;
+  if (make_tmap(&tw, w, E * N, K, BM)) return 1;
+  if (make_tmap(&tx, x, R, K, bn)) return 1;
+  Groups g;
+  g.offsets = offsets, g.tiles = tiles, g.n = E, g.w_rows = N;
+  switch (bn) {
+    case 16: return launch<16, 1, EPI_RELU2>(tw, tx, act, R, N, K, 1, total_kt, 0, status, stream, 0, g);
+    case 32: return launch<32, 1, EPI_RELU2>(tw, tx, act, R, N, K, 1, total_kt, 0, status, stream, 0, g);
+    case 64: return launch<64, 1, EPI_RELU2>(tw, tx, act, R, N, K, 1, total_kt, 0, status, stream, 0, g);
+    case 128: return launch<128, 1, EPI_RELU2>(tw, tx, act, R, N, K, 1, total_kt, 0, status, stream, 0, g);
+    case 256: return launch<256, 1, EPI_RELU2>(tw, tx, act, R, N, K, 1, total_kt, 0, status, stream, 0, g);
+    default: return ib_set_error("gemm_grouped_relu2_tcgen05: token tile %d is not one of 16, 32, 64, 128, 256", bn);
   }
 }
 

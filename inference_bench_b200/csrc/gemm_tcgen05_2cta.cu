@@ -28,6 +28,7 @@ constexpr int UMMA_K = 16;
 constexpr int kThreads = 192;
 constexpr int EPI_STORE = 0, EPI_SWIGLU = 1, EPI_ADD = 2;   // float32 out; bfloat16 silu(gate) * up; float32 out += product
 constexpr int EPI_QKV = 3;   // the q/k/v projection finished in the epilogue: per-head norm, rotation, queries out, keys and values into the cache
+constexpr int EPI_RELU2 = 5;   // bfloat16 max(product, 0)^2
 constexpr int EPI_XIELU = 4;   // bfloat16 xielu(product) with the activation's two numbers (QkvEpi::act_pq)
 constexpr int kQkvHead = 128;   // head size of the EPI_QKV form: a head is 128 accumulator columns
 constexpr uint32_t kPeerBitMask = 0xFEFFFFFFu;   // clears the bit that tells the two CTAs of a pair apart in a shared::cluster address
@@ -342,7 +343,7 @@ __global__ void __launch_bounds__(kThreads, 1)
             }
           }
         }
-      } else if constexpr (EPI == EPI_STORE || EPI == EPI_ADD || EPI == EPI_XIELU) {
+      } else if constexpr (EPI == EPI_STORE || EPI == EPI_ADD || EPI == EPI_XIELU || EPI == EPI_RELU2) {
         float* dst = (float*)out_;
         __nv_bfloat16* dst_act = (__nv_bfloat16*)out_;
         float ap = 0.f, an = 0.f;
@@ -369,6 +370,8 @@ __global__ void __launch_bounds__(kThreads, 1)
                 if (t < T) {
                   if constexpr (EPI == EPI_XIELU)
                     dst_act[(size_t)t * N + n] = __float2bfloat16_rn(ib::xielu(__uint_as_float(r[c]), ap, an));
+                  else if constexpr (EPI == EPI_RELU2)
+                    dst_act[(size_t)t * N + n] = __float2bfloat16_rn(ib::relu2(__uint_as_float(r[c])));
                   else
                     dst[(size_t)t * N + n] = __uint_as_float(r[c]);
                 }
@@ -479,6 +482,12 @@ extern "C" int ib_gemm_tcgen05_2cta(const void* x, const void* w, float* out, in
 extern "C" int ib_gemm_tcgen05_2cta_add(const void* x, const void* w, float* out, int T, int N, int K, unsigned* status, cudaStream_t stream) {
   if (T == 0 || N == 0) return 0;
   return launch<1, EPI_ADD, 256>(x, w, out, T, N, K, N, 0, status, stream);
+}
+
+// x [T, K], w [N, K] bfloat16 -> act [T, N] bfloat16 = max(x w^T, 0)^2, with the activation in the epilogue.
+extern "C" int ib_gemm_relu2_tcgen05_2cta(const void* x, const void* w, void* act, int T, int N, int K, unsigned* status, cudaStream_t stream) {
+  if (T == 0 || N == 0) return 0;
+  return launch<1, EPI_RELU2, 256>(x, w, act, T, N, K, N, 0, status, stream);
 }
 
 // x [T, K], w [N, K] bfloat16 -> act [T, N] bfloat16 = xielu(x w^T) with the two numbers pq (float32, on the device): the product of

@@ -5,7 +5,7 @@
 // `BlockPool` and the scheduler's block tables (crates/specrt/src/sched.rs:18-96, 1106-1130).
 //
 // A group with a window gives a page back as soon as every position in it has fallen out of the
-// window of the request's next token. All calls are meant for one thread.
+// window of the request's next token, unless it holds one of the first positions that the group keeps. All calls are meant for one thread.
 #include <cstdarg>
 #include <cstdio>
 #include <cstring>
@@ -73,6 +73,7 @@ struct Pool {
 struct Cache {
   int page_size, max_requests, max_tokens, table_width;
   std::vector<int> windows;            // per group, 0 = none
+  std::vector<int> keeps;              // per group: positions 0 .. keeps - 1 stay visible whatever the window (0 = none)
   std::vector<Pool> pools;             // per group
   std::vector<int> tables;             // [groups][max_requests][table_width], -1 = no page
   std::vector<int> length;             // per slot: positions whose state is in the cache
@@ -84,6 +85,9 @@ struct Cache {
     if (windows[g] <= 0) return 0;
     const int lo = len - windows[g] + 1;
     return lo > 0 ? lo / page_size : 0;
+  }
+  bool needs_page(int g, int len, int page) const {   // whether a token at position >= len can see a position of the page
+    return page >= first_live_page(g, len) || page * page_size < keeps[g];
   }
   int pages_for(int len) const { return (len + page_size - 1) / page_size; }
   bool is_live(int slot) const { return slot >= 0 && slot < max_requests && live[slot]; }
@@ -110,7 +114,8 @@ int ibh_pool_refcount(void* p, int page) {
 int ibh_pool_check(void* p) { return ((Pool*)p)->check(); }
 
 // ---------------------------------------------------------------- the cache: pools, tables, slots
-void* ibh_cache_new(int n_groups, const int* windows, int page_size, int num_pages, int max_requests, int max_tokens) {
+// windows[g]: 0 for every position, else how many positions back a token of group g sees; keeps[g]: how many of a request's first positions it sees beside them
+void* ibh_cache_new(int n_groups, const int* windows, const int* keeps, int page_size, int num_pages, int max_requests, int max_tokens) {
   if (n_groups < 0 || page_size <= 0 || num_pages <= 0 || max_requests <= 0 || max_tokens <= 0) {
     fail(1, "cache: sizes must be positive");
     return nullptr;
@@ -121,6 +126,7 @@ void* ibh_cache_new(int n_groups, const int* windows, int page_size, int num_pag
   c->max_tokens = max_tokens;
   c->table_width = (max_tokens + page_size - 1) / page_size;
   c->windows.assign(windows, windows + n_groups);
+  c->keeps.assign(keeps, keeps + n_groups);
   for (int g = 0; g < n_groups; g++) c->pools.emplace_back(num_pages);
   c->tables.assign((size_t)n_groups * max_requests * c->table_width, -1);
   c->length.assign(max_requests, 0);
@@ -158,13 +164,12 @@ void ibh_cache_pages_missing(void* cp, int slot, int new_length, int length, int
   const int cur = known ? c->length[slot] : length;
   const int last = c->pages_for(new_length);
   for (int g = 0; g < (int)c->pools.size(); g++) {
-    const int first = c->first_live_page(g, cur);
     int n = 0;
     if (!known) {
-      n = last > first ? last - first : 0;
+      for (int p = 0; p < last; p++) n += c->needs_page(g, cur, p);
     } else {
       const int* row = c->row(g, slot);
-      for (int p = first; p < last && p < c->table_width; p++) n += row[p] < 0;
+      for (int p = 0; p < last && p < c->table_width; p++) n += row[p] < 0 && c->needs_page(g, cur, p);
     }
     out[g] = n;
   }
@@ -180,8 +185,8 @@ int ibh_cache_extend(void* cp, int slot, int new_length) {
   const int last = c->pages_for(new_length);
   for (int g = 0; g < (int)c->pools.size(); g++) {
     int* row = c->row(g, slot);
-    for (int p = c->first_live_page(g, c->length[slot]); p < last; p++) {
-      if (row[p] >= 0) continue;
+    for (int p = 0; p < last; p++) {
+      if (row[p] >= 0 || !c->needs_page(g, c->length[slot], p)) continue;
       const int page = c->pools[g].allocate();
       if (page < 0) {
         for (auto& t : taken) {
@@ -225,7 +230,7 @@ int ibh_cache_commit(void* cp, int slot, int new_length) {
     const int first = c->first_live_page(g, new_length);
     int* row = c->row(g, slot);
     for (int p = 0; p < first && p < c->table_width; p++)
-      if (row[p] >= 0) {
+      if (row[p] >= 0 && !c->needs_page(g, new_length, p)) {
         c->pools[g].release(row[p]);
         row[p] = -1;
       }

@@ -1,10 +1,10 @@
-// Layer norm without a bias, fused with the residual add that precedes it, and the pieces of a block whose sublayers read
+// Layer norm, with or without a bias, fused with the residual add that precedes it, and the pieces of a block whose sublayers read
 // their input through a short causal convolution over time and whose layers are mixed by a depth-weighted average.
 // All arithmetic is float32; only a stored activation may be bfloat16.
 //
 //  * add_layernorm: v = x[t] + scale * (sum_p delta[p][t] + bias)   (scale, bias: per channel, optional; partial sums added in order)
 //                   x[t] = v (optional), x_copy[t] = v (optional)
-//                   out = w * (v - mean(v)) / sqrt(mean((v - mean)^2) + eps)
+//                   out = w * (v - mean(v)) / sqrt(mean((v - mean)^2) + eps) [+ b]
 //    With `halo` > 0 the output rows are laid out for the convolution that follows: segment s (tokens a..b of the flat batch) owns
 //    rows a + s * halo .. b + (s + 1) * halo; its first `halo` rows are the request's last `halo` normed rows of earlier steps, copied
 //    from its state slot by extra blocks of this kernel, so the convolution reads one array and its state update races with nothing.
@@ -13,7 +13,10 @@
 //  * add_layernorm_conv_single: both of the above in one kernel for a step in which every request brings one token (decoded tokens): a CTA
 //    per token norms its row, reads the request's `halo` state rows, writes the convolved row and shifts the state by one row.
 //  * depth_average: X = x[t] + scale * (sum_p delta[p][t] + bias); stack[k][t] = X; x[t] = sum_{j <= k} mix[j] * stack[j][t].
-//  * scale_values: v *= s (logits times a constant).
+//  * scale_values: v *= s (logits times a constant); softcap_values: v = cap tanh(v / cap).
+//  * embed_layernorm: the layer norm of a token's row of the embedding table.
+//  * shift_mixes: several mixes of every normed row with the row before it (a different weight per channel each), and
+//    add_layernorm_mixes_single: the residual add, the norm and the mixes in one kernel for steps of single tokens.
 #include <type_traits>
 
 #include "common.cuh"
@@ -22,16 +25,22 @@ namespace {
 
 constexpr int kLnThreads = 256;
 
+struct LnExtras {
+  const float* wb;   // the norm's bias per channel, or null
+  float mult;        // factor on the contribution where there is no per-channel scale
+  int early;         // 1: the kernels that follow may be scheduled while this one runs; 0: only when it is done (for the reason given in causal_conv_rows_kernel)
+};
+
 template <typename O>
 __global__ void __launch_bounds__(kLnThreads) add_layernorm_kernel(float* __restrict__ x, const float* __restrict__ delta, int P, size_t delta_stride,
                                                                    const float* __restrict__ dscale, const float* __restrict__ dbias,
                                                                    const float* __restrict__ w, O* __restrict__ out, const int* __restrict__ rows, int n_rows,
                                                                    int H, float eps, int write_x, float* __restrict__ x_copy, int halo,
                                                                    const int* __restrict__ seg_of_token, const int* __restrict__ seg_start,
-                                                                   const int* __restrict__ seg_slot, const float* __restrict__ state, size_t slot_stride) {
+                                                                   const int* __restrict__ seg_slot, const float* __restrict__ state, size_t slot_stride, LnExtras ex) {
   extern __shared__ __align__(16) float row[];
   __shared__ float scratch[32];
-  ib::pdl_launch_dependents();
+  if (ex.early) ib::pdl_launch_dependents();
   ib::pdl_wait();
   const int r = blockIdx.x;
   if (r >= n_rows) {   // a halo row: the request's state of earlier steps, as it is
@@ -53,7 +62,7 @@ __global__ void __launch_bounds__(kLnThreads) add_layernorm_kernel(float* __rest
         for (int p = 1; p < P; p++) a += delta[p * delta_stride + (size_t)t * H + i];
         d = dbias ? a + d : a;
       }
-      v = dscale ? __fmaf_rn(dscale[i], d, v) : v + d;
+      v = __fmaf_rn(dscale ? dscale[i] : ex.mult, d, v);
       if (write_x) xr[i] = v;
     }
     if (x_copy) x_copy[(size_t)t * H + i] = v;
@@ -69,7 +78,7 @@ __global__ void __launch_bounds__(kLnThreads) add_layernorm_kernel(float* __rest
   const float inv = rsqrtf(ib::block_sum(sq, scratch) / (float)H + eps);
   const size_t orow = halo ? (size_t)t + (size_t)(seg_of_token[t] + 1) * halo : (size_t)r;
   O* dst = out + orow * H;
-  for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = ib::from_f32<O>((row[i] - mean) * inv * w[i]);
+  for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = ib::from_f32<O>(__fmaf_rn((row[i] - mean) * inv, w[i], ex.wb ? ex.wb[i] : 0.f));
 }
 
 template <typename O>
@@ -146,10 +155,10 @@ __global__ void __launch_bounds__(kLnThreads) add_layernorm_vec_kernel(float* __
                                                                        const float* __restrict__ w, O* __restrict__ out, const int* __restrict__ rows, int n_rows,
                                                                        int H, float eps, int write_x, float* __restrict__ x_copy, int halo,
                                                                        const int* __restrict__ seg_of_token, const int* __restrict__ seg_start,
-                                                                       const int* __restrict__ seg_slot, const float* __restrict__ state, size_t slot_stride) {
+                                                                       const int* __restrict__ seg_slot, const float* __restrict__ state, size_t slot_stride, LnExtras ex) {
   extern __shared__ __align__(16) float row[];
   __shared__ float scratch[32];
-  ib::pdl_launch_dependents();
+  if (ex.early) ib::pdl_launch_dependents();
   ib::pdl_wait();
   const int r = blockIdx.x;
   if (r >= n_rows) {
@@ -171,7 +180,7 @@ __global__ void __launch_bounds__(kLnThreads) add_layernorm_vec_kernel(float* __
         for (int p = 1; p < P; p++) a = add4(a, ld4(delta + p * delta_stride + (size_t)t * H + i));
         d = dbias ? add4(a, d) : a;
       }
-      v = dscale ? fma4(ld4(dscale + i), d, v) : add4(v, d);
+      v = fma4(dscale ? ld4(dscale + i) : make_float4(ex.mult, ex.mult, ex.mult, ex.mult), d, v);
       if (write_x) st4(xr + i, v);
     }
     if (x_copy) st4(x_copy + (size_t)t * H + i, v);
@@ -189,8 +198,8 @@ __global__ void __launch_bounds__(kLnThreads) add_layernorm_vec_kernel(float* __
   const size_t orow = halo ? (size_t)t + (size_t)(seg_of_token[t] + 1) * halo : (size_t)r;
   O* dst = out + orow * H;
   for (int i = threadIdx.x * 4; i < H; i += blockDim.x * 4) {
-    const float4 v = ld4(row + i), g = ld4(w + i);
-    st4(dst + i, make_float4((v.x - mean) * inv * g.x, (v.y - mean) * inv * g.y, (v.z - mean) * inv * g.z, (v.w - mean) * inv * g.w));
+    const float4 v = ld4(row + i), g = ld4(w + i), b = ex.wb ? ld4(ex.wb + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    st4(dst + i, fma4(make_float4((v.x - mean) * inv, (v.y - mean) * inv, (v.z - mean) * inv, (v.w - mean) * inv), g, b));
   }
 }
 
@@ -343,6 +352,134 @@ __global__ void depth_average_vec_kernel(float* __restrict__ x, const float* __r
   }
 }
 
+// v = cap * tanh(v / cap)
+__global__ void softcap_values_kernel(float* __restrict__ v, size_t n, float cap) {
+  ib::pdl_launch_dependents();
+  ib::pdl_wait();
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) v[i] = cap * tanhf(v[i] / cap);
+}
+
+// x[t] = layer norm of the token's row of an embedding table, float32 (one CTA a token; sums as in add_layernorm_kernel).
+template <typename W>
+__global__ void __launch_bounds__(kLnThreads) embed_layernorm_kernel(const W* __restrict__ table, const int* __restrict__ tokens, const float* __restrict__ w,
+                                                                     const float* __restrict__ wb, float eps, float* __restrict__ x, int H, int V,
+                                                                     unsigned* __restrict__ status) {
+  extern __shared__ __align__(16) float row[];
+  __shared__ float scratch[32];
+  ib::pdl_launch_dependents();
+  ib::pdl_wait();
+  const int t = blockIdx.x;
+  int tok = tokens[t];
+  if (tok < 0 || tok >= V) {
+    if (threadIdx.x == 0) atomicOr(status, IB_ERR_BAD_TOKEN);
+    tok = 0;
+  }
+  const W* src = table + (size_t)tok * H;
+  float sum = 0.f;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float v = ib::to_f32<W>(src[i]);
+    row[i] = v;
+    sum += v;
+  }
+  const float mean = ib::block_sum(sum, scratch) / (float)H;
+  float sq = 0.f;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float c = row[i] - mean;
+    sq = __fmaf_rn(c, c, sq);
+  }
+  const float inv = rsqrtf(ib::block_sum(sq, scratch) / (float)H + eps);
+  for (int i = threadIdx.x; i < H; i += blockDim.x) x[(size_t)t * H + i] = __fmaf_rn((row[i] - mean) * inv, w[i], wb ? wb[i] : 0.f);
+}
+
+// out[m][t] = h_t + (h_(t-1) - h_t) * mu[m] per channel for M mixes. The row before a segment's first row is the request's state, which
+// becomes the segment's last row: the CTA that reads a request's old state (the first row's) is the one that writes the new one.
+template <typename O>
+__global__ void __launch_bounds__(kLnThreads) shift_mixes_kernel(const float* __restrict__ h, const float* __restrict__ mu, int M, float* __restrict__ state, size_t slot_stride,
+                                                                 const int* __restrict__ seg_of_token, const int* __restrict__ seg_start,
+                                                                 const int* __restrict__ seg_slot, O* __restrict__ out, int T, int H) {
+  ib::pdl_launch_dependents();
+  ib::pdl_wait();
+  const int t = blockIdx.x;
+  const int s = seg_of_token[t], t0 = seg_start[s];
+  const bool first = t == t0;
+  float* st = state + (size_t)seg_slot[s] * slot_stride;
+  const float* prev = first ? st : h + (size_t)(t - 1) * H;
+  const float* last = h + (size_t)(seg_start[s + 1] - 1) * H;
+  const float* cur = h + (size_t)t * H;
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < H; i += gridDim.y * blockDim.x) {
+    const float v = cur[i], d = prev[i] - v;
+    for (int m = 0; m < M; m++) out[((size_t)m * T + t) * H + i] = ib::from_f32<O>(__fmaf_rn(d, mu[(size_t)m * H + i], v));
+    if (first) st[i] = last[i];
+  }
+}
+
+// The residual add, the layer norm and the mixes in one kernel for a step whose row t is segment t (one token each); sums in the order of
+// add_layernorm's kernels, so a decoded token's normed row has the same bits whichever kernel made it.
+template <typename O, bool VEC>
+__global__ void __launch_bounds__(kLnThreads) add_layernorm_mixes_single_kernel(float* __restrict__ x, const float* __restrict__ delta, int P, size_t delta_stride,
+                                                                                const float* __restrict__ w, float eps, const float* __restrict__ mu, int M,
+                                                                                O* __restrict__ out, int T, int H, const int* __restrict__ seg_slot,
+                                                                                float* __restrict__ state, size_t slot_stride, LnExtras ex) {
+  extern __shared__ __align__(16) float row[];
+  __shared__ float scratch[32];
+  if (ex.early) ib::pdl_launch_dependents();
+  ib::pdl_wait();
+  const int t = blockIdx.x;
+  float* xr = x + (size_t)t * H;
+  float* st = state + (size_t)seg_slot[t] * slot_stride;
+  constexpr int N = VEC ? 4 : 1;
+  float sum = 0.f;
+  for (int i = threadIdx.x * N; i < H; i += blockDim.x * N) {
+    if constexpr (VEC) {
+      float4 v = ld4(xr + i);
+      if (P > 0) {
+        float4 a = ld4(delta + (size_t)t * H + i);
+        for (int p = 1; p < P; p++) a = add4(a, ld4(delta + p * delta_stride + (size_t)t * H + i));
+        v = fma4(make_float4(ex.mult, ex.mult, ex.mult, ex.mult), a, v);
+        st4(xr + i, v);
+      }
+      st4(row + i, v);
+      sum += (v.x + v.y) + (v.z + v.w);
+    } else {
+      float v = xr[i];
+      if (P > 0) {
+        float a = delta[(size_t)t * H + i];
+        for (int p = 1; p < P; p++) a += delta[p * delta_stride + (size_t)t * H + i];
+        v = __fmaf_rn(ex.mult, a, v);
+        xr[i] = v;
+      }
+      row[i] = v;
+      sum += v;
+    }
+  }
+  const float mean = ib::block_sum(sum, scratch) / (float)H;
+  float sq = 0.f;
+  for (int i = threadIdx.x * N; i < H; i += blockDim.x * N) {
+    if constexpr (VEC) {
+      const float4 v = ld4(row + i);
+      const float a = v.x - mean, b = v.y - mean, c = v.z - mean, e = v.w - mean;
+      sq = __fmaf_rn(e, e, __fmaf_rn(c, c, __fmaf_rn(b, b, __fmaf_rn(a, a, sq))));
+    } else {
+      const float c = row[i] - mean;
+      sq = __fmaf_rn(c, c, sq);
+    }
+  }
+  const float inv = rsqrtf(ib::block_sum(sq, scratch) / (float)H + eps);
+  for (int i = threadIdx.x * N; i < H; i += blockDim.x * N) {
+    if constexpr (VEC) {
+      const float4 v = ld4(row + i), b = ex.wb ? ld4(ex.wb + i) : make_float4(0.f, 0.f, 0.f, 0.f), old = ld4(st + i);
+      const float4 h = fma4(make_float4((v.x - mean) * inv, (v.y - mean) * inv, (v.z - mean) * inv, (v.w - mean) * inv), ld4(w + i), b);
+      const float4 d = make_float4(old.x - h.x, old.y - h.y, old.z - h.z, old.w - h.w);
+      st4(st + i, h);
+      for (int m = 0; m < M; m++) st4(out + ((size_t)m * T + t) * H + i, fma4(d, ld4(mu + (size_t)m * H + i), h));
+    } else {
+      const float h = __fmaf_rn((row[i] - mean) * inv, w[i], ex.wb ? ex.wb[i] : 0.f), d = st[i] - h;
+      st[i] = h;
+      for (int m = 0; m < M; m++) out[((size_t)m * T + t) * H + i] = ib::from_f32<O>(__fmaf_rn(d, mu[(size_t)m * H + i], h));
+    }
+  }
+}
+
 __global__ void scale_values_kernel(float* __restrict__ v, size_t n, float s) {
   ib::pdl_launch_dependents();
   ib::pdl_wait();
@@ -353,8 +490,11 @@ __global__ void scale_values_kernel(float* __restrict__ v, size_t n, float s) {
 
 extern "C" int ib_add_layernorm(float* x, const float* delta, int P, long long delta_stride, const float* dscale, const float* dbias, const float* w, void* out,
                                 int out_dtype, const int* rows, int n_rows, int H, float eps, int write_x, float* x_copy, int halo, const int* seg_of_token,
-                                const int* seg_start, const int* seg_slot, int n_segments, const float* state, long long slot_stride, cudaStream_t stream) {
+                                const int* seg_start, const int* seg_slot, int n_segments, const float* state, long long slot_stride, const float* wb,
+                                float mult, int early, cudaStream_t stream) {
+  // wb: the norm's bias per channel, or null; mult: factor on the contribution where dscale is null; early: see LnExtras
   if (n_rows == 0) return 0;
+  const LnExtras ex = {wb, mult, early};
   IB_CHECK_ARG(n_rows > 0 && H > 0 && P >= 0 && halo >= 0, "add_layernorm: bad sizes rows=%d H=%d P=%d halo=%d", n_rows, H, P, halo);
   IB_CHECK_ARG(!(halo && rows), "add_layernorm: gathered rows have no layout for a convolution");
   IB_CHECK_ARG(!halo || (seg_of_token && seg_start && seg_slot && state && n_segments > 0), "add_layernorm: the convolution's layout needs the step's segments and the state");
@@ -364,10 +504,10 @@ extern "C" int ib_add_layernorm(float* x, const float* delta, int P, long long d
   auto go = [&](auto kernel, auto* o) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     ib::launch(kernel, grid, kLnThreads, smem, stream, x, delta, P, (size_t)delta_stride, dscale, dbias, w, o, rows, n_rows, H, eps, write_x, x_copy, halo, seg_of_token,
-               seg_start, seg_slot, state, (size_t)slot_stride);
+               seg_start, seg_slot, state, (size_t)slot_stride, ex);
   };
   auto al = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
-  const bool vec = H % 4 == 0 && al(x) && al(delta) && delta_stride % 4 == 0 && al(dscale) && al(dbias) && al(w) && al(out) && al(x_copy) && al(state) && slot_stride % 4 == 0;
+  const bool vec = H % 4 == 0 && al(wb) && al(x) && al(delta) && delta_stride % 4 == 0 && al(dscale) && al(dbias) && al(w) && al(out) && al(x_copy) && al(state) && slot_stride % 4 == 0;
   if (out_dtype != IB_F32 && out_dtype != IB_BF16) return ib_set_error("add_layernorm: unknown output dtype %d", out_dtype);
   if (vec && out_dtype == IB_F32) go(add_layernorm_vec_kernel<float>, (float*)out);
   else if (vec) go(add_layernorm_vec_kernel<__nv_bfloat16>, (__nv_bfloat16*)out);
@@ -438,5 +578,65 @@ extern "C" int ib_scale_values(float* v, long long n, float s, cudaStream_t stre
   if (n <= 0) return 0;
   ib::launch(scale_values_kernel, (unsigned)min((long long)1024, (n + 255) / 256), 256, 0, stream, v, (size_t)n, s);
   IB_CHECK_LAUNCH("scale_values");
+  return 0;
+}
+
+extern "C" int ib_softcap_values(float* v, long long n, float cap, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  IB_CHECK_ARG(cap > 0.f, "softcap_values: the cap %g must be positive", (double)cap);
+  ib::launch(softcap_values_kernel, (unsigned)min((long long)1024, (n + 255) / 256), 256, 0, stream, v, (size_t)n, cap);
+  IB_CHECK_LAUNCH("softcap_values");
+  return 0;
+}
+
+extern "C" int ib_embed_layernorm(const void* table, int dtype, const int* tokens, const float* w, const float* wb, float eps, float* x, int T, int H, int V, unsigned* status,
+                                  cudaStream_t stream) {
+  if (T == 0) return 0;
+  const size_t smem = (size_t)H * sizeof(float);
+  IB_CHECK_ARG(T > 0 && H > 0 && V > 0 && smem <= 200 * 1024, "embed_layernorm: bad sizes T=%d H=%d V=%d", T, H, V);
+  auto go = [&](auto kernel, auto* tab) {
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    ib::launch(kernel, (unsigned)T, kLnThreads, smem, stream, tab, tokens, w, wb, eps, x, H, V, status);
+  };
+  if (dtype == IB_F32) go(embed_layernorm_kernel<float>, (const float*)table);
+  else if (dtype == IB_BF16) go(embed_layernorm_kernel<__nv_bfloat16>, (const __nv_bfloat16*)table);
+  else return ib_set_error("embed_layernorm: unknown table dtype %d", dtype);
+  IB_CHECK_LAUNCH("embed_layernorm");
+  return 0;
+}
+
+// mu float32 [M][H], out [M][T][H].
+extern "C" int ib_shift_mixes(const float* h, const float* mu, int M, float* state, long long slot_stride, const int* seg_of_token, const int* seg_start,
+                              const int* seg_slot, void* out, int out_dtype, int T, int H, cudaStream_t stream) {
+  if (T == 0) return 0;
+  IB_CHECK_ARG(T > 0 && H > 0 && M > 0, "shift_mixes: bad sizes T=%d H=%d mixes=%d", T, H, M);
+  const dim3 grid((unsigned)T, (unsigned)min((H + kLnThreads - 1) / kLnThreads, 64));
+  if (out_dtype == IB_F32) ib::launch(shift_mixes_kernel<float>, grid, kLnThreads, 0, stream, h, mu, M, state, (size_t)slot_stride, seg_of_token, seg_start, seg_slot, (float*)out, T, H);
+  else if (out_dtype == IB_BF16)
+    ib::launch(shift_mixes_kernel<__nv_bfloat16>, grid, kLnThreads, 0, stream, h, mu, M, state, (size_t)slot_stride, seg_of_token, seg_start, seg_slot, (__nv_bfloat16*)out, T, H);
+  else return ib_set_error("shift_mixes: unknown output dtype %d", out_dtype);
+  IB_CHECK_LAUNCH("shift_mixes");
+  return 0;
+}
+
+extern "C" int ib_add_layernorm_mixes_single(float* x, const float* delta, int P, long long delta_stride, float mult, const float* w, const float* wb, float eps,
+                                             const float* mu, int M, void* out, int out_dtype, int T, int H, const int* seg_slot, float* state, long long slot_stride,
+                                             int early, cudaStream_t stream) {
+  if (T == 0) return 0;
+  const size_t smem = (size_t)H * sizeof(float);
+  IB_CHECK_ARG(T > 0 && H > 0 && P >= 0 && M > 0 && smem <= 200 * 1024, "add_layernorm_mixes_single: bad sizes T=%d H=%d P=%d mixes=%d", T, H, P, M);
+  const LnExtras ex = {wb, mult, early};
+  auto go = [&](auto kernel, auto* o) {
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    ib::launch(kernel, (unsigned)T, kLnThreads, smem, stream, x, delta, P, (size_t)delta_stride, w, eps, mu, M, o, T, H, seg_slot, state, (size_t)slot_stride, ex);
+  };
+  auto al = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  const bool vec = H % 4 == 0 && al(x) && al(delta) && delta_stride % 4 == 0 && al(w) && al(wb) && al(mu) && al(out) && al(state) && slot_stride % 4 == 0;
+  if (out_dtype != IB_F32 && out_dtype != IB_BF16) return ib_set_error("add_layernorm_mixes_single: unknown output dtype %d", out_dtype);
+  if (vec && out_dtype == IB_F32) go(add_layernorm_mixes_single_kernel<float, true>, (float*)out);
+  else if (vec) go(add_layernorm_mixes_single_kernel<__nv_bfloat16, true>, (__nv_bfloat16*)out);
+  else if (out_dtype == IB_F32) go(add_layernorm_mixes_single_kernel<float, false>, (float*)out);
+  else go(add_layernorm_mixes_single_kernel<__nv_bfloat16, false>, (__nv_bfloat16*)out);
+  IB_CHECK_LAUNCH("add_layernorm_mixes_single");
   return 0;
 }

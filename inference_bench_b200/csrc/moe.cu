@@ -6,12 +6,13 @@
 //    groups of neighbours, a group's score is its largest s (or the sum of its few largest), only the `keep` best groups stay eligible; the `top`
 //    eligible experts with the largest s are chosen (ties: the lower index), each weighted s * route_scale, or
 //    s / (sum of the chosen s) * route_scale with `renorm`. With a correction, groups and experts are chosen by s + correction[e]
-//    and weighted by s alone.
+//    and weighted by s alone. With `score` = 2 the experts are chosen by their logits (plus a bias each) and weighted by the softmax over
+//    the chosen logits alone.
 //  * moe_sort: counts the (token, choice) pairs of every expert, lays the experts' rows out one after the other
 //    (offsets[e] .. offsets[e + 1]) and gives every pair a row of its expert's range; tile_start[e] is the first tile of expert e.
 //  * gemm_grouped: out[r] = W[e(r)] x[src(r)] for every regrouped row r: a 64 x 64 tile belongs to one expert; float32
 //    FMA chains per output (a row's result does not depend on its place among the rows). With `gated`, W holds gate
-//    rows then up rows and the output is silu(gate) * up.
+//    rows then up rows and the output is silu(gate) * up. With `relu2` the output is the square of max(product, 0).
 //  * moe_combine: out[t] = sum_p base[p][t] + sum_k weight[t][k] * y[row(t, k)], in the order of the choices (without weights: the plain sum).
 //  * scatter_scaled_rows: out[row(t, k)] = weight[t][k] * x[t]: the step's rows in the experts' order with the router's weight on the
 //    expert's input (an expert is not linear, so a weight on its input is not one on its output).
@@ -35,7 +36,8 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 
 __global__ void moe_route_kernel(const float* __restrict__ logits, int P, size_t stride_p, int T, int E, int n_groups, int keep, int top, float route_scale,
                                  int renorm, int* __restrict__ idx_out, float* __restrict__ wt_out, int score, const float* __restrict__ correction,
-                                 int group_top) {
+                                 int group_top, int row, const float* __restrict__ logit_bias) {
+  // row: entries of a row of logits (the experts' are its first E). logit_bias: float32 [E] added to the logits, or null.
   // correction: a number per expert added to its score for the choice (of groups and of experts) and left out of the weights, or null.
   // group_top: a group's score is the sum of its `group_top` largest choice scores (1: its largest).
   // Choice scores may be negative: what cannot be chosen counts as minus infinity.
@@ -50,14 +52,15 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int P, size_t
   float* g = c + E;
   float mx = -INFINITY;
   for (int e = lane; e < E; e += 32) {
-    float z = logits[(size_t)t * E + e];
-    for (int p = 1; p < P; p++) z += logits[p * stride_p + (size_t)t * E + e];
+    float z = logits[(size_t)t * row + e];
+    for (int p = 1; p < P; p++) z += logits[p * stride_p + (size_t)t * row + e];
+    if (logit_bias) z += logit_bias[e];
     s[e] = z;
     mx = fmaxf(mx, z);
   }
   if (score == 1) {   // every expert's own sigmoid
     for (int e = lane; e < E; e += 32) s[e] = 1.f / (1.f + expf(-s[e]));
-  } else {
+  } else if (score == 0) {
     mx = ib::warp_max(mx);
     float sum = 0.f;
     for (int e = lane; e < E; e += 32) {
@@ -103,7 +106,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int P, size_t
       if (g[e / per] == g[e / per]) c[e] = -INFINITY;   // its group was not kept
     __syncwarp();
   }
-  float chosen_sum = 0.f;
+  float chosen_sum = 0.f, chosen_max = 0.f;
   for (int r = 0; r < top; r++) {
     float bv = -INFINITY;
     int bi = 0x7fffffff;
@@ -111,8 +114,14 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int P, size_t
       if (c[e] > bv) bv = c[e], bi = e;
     warp_argmax(bv, bi);
     float w = 0.f;
-    if (bi >= E) bi = 0;   // fewer experts that can be chosen than choices: weight zero
-    else w = s[bi];
+    if (bi >= E) {   // fewer experts that can be chosen than choices: weight zero
+      bi = 0;
+    } else if (score == 2) {   // the softmax over the chosen logits: the first choice has the largest
+      if (r == 0) chosen_max = s[bi];
+      w = expf(s[bi] - chosen_max);
+    } else {
+      w = s[bi];
+    }
     if (lane == 0) {
       idx_out[(size_t)t * top + r] = bi;
       wt_out[(size_t)t * top + r] = w;
@@ -172,7 +181,9 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ 
 template <typename X, typename W, typename O>
 __global__ void __launch_bounds__(256) gemm_grouped_kernel(const X* __restrict__ x, const int* __restrict__ src_row, const W* __restrict__ w,
                                                            O* __restrict__ out, const int* __restrict__ offsets, const int* __restrict__ tile_start, int E,
-                                                           int N, int K, int gated) {
+                                                           int N, int K, int act) {
+  // act: 0 the product, 1 silu(gate) * up (w holds gate rows, then up rows), 2 the square of max(product, 0)
+  const bool gated = act == 1;
   constexpr int BK = 16;
   __shared__ float xs[BK][SM_ + 1];
   __shared__ float ws[BK][64 + 1];
@@ -258,6 +269,8 @@ __global__ void __launch_bounds__(256) gemm_grouped_kernel(const X* __restrict__
       float v = acc[i][j];
       if (gated) {
         v = (v / (1.f + expf(-v))) * acu[i][j];
+      } else if (act == 2) {
+        v = ib::relu2(v);
       }
       out[(size_t)row * N + n] = ib::from_f32<O>(v);
     }
@@ -274,13 +287,23 @@ __global__ void gather_rows_kernel(const uint4* __restrict__ x, const int* __res
 }
 
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ row_of_pair, const float* __restrict__ wt, int top,
-                                   const float* __restrict__ base, int P, size_t stride_p, float* __restrict__ out, int H) {
+                                   const float* __restrict__ base, int P, size_t stride_p, float* __restrict__ out, int H, const float* __restrict__ gate,
+                                   int gate_P, size_t gate_stride, int gate_row) {
+  // gate: float32 partial sums [gate_P][T][gate_row] offset to one column, or null: `base` counts times the sigmoid of the token's entry there
   ib::pdl_launch_dependents();
   ib::pdl_wait();
   const int t = blockIdx.y;
+  float f = 1.f;
+  if (gate) {
+    const float* gr = gate + (size_t)t * gate_row;
+    float z = gr[0];
+    for (int p = 1; p < gate_P; p++) z += gr[p * gate_stride];
+    f = 1.f / (1.f + expf(-z));
+  }
   for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < H; i += gridDim.x * blockDim.x) {
     float a = 0.f;
     for (int p = 0; p < P; p++) a += base[p * stride_p + (size_t)t * H + i];
+    if (gate) a *= f;
     if (wt) {
       for (int k = 0; k < top; k++) a = fmaf(wt[(size_t)t * top + k], y[(size_t)row_of_pair[(size_t)t * top + k] * H + i], a);
     } else {
@@ -306,17 +329,20 @@ __global__ void scatter_scaled_rows_kernel(const X* __restrict__ x, const int* _
 }  // namespace
 
 extern "C" int ib_moe_route(const float* logits, int P, long long stride_p, int T, int E, int n_groups, int keep, int top, float route_scale, int renorm,
-                            int* idx_out, float* wt_out, int score, const float* correction, int group_top, cudaStream_t stream) {
+                            int* idx_out, float* wt_out, int score, const float* correction, int group_top, int row, const float* logit_bias, cudaStream_t stream) {
+  // row: entries of a row of logits (0: E). logit_bias: see the kernel.
+  if (row <= 0) row = E;
   // correction: float32 [E] added to the scores for the choice only, or null; group_top: how many of a group's largest choice scores make its score (1 to 4).
   if (T == 0) return 0;
   IB_CHECK_ARG(group_top >= 1 && group_top <= 4, "moe_route: a group's score is the sum of its %d largest scores (1 to 4)", group_top);
   IB_CHECK_ARG(P >= 1 && E > 0 && top > 0 && top <= E, "moe_route: bad sizes P=%d experts=%d top=%d", P, E, top);
-  IB_CHECK_ARG(score == 0 || score == 1, "moe_route: score %d is neither 0 (softmax) nor 1 (sigmoid)", score);
+  IB_CHECK_ARG(score >= 0 && score <= 2, "moe_route: score %d is not known (0: softmax, 1: sigmoid, 2: softmax over the chosen logits)", score);
+  IB_CHECK_ARG(row >= E, "moe_route: rows of %d logits do not hold %d experts", row, E);
   IB_CHECK_ARG(n_groups >= 1 && E % n_groups == 0 && keep >= 1 && keep <= n_groups, "moe_route: %d experts in %d groups of which %d stay", E, n_groups, keep);
   const size_t smem = (size_t)kRouteWarps * (2 * E + n_groups) * sizeof(float);
   IB_CHECK_ARG(smem <= 48 * 1024, "moe_route: %d experts need %zu bytes of shared memory, more than 48 KiB", E, smem);
   ib::launch(moe_route_kernel, (unsigned)((T + kRouteWarps - 1) / kRouteWarps), kRouteWarps * 32, smem, stream, logits, P, (size_t)stride_p, T, E, n_groups, keep,
-             top, route_scale, renorm, idx_out, wt_out, score, correction, group_top);
+             top, route_scale, renorm || score == 2, idx_out, wt_out, score, correction, group_top, row, logit_bias);
   IB_CHECK_LAUNCH("moe_route");
   return 0;
 }
@@ -337,12 +363,13 @@ extern "C" int ib_moe_sort(const int* idx, int R, int top, int E, int tile_rows,
 }
 
 extern "C" int ib_gemm_grouped(const void* x, int x_dtype, const int* src_row, const void* w, int w_dtype, void* out, int out_dtype, const int* offsets,
-                               const int* tile_start, int R, int E, int N, int K, int gated, cudaStream_t stream) {
+                               const int* tile_start, int R, int E, int N, int K, int act, cudaStream_t stream) {
   if (R == 0 || N == 0) return 0;
+  IB_CHECK_ARG(act >= 0 && act <= 2, "gemm_grouped: activation %d is not known (0: none, 1: gated SiLU, 2: squared ReLU)", act);
   IB_CHECK_ARG(R > 0 && E > 0 && N > 0 && K > 0, "gemm_grouped: bad sizes rows=%d experts=%d N=%d K=%d", R, E, N, K);
   dim3 grid((N + 63) / 64, R / SM_ + E);   // no more tiles than this, whatever the counts
   IB_CHECK_ARG(grid.y <= 65535, "gemm_grouped: %d rows exceed the grid limit", R);
-  auto go = [&](auto kernel, auto* xp, auto* wp, auto* op) { ib::launch(kernel, grid, 256, 0, stream, xp, src_row, wp, op, offsets, tile_start, E, N, K, gated); };
+  auto go = [&](auto kernel, auto* xp, auto* wp, auto* op) { ib::launch(kernel, grid, 256, 0, stream, xp, src_row, wp, op, offsets, tile_start, E, N, K, act); };
   using bf = __nv_bfloat16;
   if (x_dtype == IB_F32 && w_dtype == IB_F32 && out_dtype == IB_F32) go(gemm_grouped_kernel<float, float, float>, (const float*)x, (const float*)w, (float*)out);
   else if (x_dtype == IB_BF16 && w_dtype == IB_BF16 && out_dtype == IB_F32) go(gemm_grouped_kernel<bf, bf, float>, (const bf*)x, (const bf*)w, (float*)out);
@@ -353,12 +380,13 @@ extern "C" int ib_gemm_grouped(const void* x, int x_dtype, const int* src_row, c
 }
 
 extern "C" int ib_moe_combine(const float* y, const int* row_of_pair, const float* wt, int top, const float* base, int P, long long stride_p, float* out, int T,
-                              int H, cudaStream_t stream) {
+                              int H, const float* gate, int gate_P, long long gate_stride, int gate_row, cudaStream_t stream) {
   if (T == 0) return 0;
+  IB_CHECK_ARG(!gate || (gate_P >= 1 && gate_row >= 1), "moe_combine: a gate of %d parts and rows of %d", gate_P, gate_row);
   IB_CHECK_ARG(T > 0 && H > 0 && top > 0 && P >= 0, "moe_combine: bad sizes T=%d H=%d top=%d P=%d", T, H, top, P);
   IB_CHECK_ARG(T <= 65535, "moe_combine: T=%d rows exceed the grid limit 65535", T);
   dim3 grid(min((H + 255) / 256, 64), T);
-  ib::launch(moe_combine_kernel, grid, 256, 0, stream, y, row_of_pair, wt, top, base, P, (size_t)stride_p, out, H);
+  ib::launch(moe_combine_kernel, grid, 256, 0, stream, y, row_of_pair, wt, top, base, P, (size_t)stride_p, out, H, gate, gate_P, (size_t)gate_stride, gate_row);
   IB_CHECK_LAUNCH("moe_combine");
   return 0;
 }

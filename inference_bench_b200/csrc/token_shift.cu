@@ -10,6 +10,7 @@
 //  * loop_pack: before a pass over looped layers: packed_t = [x_t + pending | x0_t] in the activation dtype (the input of the matrix
 //    that makes the pass's stream) and x_t = step vector, to which the next norm adds the product.
 //  * xielu_rows: act = z > 0 ? ap z^2 + z / 2 : an (exp(z) - 1 - z) + z / 2 with ap = softplus(p), an = 1/2 + softplus(q).
+//  * relu2_rows: act = max(z, 0)^2.
 //  * gated_rmsnorm: out = scale * w * o / sqrt(mean(o^2) + eps) * sigmoid(gate) over a whole row of all heads.
 #include "common.cuh"
 
@@ -118,6 +119,19 @@ __global__ void xielu_rows_kernel(const float* __restrict__ z, int P, size_t str
 }
 
 template <typename O>
+__global__ void relu2_rows_kernel(const float* __restrict__ z, int P, size_t stride, O* __restrict__ act, int I) {
+  ib::pdl_launch_dependents();
+  ib::pdl_wait();
+  const int t = blockIdx.y;
+  const float* row = z + (size_t)t * I;
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < I; i += gridDim.x * blockDim.x) {
+    float v = row[i];
+    for (int p = 1; p < P; p++) v += row[p * stride + i];
+    act[(size_t)t * I + i] = ib::from_f32<O>(ib::relu2(v));
+  }
+}
+
+template <typename O>
 __global__ void gated_rmsnorm_kernel(const float* __restrict__ o, const float* __restrict__ w, float eps, const float* __restrict__ gate, int P, size_t gate_stride,
                                      int gate_row, float scale, O* __restrict__ out, int out_row, int H) {
   // o: [T][H]; gate: partial sums [P][T][gate_row], already offset to the gate's first column; out: rows of out_row values, offset to the first column
@@ -208,6 +222,17 @@ extern "C" int ib_xielu_rows(const float* z, int P, long long stride, const floa
   else if (act_dtype == IB_BF16) ib::launch(xielu_rows_kernel<__nv_bfloat16>, grid, 256, 0, stream, z, P, (size_t)stride, pq, (__nv_bfloat16*)act, I);
   else return ib_set_error("xielu_rows: unknown output dtype %d", act_dtype);
   IB_CHECK_LAUNCH("xielu_rows");
+  return 0;
+}
+
+extern "C" int ib_relu2_rows(const float* z, int P, long long stride, void* act, int act_dtype, int T, int I, cudaStream_t stream) {
+  if (T == 0) return 0;
+  IB_CHECK_ARG(T > 0 && I > 0 && P >= 1 && T <= 65535, "relu2_rows: bad sizes T=%d I=%d P=%d", T, I, P);
+  dim3 grid((unsigned)min((I + 255) / 256, 64), (unsigned)T);
+  if (act_dtype == IB_F32) ib::launch(relu2_rows_kernel<float>, grid, 256, 0, stream, z, P, (size_t)stride, (float*)act, I);
+  else if (act_dtype == IB_BF16) ib::launch(relu2_rows_kernel<__nv_bfloat16>, grid, 256, 0, stream, z, P, (size_t)stride, (__nv_bfloat16*)act, I);
+  else return ib_set_error("relu2_rows: unknown output dtype %d", act_dtype);
+  IB_CHECK_LAUNCH("relu2_rows");
   return 0;
 }
 

@@ -119,20 +119,26 @@ class Runtime:
         ops.silu_mul(gu, act)
         return act
 
-    def up_xielu(self, x: torch.Tensor, lw: LinearWeights, pq: torch.Tensor) -> torch.Tensor:
-        """x [T, K] -> xielu(x W^T) in the activation dtype, [T, N], with the activation's two numbers pq (float32 [2]). bfloat16 products
+    def up_act(self, x: torch.Tensor, lw: LinearWeights, kind: str, pq: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """x [T, K] -> activation of x W^T in the activation dtype, [T, N]: kind "xielu" with its two numbers pq (float32 [2]), or "relu2"
+        (the square of max(z, 0)). bfloat16 products
         that need not cut their k-range apply the activation in the tensor-core kernel's epilogue, on the float32 accumulators;
         otherwise the product and the row-wise kernel that adds the partial sums."""
         T = x.shape[0]
         if self.mode == "bfloat16" and self.gemm != "simt" and self.options.swiglu_epilogue:
             from ..kernels import gemm_tcgen05
-            if gemm_tcgen05.xielu_in_epilogue(T, lw.n, lw.k, self.sm_count):
+            if gemm_tcgen05.act_in_epilogue(T, lw.n, lw.k, self.sm_count):
                 act = self.empty((T, lw.n))
-                gemm_tcgen05.gemm_xielu(self, x, lw, pq, act)
+                gemm_tcgen05.gemm_act(self, x, lw, kind, act, pq)
                 return act
         z = self.linear(x, lw)
         act = self.empty((T, lw.n))
-        ops.xielu_rows(z, pq, act)
+        if kind == "xielu":
+            ops.xielu_rows(z, pq, act)
+        elif kind == "relu2":
+            ops.relu2_rows(z, act)
+        else:
+            raise L.KernelError(f"activation {kind!r} is not known (xielu, relu2)")
         return act
 
     # ---------------------------------------------------------------- status word

@@ -56,13 +56,13 @@ L.register("ib_attention_decode_fused", [L._p, L._i, L._ll, L._p, L._p, L._f, L.
 L.register("ib_attention_prefill_tc", [L._p, C.POINTER(L.KvView), L._p, L._p, L._i, L._p, L._p, L._i, L._f, L._p, L._i, L._p, L._p])
 L.register("ib_attention_prefill_ws", [L._p, C.POINTER(L.KvView), L._p, L._p, L._i, L._p, L._p, L._i, L._f, L._p, L._i, L._p, L._ll, L._p, L._p])
 # the same with capped scores and a sink (softcap, sink before the status word)
-# (softcap, sink, the output's tail or null, then the status word)
+# (softcap, sink, the output's tail or null, the kept first positions, then the status word)
 L.register("ib_attention_decode_capped", [L._p, C.POINTER(L.KvView), L._p, L._i, L._p, L._p, L._i, L._f, L._p, L._p, L._p, L._i, L._i, L._i, L._f, L._i, C.POINTER(L.AttnTail),
-                                          L._p, L._p])
+                                          L._i, L._p, L._p])
 L.register("ib_attention_decode_stream_capped", [L._p, C.POINTER(L.KvView), L._p, L._i, L._p, L._p, L._i, L._f, L._p, L._p, L._p, L._i, L._i, L._i, L._p, L._ll, L._f, L._i,
-                                                 C.POINTER(L.AttnTail), L._p, L._p])
+                                                 C.POINTER(L.AttnTail), L._i, L._p, L._p])
 L.register("ib_attention_prefill_ws_capped", [L._p, C.POINTER(L.KvView), L._p, L._p, L._i, L._p, L._p, L._i, L._f, L._p, L._i, L._p, L._ll, L._f, L._i, C.POINTER(L.AttnTail),
-                                              L._p, L._p])
+                                              L._i, L._p, L._p])
 L.KERNELS_PER_CALL["ib_attention_decode_capped"] = 2
 L.KERNELS_PER_CALL["ib_attention_decode_stream_capped"] = 2
 
@@ -172,16 +172,17 @@ def decode_fused(ctx, qkv: torch.Tensor, q_norm_w, k_norm_w, eps: float, cos, si
 
 def paged_attention(ctx, q: torch.Tensor, cache: ops.KvLayerView, heads: int, window: Optional[int], scale: float, qk_dim: Optional[int] = None,
                     v_dim: Optional[int] = None, softcap: float = 0.0, sink: bool = False, chunk: int = 0, sink_values: Optional[torch.Tensor] = None,
-                    gate: Optional[tuple] = None, out_scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    gate: Optional[tuple] = None, out_scale: float = 1.0, out: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
     """q [T, heads * qk_dim] (activation dtype) -> attention output [T, heads * v_dim] of the same dtype. qk_dim, v_dim: the head sizes
     (default: the cache's row); softcap > 0 caps the scores with a tanh; sink adds one to the softmax's denominator, or with sink_values
     (float32 [heads]) exp of the head's value. chunk > 0: instead of a window, a position sees the earlier positions of its own block of
     `chunk` positions, blocks counted from position 0. gate = (float32 partial sums [P, T, row], the first head's column): head h's
     output is multiplied by the sigmoid of its column; out_scale multiplies the output. out: a buffer [T, >= heads * v_dim] whose first
-    columns are written, instead of a new one."""
+    columns are written, instead of a new one. keep_first (with a window): the request's first positions, which are seen whatever the window."""
     rt = ctx.rt
     view = cache.c_view()
     T = q.shape[0]
+    keep_first = int(keep_first) if window else 0
     qk_dim, v_dim = qk_dim or view.head_dim, v_dim or view.head_dim
     if chunk and window:
         raise L.KernelError("paged_attention: a window and blocks of positions exclude one another")
@@ -190,7 +191,7 @@ def paged_attention(ctx, q: torch.Tensor, cache: ops.KvLayerView, heads: int, wi
     elif out.dim() != 2 or out.shape[0] != T or out.shape[1] < heads * v_dim or out.dtype != q.dtype or not out.is_contiguous():
         raise L.KernelError(f"paged_attention: out must be a contiguous [{T}, >= {heads * v_dim}] of {q.dtype}, got {tuple(out.shape)} of {out.dtype}")
     tailed = chunk > 0 or sink_values is not None or gate is not None or out_scale != 1.0 or out.shape[1] != heads * v_dim
-    capped = softcap > 0 or sink or tailed
+    capped = softcap > 0 or sink or tailed or keep_first > 0
     generic = qk_dim != view.head_dim or v_dim != view.head_dim or not has_tensor_core_kernel(q.dtype, view.head_dim, heads, view.kv_heads)
     generic = generic or (tailed and out.shape[1] % 8 != 0)
     work = None if generic else _work_lists(ctx)
@@ -198,7 +199,7 @@ def paged_attention(ctx, q: torch.Tensor, cache: ops.KvLayerView, heads: int, wi
         generic = True    # prompt portions with capped scores run on the kernel that TMA feeds, or on the generic one
     if generic:
         ops.attention_generic(q, cache, ctx.positions, ctx.seg_of_token, window, scale, out, heads, rt.status, qk_dim, v_dim, softcap, sink, chunk=chunk,
-                              sink_values=sink_values, gate=gate, out_scale=out_scale)
+                              sink_values=sink_values, gate=gate, out_scale=out_scale, keep_first=keep_first)
         return out
     tail_ref = None
     if tailed:
@@ -213,7 +214,7 @@ def paged_attention(ctx, q: torch.Tensor, cache: ops.KvLayerView, heads: int, wi
             t.gate, t.gate_parts, t.gate_row, t.gate_stride = g.data_ptr() + 4 * col, g.shape[0], g.shape[2], T * g.shape[2]
         tail_ref = C.byref(t)
     window = -int(chunk) if chunk else window   # the kernels take blocks of positions as a negative window
-    extra = (float(softcap), 1 if sink else 0, tail_ref) if capped else ()
+    extra = (float(softcap), 1 if sink else 0, tail_ref, keep_first) if capped else ()
     tail = "_capped" if capped else ""
     stream = ops._stream()
     if work["n_dec"]:

@@ -25,10 +25,13 @@ L.register("ib_gemm_tcgen05_2cta", [L._p, L._p, L._p, L._i, L._i, L._i, L._p, L.
 L.register("ib_gemm_swiglu_tcgen05_2cta", [L._p, L._p, L._p, L._i, L._i, L._i, L._p, L._p])
 L.register("ib_gemm_xielu_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p, L._p, L._p])
 L.register("ib_gemm_xielu_tcgen05_2cta", [L._p, L._p, L._p, L._i, L._i, L._i, L._p, L._p, L._p])
+L.register("ib_gemm_relu2_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p, L._p])
+L.register("ib_gemm_relu2_tcgen05_2cta", [L._p, L._p, L._p, L._i, L._i, L._i, L._p, L._p])
 L.register("ib_gemm_tcgen05_2cta_add", [L._p, L._p, L._p, L._i, L._i, L._i, L._p, L._p])
 L.register("ib_gemm_qkv_tcgen05_2cta", [L._p, L._p, L._i, L._i, L._p, L._p, L._f, L._p, L._p, L._p, L._p, L._p, C.POINTER(L.KvView), L._i, L._i, L._p, L._p])
 
 L.register("ib_gemm_grouped_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._p, L._p, L._i, L._p, L._p])
+L.register("ib_gemm_grouped_relu2_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._p, L._p, L._i, L._p, L._p])
 L.register("ib_gemm_grouped_swiglu_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._p, L._p, L._i, L._p, L._p])
 
 # Runtime options that steer the choice (config/runtime_options.py): `pair_min_tokens` (129: the fused gate/up product runs on the
@@ -252,32 +255,37 @@ def gemm_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, sta
     L.call("ib_gemm_swiglu_tcgen05", x.data_ptr(), w_gate_up.data_ptr(), act.data_ptr(), T, I, K, bn, 1 if half else 0, status.data_ptr(), ops._stream())
 
 
-XIELU_MIN_ROW_BLOCKS = 32   # 128-row blocks of the matrix from which up to 128 tokens keep the whole k-range in one CTA (that many CTAs fill the memory system)
+ACT_MIN_ROW_BLOCKS = 32   # 128-row blocks of the matrix from which up to 128 tokens keep the whole k-range in one CTA (that many CTAs fill the memory system)
 
 
-def xielu_in_epilogue(T: int, N: int, K: int, sm_count: int = FITTED_SM_COUNT) -> bool:
-    """Whether the product of T tokens with an [N, K] matrix applies the xIELU activation in its epilogue: above 128 tokens always; up to
+def act_in_epilogue(T: int, N: int, K: int, sm_count: int = FITTED_SM_COUNT) -> bool:
+    """Whether the product of T tokens with an [N, K] matrix applies an activation (xIELU, squared ReLU) in its epilogue: above 128 tokens always; up to
     128 when the matrix has enough row blocks to fill the GPU without cutting the k-range (otherwise the k-range is split over CTAs and
-    `ops.xielu_rows` adds the partial sums). A function of the sizes only."""
+    a row-wise kernel adds the partial sums). A function of the sizes only."""
     if not supports(K):
         return False
-    return T > 128 or -(-N // 128) >= XIELU_MIN_ROW_BLOCKS or choose(T, N, K, True, sm_count)[1] == 1
+    return T > 128 or -(-N // 128) >= ACT_MIN_ROW_BLOCKS or choose(T, N, K, True, sm_count)[1] == 1
 
 
-def gemm_xielu(rt, x: torch.Tensor, lw, pq: torch.Tensor, act: torch.Tensor) -> None:
-    """act [T, N] bfloat16 = xielu(x w^T) with pq = (p, q) float32 on the device; the kernel's form is chosen like `linear`'s, without
-    cutting the k-range."""
+def gemm_act(rt, x: torch.Tensor, lw, kind: str, act: torch.Tensor, pq: Optional[torch.Tensor] = None) -> None:
+    """act [T, N] bfloat16 = activation of x w^T: kind "xielu" with pq = (p, q) float32 on the device, or "relu2" (max(z, 0)^2); the kernel's form is
+    chosen like `linear`'s, without cutting the k-range."""
     T, K = x.shape
     ops._check("x", x, torch.bfloat16)
     ops._check("w", lw.weight, torch.bfloat16, (lw.n, K))
     ops._check("act", act, torch.bfloat16, (T, lw.n))
-    ops._check("pq", pq, torch.float32, (2,))
+    extra = ()
+    if kind == "xielu":
+        ops._check("pq", pq, torch.float32, (2,))
+        extra = (pq.data_ptr(),)
+    elif kind != "relu2":
+        raise L.KernelError(f"gemm_act: activation {kind!r} is not known (xielu, relu2)")
     how = ("pair",) if T >= rt.options.pair_always_tokens else (plan(T, lw.n, K, rt.sm_count, False) if T > 128 else None)
     if how is not None and how[0] == "pair":
-        L.call("ib_gemm_xielu_tcgen05_2cta", x.data_ptr(), lw.weight.data_ptr(), act.data_ptr(), T, lw.n, K, pq.data_ptr(), rt.status.data_ptr(), ops._stream())
+        L.call(f"ib_gemm_{kind}_tcgen05_2cta", x.data_ptr(), lw.weight.data_ptr(), act.data_ptr(), T, lw.n, K, *extra, rt.status.data_ptr(), ops._stream())
         return
     bn, _, wide = how[1:] if how is not None else choose(T, lw.n, K, False, rt.sm_count)
-    L.call("ib_gemm_xielu_tcgen05", x.data_ptr(), lw.weight.data_ptr(), act.data_ptr(), T, lw.n, K, bn, 1 if wide else 0, pq.data_ptr(), rt.status.data_ptr(), ops._stream())
+    L.call(f"ib_gemm_{kind}_tcgen05", x.data_ptr(), lw.weight.data_ptr(), act.data_ptr(), T, lw.n, K, bn, 1 if wide else 0, *extra, rt.status.data_ptr(), ops._stream())
 
 
 # ---------------------------------------------------------------- products on regrouped rows (routed experts)
@@ -293,10 +301,10 @@ def grouped_token_tile(rows: int, groups: int, inter: int = 0, sm_count: int = F
     return 256 if ctas >= 2 * sm_count else 128
 
 
-def grouped_supported(k: int, inter: int, bn: int) -> bool:
-    """Whether the tcgen05 kernel takes the experts' two products: inner sizes that are multiples of 8, and for tiles of 16 or 32 tokens
-    (64 gate rows and their up rows in one accumulator) an expert size that is a multiple of 64."""
-    return k % 8 == 0 and inter % 8 == 0 and (bn >= 64 or inter % 64 == 0)
+def grouped_supported(k: int, inter: int, bn: int, gated: bool = True) -> bool:
+    """Whether the tcgen05 kernel takes the experts' two products: inner sizes that are multiples of 8, and for gated experts and tiles of 16 or
+    32 tokens (64 gate rows and their up rows in one accumulator) an expert size that is a multiple of 64."""
+    return k % 8 == 0 and inter % 8 == 0 and (not gated or bn >= 64 or inter % 64 == 0)
 
 
 def gemm_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bn: int, offsets: torch.Tensor, tiles: torch.Tensor, status: torch.Tensor) -> None:
@@ -308,6 +316,16 @@ def gemm_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bn: int, o
     ops._check("w", w, torch.bfloat16, (E, N, K))
     ops._check("out", out, torch.float32, (R, N))
     L.call("ib_gemm_grouped_tcgen05", x.data_ptr(), w.data_ptr(), out.data_ptr(), R, N, K, bn, offsets.data_ptr(), tiles.data_ptr(), E, status.data_ptr(), ops._stream())
+
+
+def gemm_grouped_relu2(x: torch.Tensor, w: torch.Tensor, act: torch.Tensor, bn: int, offsets: torch.Tensor, tiles: torch.Tensor, status: torch.Tensor) -> None:
+    """act [R, N] bfloat16 = max(w[e] x[r], 0)^2 for the regrouped rows; arguments as for `gemm_grouped`."""
+    R, K = x.shape
+    E, N, _ = w.shape
+    ops._check("x", x, torch.bfloat16)
+    ops._check("w", w, torch.bfloat16, (E, N, K))
+    ops._check("act", act, torch.bfloat16, (R, N))
+    L.call("ib_gemm_grouped_relu2_tcgen05", x.data_ptr(), w.data_ptr(), act.data_ptr(), R, N, K, bn, offsets.data_ptr(), tiles.data_ptr(), E, status.data_ptr(), ops._stream())
 
 
 def gemm_grouped_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, bn: int, offsets: torch.Tensor, tiles: torch.Tensor, status: torch.Tensor) -> None:

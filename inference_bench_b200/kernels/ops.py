@@ -247,8 +247,8 @@ def qk_norm_rope_kv(qkv: torch.Tensor, q_norm_w: Optional[torch.Tensor], k_norm_
 def attention_generic(q: torch.Tensor, kv: KvLayerView, positions: torch.Tensor, seg_of_token: torch.Tensor, window: Optional[int],
                       scale: float, out: torch.Tensor, heads: int, status: torch.Tensor, qk_dim: Optional[int] = None, v_dim: Optional[int] = None,
                       softcap: float = 0.0, sink: bool = False, chunk: int = 0, sink_values: Optional[torch.Tensor] = None,
-                      gate: Optional[tuple] = None, out_scale: float = 1.0) -> None:
-    """softcap > 0: scores become softcap * tanh(score / softcap); sink: the softmax's denominator has one added (a key of score 0
+                      gate: Optional[tuple] = None, out_scale: float = 1.0, keep_first: int = 0) -> None:
+    """keep_first > 0 (with a window): the first positions of the request are seen as well. softcap > 0: scores become softcap * tanh(score / softcap); sink: the softmax's denominator has one added (a key of score 0
     without a value; with sink_values, float32 [heads], a key of that score per head); qk_dim, v_dim: a query/key head's and a value
     head's size (default: the cache's row). chunk > 0: a position sees the earlier positions of its own block of `chunk` positions
     (counted from 0) instead of a window. gate = (float32 partial sums [P, T, row], column of the first head): head h's output is
@@ -275,7 +275,8 @@ def attention_generic(q: torch.Tensor, kv: KvLayerView, positions: torch.Tensor,
     _check("seg_of_token", seg_of_token, torch.int32, (T,))
     L.call("ib_attention_generic", q.data_ptr(), dtype_code(q.dtype), C.byref(view), positions.data_ptr(), seg_of_token.data_ptr(),
            int(window or 0), float(scale), out.data_ptr(), T, heads, status.data_ptr(), qk_dim, v_dim, float(softcap or 0.0), 1 if sink else 0,
-           int(chunk or 0), _ptr(sink_values), g_ptr, g_P, g_stride, g_row, float(out_scale), out.shape[1], _stream())
+           int(chunk or 0), _ptr(sink_values), g_ptr, g_P, g_stride, g_row, float(out_scale), out.shape[1],
+           int(keep_first), _stream())
 
 
 def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
@@ -500,7 +501,9 @@ def latent_attention_mma(q_full: torch.Tensor, kv: KvLayerView, positions: torch
 
 
 # ---------------------------------------------------------------- routed experts (csrc/moe.cu)
-L.register("ib_moe_route", [L._p, L._i, L._ll, L._i, L._i, L._i, L._i, L._i, L._f, L._i, L._p, L._p, L._i, L._p, L._i, L._p])
+L.register("ib_moe_route", [L._p, L._i, L._ll, L._i, L._i, L._i, L._i, L._i, L._f, L._i, L._p, L._p, L._i, L._p, L._i, L._i, L._p, L._p])
+ROUTE_SCORES = {"softmax": 0, "sigmoid": 1, "chosen_softmax": 2}
+GROUPED_ACTS = {"none": 0, "swiglu": 1, "relu2": 2}
 L.register("ib_scatter_scaled_rows", [L._p, L._i, L._p, L._p, L._i, L._p, L._i, L._i, L._p])
 L.register("ib_moe_sort", [L._p, L._i, L._i, L._i, L._i, L._p, L._p, L._p, L._p, L._p])
 L.register("ib_gather_rows", [L._p, L._p, L._p, L._i, L._i, L._i, L._p])
@@ -521,24 +524,29 @@ def gather_rows(x: torch.Tensor, src_row: torch.Tensor, out: torch.Tensor) -> No
         raise L.KernelError(f"gather_rows: x has {x.shape[1]} columns, out {K}")
     L.call("ib_gather_rows", x.data_ptr(), src_row.data_ptr(), out.data_ptr(), R, K, x.element_size(), _stream())
 L.register("ib_gemm_grouped", [L._p, L._i, L._p, L._p, L._i, L._p, L._i, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p])
-L.register("ib_moe_combine", [L._p, L._p, L._p, L._i, L._p, L._i, L._ll, L._p, L._i, L._i, L._p])
+L.register("ib_moe_combine", [L._p, L._p, L._p, L._i, L._p, L._i, L._ll, L._p, L._i, L._i, L._p, L._i, L._ll, L._i, L._p])
 
 
 def moe_route(logits: torch.Tensor, n_groups: int, keep: int, top: int, route_scale: float, renorm: bool, idx: torch.Tensor, wt: torch.Tensor,
-              score: str = "softmax", correction: Optional[torch.Tensor] = None, group_top: int = 1) -> None:
-    """logits float32 [P, T, E] (partial sums) -> idx int32 [T, top], wt float32 [T, top]. score: "softmax" over all experts, or
-    "sigmoid" of every expert's logit on its own. correction: float32 [E] added to the scores where groups and experts are chosen (the
+              score: str = "softmax", correction: Optional[torch.Tensor] = None, group_top: int = 1, experts: Optional[int] = None,
+              logit_bias: Optional[torch.Tensor] = None) -> None:
+    """logits float32 [P, T, E] (partial sums) -> idx int32 [T, top], wt float32 [T, top]. score: "softmax" over all experts, "sigmoid" of every
+    expert's logit on its own, or "chosen_softmax" (chosen by the logits, weighted by the softmax over the chosen ones). experts: how many
+    of a row's first entries are experts (default: all). logit_bias: float32 [E] added to the logits. correction: float32 [E] added to the scores where groups and experts are chosen (the
     weights are the scores without it). group_top: a group's score is the sum of its `group_top` largest choice scores (1: the largest)."""
-    if score not in ("softmax", "sigmoid"):
-        raise L.KernelError(f"moe_route: score {score!r} is not known (softmax, sigmoid)")
+    if score not in ROUTE_SCORES:
+        raise L.KernelError(f"moe_route: score {score!r} is not known ({', '.join(ROUTE_SCORES)})")
     _check("logits", logits, torch.float32)
-    P, T, E = logits.shape
+    P, T, row = logits.shape
+    E = row if experts is None else int(experts)
+    if logit_bias is not None:
+        _check("logit_bias", logit_bias, torch.float32, (E,))
     _check("idx", idx, torch.int32, (T, top))
     _check("wt", wt, torch.float32, (T, top))
     if correction is not None:
         _check("correction", correction, torch.float32, (E,))
-    L.call("ib_moe_route", logits.data_ptr(), P, T * E, T, E, n_groups, keep, top, float(route_scale), 1 if renorm else 0, idx.data_ptr(), wt.data_ptr(),
-           1 if score == "sigmoid" else 0, _ptr(correction), int(group_top), _stream())
+    L.call("ib_moe_route", logits.data_ptr(), P, T * row, T, E, n_groups, keep, top, float(route_scale), 1 if renorm else 0, idx.data_ptr(), wt.data_ptr(),
+           ROUTE_SCORES[score], _ptr(correction), int(group_top), row, _ptr(logit_bias), _stream())
 
 
 def moe_sort(idx: torch.Tensor, n_experts: int, offsets: torch.Tensor, tile_start: torch.Tensor, row_of_pair: torch.Tensor, token_of_row: torch.Tensor,
@@ -556,10 +564,13 @@ def moe_sort(idx: torch.Tensor, n_experts: int, offsets: torch.Tensor, tile_star
 
 
 def gemm_grouped(x: torch.Tensor, src_row: Optional[torch.Tensor], w: torch.Tensor, out: torch.Tensor, offsets: torch.Tensor, tile_start: torch.Tensor,
-                 gated: bool, tensor_cores: bool = False) -> None:
+                 gated: bool, tensor_cores: bool = False, act: str = "none") -> None:
     """out[r] = w[e(r)] x[src_row[r] or r] for the regrouped rows r (expert e's rows are offsets[e]..offsets[e+1]); w [E, N or 2N, K]; with
-    `gated`, w holds gate rows then up rows and out = silu(gate) * up."""
+    `gated`, w holds gate rows then up rows and out = silu(gate) * up; act "relu2" (not gated): out = max(product, 0)^2."""
     R, N = out.shape
+    if act not in ("none", "relu2") or (gated and act != "none"):
+        raise L.KernelError(f"gemm_grouped: activation {act!r} (none, relu2; a gated product has its own)")
+    code = GROUPED_ACTS["swiglu" if gated else act]
     E, rows_w, K = w.shape
     if rows_w != (2 * N if gated else N) or x.shape[1] != K:
         raise L.KernelError(f"gemm_grouped: w {tuple(w.shape)}, x {tuple(x.shape)}, out {tuple(out.shape)} do not fit (gated={gated})")
@@ -572,10 +583,10 @@ def gemm_grouped(x: torch.Tensor, src_row: Optional[torch.Tensor], w: torch.Tens
         if not rows_mma_fits(x, w):
             raise L.KernelError("gemm_grouped: the tensor-core kernel needs bfloat16 operands with an inner size that is a multiple of 8")
         L.call("ib_gemm_grouped_mma", x.data_ptr(), _ptr(src_row), w.data_ptr(), out.data_ptr(), dtype_code(out.dtype), offsets.data_ptr(), tile_start.data_ptr(), R, E,
-               N, K, 1 if gated else 0, _stream())
+               N, K, code, _stream())
         return
     L.call("ib_gemm_grouped", x.data_ptr(), dtype_code(x.dtype), _ptr(src_row), w.data_ptr(), dtype_code(w.dtype), out.data_ptr(), dtype_code(out.dtype),
-           offsets.data_ptr(), tile_start.data_ptr(), R, E, N, K, 1 if gated else 0, _stream())
+           offsets.data_ptr(), tile_start.data_ptr(), R, E, N, K, code, _stream())
 
 
 def scatter_scaled_rows(x: torch.Tensor, row_of_pair: torch.Tensor, wt: torch.Tensor, out: torch.Tensor) -> None:
@@ -589,9 +600,11 @@ def scatter_scaled_rows(x: torch.Tensor, row_of_pair: torch.Tensor, wt: torch.Te
     L.call("ib_scatter_scaled_rows", x.data_ptr(), dtype_code(x.dtype), row_of_pair.data_ptr(), wt.data_ptr(), top, out.data_ptr(), T * top, K, _stream())
 
 
-def moe_combine(y: torch.Tensor, row_of_pair: torch.Tensor, wt: torch.Tensor, base: Optional[torch.Tensor], out: torch.Tensor, weighted: bool = True) -> None:
+def moe_combine(y: torch.Tensor, row_of_pair: torch.Tensor, wt: torch.Tensor, base: Optional[torch.Tensor], out: torch.Tensor, weighted: bool = True,
+                gate: Optional[tuple] = None) -> None:
     """out[t] = sum_p base[p][t] + sum_k wt[t, k] * y[row_of_pair[t * top + k]]; y float32 [R, H], base float32 [P, T, H] or None.
-    weighted=False: the plain sum over a token's choices (wt gives the shape only)."""
+    weighted=False: the plain sum over a token's choices (wt gives the shape only). gate = (float32 partial sums [P, T, row], column): base counts
+    times the sigmoid of the token's entry in that column."""
     T, top = wt.shape
     H = y.shape[1]
     _check("y", y, torch.float32, (T * top, H))
@@ -602,11 +615,25 @@ def moe_combine(y: torch.Tensor, row_of_pair: torch.Tensor, wt: torch.Tensor, ba
         if base.dim() != 3 or tuple(base.shape[1:]) != (T, H):
             raise L.KernelError(f"moe_combine: base must be [P, {T}, {H}], got {tuple(base.shape)}")
         P = base.shape[0]
-    L.call("ib_moe_combine", y.data_ptr(), row_of_pair.data_ptr(), wt.data_ptr() if weighted else None, top, _ptr(base), P, T * H, out.data_ptr(), T, H, _stream())
+    g_ptr, g_P, g_stride, g_row = None, 0, 0, 0
+    if gate is not None:
+        g, col = gate
+        _check("gate", g, torch.float32)
+        g_P, g_row = g.shape[0], g.shape[2]
+        if g.dim() != 3 or g.shape[1] != T or not 0 <= col < g_row:
+            raise L.KernelError(f"moe_combine: the gate's partial sums {tuple(g.shape)} have no column {col} for {T} tokens")
+        g_ptr, g_stride = g.data_ptr() + 4 * col, T * g_row
+    L.call("ib_moe_combine", y.data_ptr(), row_of_pair.data_ptr(), wt.data_ptr() if weighted else None, top, _ptr(base), P, T * H, out.data_ptr(), T, H,
+           g_ptr, g_P, g_stride, g_row, _stream())
 
 
 # ---------------------------------------------------------------- layer norm, input convolution, depth average (csrc/layernorm.cu)
-L.register("ib_add_layernorm", [L._p, L._p, L._i, L._ll, L._p, L._p, L._p, L._p, L._i, L._p, L._i, L._i, L._f, L._i, L._p, L._i, L._p, L._p, L._p, L._i, L._p, L._ll, L._p])
+L.register("ib_add_layernorm", [L._p, L._p, L._i, L._ll, L._p, L._p, L._p, L._p, L._i, L._p, L._i, L._i, L._f, L._i, L._p, L._i, L._p, L._p, L._p, L._i, L._p, L._ll, L._p, L._f,
+                               L._i, L._p])
+L.register("ib_softcap_values", [L._p, L._ll, L._f, L._p])
+L.register("ib_embed_layernorm", [L._p, L._i, L._p, L._p, L._p, L._f, L._p, L._i, L._i, L._i, L._p, L._p])
+L.register("ib_shift_mixes", [L._p, L._p, L._i, L._p, L._ll, L._p, L._p, L._p, L._p, L._i, L._i, L._i, L._p])
+L.register("ib_add_layernorm_mixes_single", [L._p, L._p, L._i, L._ll, L._f, L._p, L._p, L._f, L._p, L._i, L._p, L._i, L._i, L._i, L._p, L._p, L._ll, L._i, L._p])
 L.register("ib_causal_conv_rows", [L._p, L._p, L._i, L._p, L._i, L._i, L._i, L._p, L._p, L._p, L._i, L._p, L._ll, L._p])
 L.register("ib_depth_average", [L._p, L._p, L._i, L._ll, L._p, L._p, L._p, L._ll, L._i, L._p, L._i, L._i, L._p])
 L.register("ib_scale_values", [L._p, L._ll, L._f, L._p])
@@ -630,9 +657,10 @@ class ConvLayout:
 
 def add_layernorm(x: torch.Tensor, delta: Optional[torch.Tensor], w: torch.Tensor, out: torch.Tensor, eps: float, rows: Optional[torch.Tensor] = None,
                   delta_scale: Optional[torch.Tensor] = None, delta_bias: Optional[torch.Tensor] = None, x_copy: Optional[torch.Tensor] = None,
-                  layout: Optional[ConvLayout] = None) -> None:
+                  layout: Optional[ConvLayout] = None, b: Optional[torch.Tensor] = None, delta_mult: float = 1.0, early: bool = True) -> None:
     """v = x + delta_scale * (sum_p delta[p] + delta_bias) (x updated in place unless `rows` gathers); x_copy = v (optional);
-    out = w * (v - mean) / sqrt(var + eps). With `layout` out is float32 [T + halo * segments, H] in the layout of `ConvLayout`."""
+    out = w * (v - mean) / sqrt(var + eps) (+ b, float32 [H]). delta_mult: a constant in the place of delta_scale. early: whether the kernels that
+    follow may be scheduled while this one runs. With `layout` out is float32 [T + halo * segments, H] in the layout of `ConvLayout`."""
     T, H = x.shape
     _check("x", x, torch.float32)
     _check("w", w, torch.float32, (H,))
@@ -647,6 +675,8 @@ def add_layernorm(x: torch.Tensor, delta: Optional[torch.Tensor], w: torch.Tenso
     for name, v in (("delta_scale", delta_scale), ("delta_bias", delta_bias)):
         if v is not None:
             _check(name, v, torch.float32, (H,))
+    if b is not None:
+        _check("b", b, torch.float32, (H,))
     if x_copy is not None:
         _check("x_copy", x_copy, torch.float32, (T, H))
     if rows is not None:
@@ -655,7 +685,7 @@ def add_layernorm(x: torch.Tensor, delta: Optional[torch.Tensor], w: torch.Tenso
     L.call("ib_add_layernorm", x.data_ptr(), _ptr(delta), P, stride, _ptr(delta_scale), _ptr(delta_bias), w.data_ptr(), out.data_ptr(), dtype_code(out.dtype),
            _ptr(rows), n_rows, H, float(eps), 0 if rows is not None else 1, _ptr(x_copy), lay.halo if lay else 0, _ptr(lay.seg_of_token) if lay else None,
            _ptr(lay.seg_start) if lay else None, _ptr(lay.seg_slot) if lay else None, lay.n_segments if lay else 0, _ptr(lay.state) if lay else None,
-           lay.slot_stride if lay else 0, _stream())
+           lay.slot_stride if lay else 0, _ptr(b), float(delta_mult), 1 if early else 0, _stream())
 
 
 def causal_conv_rows(ext: torch.Tensor, w: torch.Tensor, out: torch.Tensor, layout: ConvLayout) -> None:
@@ -725,11 +755,65 @@ def scale_values(v: torch.Tensor, s: float) -> None:
     L.call("ib_scale_values", v.data_ptr(), v.numel(), float(s), _stream())
 
 
+def softcap_values(v: torch.Tensor, cap: float) -> None:
+    """v = cap * tanh(v / cap), float32, in place."""
+    _check("v", v, torch.float32)
+    L.call("ib_softcap_values", v.data_ptr(), v.numel(), float(cap), _stream())
+
+
+def embed_layernorm(table: torch.Tensor, tokens: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], eps: float, x: torch.Tensor, status: torch.Tensor) -> None:
+    """x[t] = layer norm (weight w, bias b) of table[tokens[t]], float32."""
+    V, H = table.shape
+    T = tokens.shape[0]
+    _check("table", table)
+    _check("tokens", tokens, torch.int32)
+    _check("w", w, torch.float32, (H,))
+    if b is not None:
+        _check("b", b, torch.float32, (H,))
+    _check("x", x, torch.float32, (T, H))
+    L.call("ib_embed_layernorm", table.data_ptr(), dtype_code(table.dtype), tokens.data_ptr(), w.data_ptr(), _ptr(b), float(eps), x.data_ptr(), T, H, V, status.data_ptr(), _stream())
+
+
+def shift_mixes(h: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, seg_of_token: torch.Tensor, seg_start: torch.Tensor, seg_slot: torch.Tensor, out: torch.Tensor) -> None:
+    """out[m, t] = h[t] + (h[t - 1] - h[t]) * mu[m] for every mix m; the row before a segment's first is state[slot] (float32 [slots, H]), which
+    then becomes the segment's last row of h. h float32 [T, H], mu float32 [M, H], out [M, T, H]."""
+    T, H = h.shape
+    M = mu.shape[0]
+    _check("h", h, torch.float32)
+    _check("mu", mu, torch.float32, (M, H))
+    _check("state", state, torch.float32)
+    _check("out", out, None, (M, T, H))
+    L.call("ib_shift_mixes", h.data_ptr(), mu.data_ptr(), M, state.data_ptr(), state.stride(0), seg_of_token.data_ptr(), seg_start.data_ptr(), seg_slot.data_ptr(),
+           out.data_ptr(), dtype_code(out.dtype), T, H, _stream())
+
+
+def add_layernorm_mixes_single(x: torch.Tensor, delta: Optional[torch.Tensor], mult: float, w: torch.Tensor, b: Optional[torch.Tensor], eps: float, mu: torch.Tensor,
+                               state: torch.Tensor, seg_slot: torch.Tensor, out: torch.Tensor, early: bool = True) -> None:
+    """x += mult * sum_p delta[p], the layer norm and `shift_mixes` in one kernel for a step whose row t is segment t."""
+    T, H = x.shape
+    M = mu.shape[0]
+    _check("x", x, torch.float32)
+    _check("w", w, torch.float32, (H,))
+    if b is not None:
+        _check("b", b, torch.float32, (H,))
+    _check("mu", mu, torch.float32, (M, H))
+    _check("state", state, torch.float32)
+    _check("seg_slot", seg_slot, torch.int32)
+    _check("out", out, None, (M, T, H))
+    d_ptr, P, stride = _delta(x, delta)
+    L.call("ib_add_layernorm_mixes_single", x.data_ptr(), d_ptr, P, stride, float(mult), w.data_ptr(), _ptr(b), float(eps), mu.data_ptr(), M, out.data_ptr(),
+           dtype_code(out.dtype), T, H, seg_slot.data_ptr(), state.data_ptr(), state.stride(0), 1 if early else 0, _stream())
+
+
 # ---------------------------------------------------------------- gated linear recurrence (csrc/gated_recurrence.cu)
 L.register("ib_gated_recurrence", [L._p, L._i, L._ll, L._p, L._p, L._p, L._ll, L._p, L._p, L._i, L._p, L._i, L._i, L._i, L._p, L._p, L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p])
 L.register("ib_recurrence_chunks_finish", [L._p, L._i, L._p, L._i, L._p, L._p, L._ll, L._p, L._p, L._p, L._p, L._i, L._i, L._i, L._p])
 L.KERNELS_PER_CALL["ib_recurrence_chunks_finish"] = 2
 RECURRENCE_CHUNK = 64   # rows of a chunk of the chunked form (csrc/gated_recurrence.cu: chunk_apply takes 64 rows a CTA)
+L.register("ib_recurrence_parts", [L._p, L._p, L._p, L._i, L._ll, L._i, L._p, L._p, L._ll, L._p, L._p, L._i, L._p, L._i, L._i, L._i, L._p, L._p, L._p, L._p, L._p, L._i,
+                                   L._p, L._p, L._i, L._f, L._p, L._p])
+L.register("ib_decay_rows", [L._p, L._i, L._ll, L._i, L._p, L._p, L._p, L._i, L._i, L._p])
+L.register("ib_head_norm_gate", [L._p, L._p, L._f, L._p, L._i, L._ll, L._i, L._p, L._i, L._i, L._i, L._i, L._p])
 L.register("ib_head_rmsnorm", [L._p, L._p, L._f, L._p, L._i, L._ll, L._i, L._p])
 
 
@@ -781,6 +865,107 @@ def gated_recurrence(proj: torch.Tensor, f_bias: torch.Tensor, lower: torch.Tens
            chunk_state.data_ptr(), chunk_decay.data_ptr(), qa.data_ptr(), out.data_ptr(), heads, dim, vdim, _stream())
 
 
+@dataclass
+class Parts:
+    """Float32 partial sums of one part of a projection: `count` sums, `stride` elements apart, rows of `row` elements; `tensor` holds them from
+    element `offset` on (a column of a wider projection, or one of several products stored together)."""
+    tensor: torch.Tensor
+    count: int
+    stride: int
+    row: int
+    offset: int = 0
+
+    @classmethod
+    def columns(cls, proj: torch.Tensor, col: int = 0) -> "Parts":
+        """The columns from `col` on of a projection [P, T, R]."""
+        P, T, R = proj.shape
+        return cls(proj, P, T * R, R, col)
+
+    def ptr(self) -> int:
+        return self.tensor.data_ptr() + 4 * self.offset
+
+
+def recurrence(form: str, q: Parts, k: Parts, v: Parts, head_param: torch.Tensor, state: torch.Tensor, seg_start: torch.Tensor, seg_slot: torch.Tensor, n_segments: int,
+               out: torch.Tensor, heads: int, dim: int, vdim: int, seg_list: Optional[torch.Tensor] = None, long_segs: Optional[torch.Tensor] = None,
+               chunks: Optional[torch.Tensor] = None, cos: Optional[torch.Tensor] = None, sin: Optional[torch.Tensor] = None, k_scale: float = 1.0,
+               decay: Optional[torch.Tensor] = None) -> None:
+    """Linear recurrences over float32 partial sums of q, k (heads * dim columns) and v (heads * vdim), into out float32 [T, heads, vdim].
+    form "turned": S <- head_param[head] S + k v^T, o = S^T q, with q and k turned by cos and sin (float32 [T, n]: entry i with i + n; None for no
+    rotation) and k times k_scale. form "bonus": o = (S + diag(u) k v^T)^T q, then S <- diag(decay) S + k v^T, with u = head_param [heads * dim]
+    and decay float32 [T, heads * dim]. state, seg_list, long_segs, chunks: as for `gated_recurrence`."""
+    if form not in ("turned", "bonus"):
+        raise L.KernelError(f"recurrence: form {form!r} is not known (turned, bonus)")
+    T = out.shape[0]
+    _check("out", out, torch.float32, (T, heads, vdim))
+    if len({(p.count, p.stride, p.row) for p in (q, k, v)}) != 1:
+        raise L.KernelError("recurrence: q, k and v must be laid out alike")
+    for name, p, n in (("q", q, heads * dim), ("k", k, heads * dim), ("v", v, heads * vdim)):
+        _check(name, p.tensor, torch.float32)
+        if p.row < n or p.offset + (p.count - 1) * p.stride + (T - 1) * p.row + n > p.tensor.numel():
+            raise L.KernelError(f"recurrence: {name} does not hold {T} rows of {n} entries in {p.count} partial sums")
+    _check("head_param", head_param, torch.float32, (heads,) if form == "turned" else (heads * dim,))
+    if form == "bonus":
+        _check("decay", decay, torch.float32, (T, heads * dim))
+    half = 0
+    if cos is not None:
+        half = cos.shape[1]
+        _check("cos", cos, torch.float32, (T, half))
+        _check("sin", sin, torch.float32, (T, half))
+    _check("state", state, torch.float32)
+    if tuple(state.shape[1:]) != (heads, dim, vdim):
+        raise L.KernelError(f"recurrence: the state must be [slots, {heads}, {dim}, {vdim}], got {tuple(state.shape)}")
+    _check("seg_start", seg_start, torch.int32)
+    _check("seg_slot", seg_slot, torch.int32)
+
+    def walk(n, segs, table, chunk_state, chunk_decay, qa):
+        L.call("ib_recurrence_parts", q.ptr(), k.ptr(), v.ptr(), q.count, q.stride, q.row, head_param.data_ptr(), state.data_ptr(), heads * dim * vdim, seg_start.data_ptr(),
+               seg_slot.data_ptr(), n, out.data_ptr(), heads, dim, vdim, _ptr(segs), _ptr(table), _ptr(chunk_state), _ptr(chunk_decay), _ptr(qa), 2 if form == "turned" else 3,
+               _ptr(cos), _ptr(sin), half, float(k_scale), _ptr(decay), _stream())
+
+    if long_segs is None:
+        if seg_list is not None:
+            _check("seg_list", seg_list, torch.int32)
+            n_segments = seg_list.shape[0]
+        walk(n_segments, seg_list, None, None, None, None)
+        return
+    _check("long_segs", long_segs, torch.int32)
+    _check("chunks", chunks, torch.int32)
+    if seg_list is not None and seg_list.shape[0]:
+        walk(seg_list.shape[0], seg_list, None, None, None, None)
+    m = chunks.shape[0]
+    chunk_state = torch.empty((m, heads, dim, vdim), dtype=torch.float32, device=out.device)
+    chunk_decay = torch.empty((m, heads, dim), dtype=torch.float32, device=out.device)
+    qa = torch.empty((T, heads, dim), dtype=torch.float32, device=out.device)
+    walk(m, None, chunks, chunk_state, chunk_decay, qa)
+    L.call("ib_recurrence_chunks_finish", long_segs.data_ptr(), long_segs.shape[0], chunks.data_ptr(), m, seg_slot.data_ptr(), state.data_ptr(), heads * dim * vdim,
+           chunk_state.data_ptr(), chunk_decay.data_ptr(), qa.data_ptr(), out.data_ptr(), heads, dim, vdim, _stream())
+
+
+def decay_rows(low: torch.Tensor, w2: torch.Tensor, w0: torch.Tensor, decay: torch.Tensor) -> None:
+    """decay[t, c] = exp(-exp(w0[c] + sum_j w2[j, c] tanh(sum_p low[p, t, j]))): low float32 [P, T, rank], w2 float32 [rank, C], w0 float32 [C]."""
+    _check("low", low, torch.float32)
+    P, T, rank = low.shape
+    C_ = w0.shape[0]
+    _check("w2", w2, torch.float32, (rank, C_))
+    _check("w0", w0, torch.float32)
+    _check("decay", decay, torch.float32, (T, C_))
+    L.call("ib_decay_rows", low.data_ptr(), P, T * rank, rank, w2.data_ptr(), w0.data_ptr(), decay.data_ptr(), T, C_, _stream())
+
+
+def head_norm_gate(o: torch.Tensor, w: Optional[torch.Tensor], eps: float, gate: Parts, out: torch.Tensor) -> None:
+    """out[t, a, :] = w * o[t, a, :] / sqrt(mean(o[t, a, :]^2) + eps) * silu(gate[t, a, :]): o float32 [T, heads, V], w float32 [heads * V] or None (no
+    weight), gate float32 partial sums of heads * V columns, out [T, heads * V]."""
+    T, heads, V = o.shape
+    _check("o", o, torch.float32)
+    if w is not None:
+        _check("w", w, torch.float32, (heads * V,))
+    _check("gate", gate.tensor, torch.float32)
+    if gate.row < heads * V or gate.offset + (gate.count - 1) * gate.stride + (T - 1) * gate.row + heads * V > gate.tensor.numel():
+        raise L.KernelError(f"head_norm_gate: the gate does not hold {T} rows of {heads * V} entries in {gate.count} partial sums")
+    _check("out", out, None, (T, heads * V))
+    L.call("ib_head_norm_gate", o.data_ptr(), _ptr(w), float(eps), gate.ptr(), gate.count, gate.stride, gate.row, out.data_ptr(), dtype_code(out.dtype), T, heads, V, _stream())
+
+
 def head_rmsnorm(o: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor) -> None:
     """out[t, a, :] = w * o[t, a, :] / sqrt(mean(o[t, a, :]^2) + eps); o float32 [T, heads, V], out [T, heads * V] in its own dtype."""
     T, heads, V = o.shape
@@ -796,6 +981,7 @@ L.register("ib_add_rmsnorm_ext", [L._p, L._p, L._i, L._ll, L._p, L._p, L._f, L._
 L.register("ib_loop_pack", [L._p, L._p, L._i, L._ll, L._p, L._p, L._p, L._i, L._i, L._i, L._p])
 L.register("ib_add_bias_rows", [L._p, L._p, L._i, L._i, L._p])
 L.register("ib_xielu_rows", [L._p, L._i, L._ll, L._p, L._p, L._i, L._i, L._i, L._p])
+L.register("ib_relu2_rows", [L._p, L._i, L._ll, L._p, L._i, L._i, L._i, L._p])
 L.register("ib_gated_rmsnorm", [L._p, L._p, L._f, L._p, L._i, L._ll, L._i, L._f, L._p, L._i, L._i, L._i, L._i, L._p])
 
 
@@ -870,6 +1056,14 @@ def xielu_rows(z: torch.Tensor, pq: torch.Tensor, act: torch.Tensor) -> None:
     _check("pq", pq, torch.float32, (2,))
     _check("act", act, None, (T, I))
     L.call("ib_xielu_rows", z.data_ptr(), P, T * I, pq.data_ptr(), act.data_ptr(), dtype_code(act.dtype), T, I, _stream())
+
+
+def relu2_rows(z: torch.Tensor, act: torch.Tensor) -> None:
+    """act = max(sum_p z[p], 0)^2."""
+    _check("z", z, torch.float32)
+    P, T, I = z.shape
+    _check("act", act, None, (T, I))
+    L.call("ib_relu2_rows", z.data_ptr(), P, T * I, act.data_ptr(), dtype_code(act.dtype), T, I, _stream())
 
 
 def gated_rmsnorm(o: torch.Tensor, w: torch.Tensor, eps: float, gate: torch.Tensor, gate_col: int, scale: float, out: torch.Tensor, out_col: int = 0) -> None:
@@ -1047,3 +1241,43 @@ def sigmoid_attention(q: torch.Tensor, kv: KvLayerView, positions: torch.Tensor,
         return
     L.call("ib_sigmoid_attention", q.data_ptr(), dtype_code(q.dtype), C.byref(view), positions.data_ptr(), seg_of_token.data_ptr(), float(scale), _ptr(r1), _ptr(r2),
            _ptr(pb), out.data_ptr(), _ptr(part), T, heads, qk_dim, v_dim, n_slices, slice_keys, status.data_ptr(), _stream())
+
+
+# ---------------------------------------------------------------- attention with several score maps over the same values (csrc/diff_attention.cu)
+L.register("ib_map_qkv", [L._p, L._i, L._ll, L._i, L._p, L._p, L._p, L._i, L._i, L._p, L._p, L._p, L._i, C.POINTER(L.KvView), L._i, L._i, L._i, L._i, L._i, L._i, L._p, L._p])
+L.register("ib_diff_combine", [L._p, L._i, L._f, L._f, L._f, L._p, L._ll, L._i, L._p])
+
+
+def map_qkv(proj: torch.Tensor, bias: Optional[torch.Tensor], cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], interleaved: bool, positions: torch.Tensor,
+            seg_of_token: torch.Tensor, q_out: torch.Tensor, kv: KvLayerView, heads: int, maps: int, dim: int, v_dim: int, status: torch.Tensor, write_kv: bool = True) -> None:
+    """proj float32 [P, T, R] = [heads x maps x dim | kv_heads x maps x dim | kv_heads x v_dim] (the queries alone without write_kv), bias float32 [R].
+    q_out [T, heads * maps * maps * dim]: a row of maps * dim entries per (head, map), zero outside the map's part. Keys (all maps of a kv head in
+    one row) and values go into the paged cache. interleaved: entries 2i and 2i + 1 are turned together, else i and i + rotary_dim/2."""
+    _check("proj", proj, torch.float32)
+    P, T, R = proj.shape
+    view = kv.c_view()
+    want = heads * maps * dim + (view.kv_heads * (maps * dim + v_dim) if write_kv else 0)
+    if R != want:
+        raise L.KernelError(f"map_qkv: the projection has {R} columns, expected {want}")
+    if bias is not None:
+        _check("bias", bias, torch.float32, (R,))
+    _check("q_out", q_out, None, (T, heads * maps * maps * dim))
+    _check("positions", positions, torch.int32, (T,))
+    _check("seg_of_token", seg_of_token, torch.int32, (T,))
+    half = 0
+    if cos is not None:
+        half = cos.shape[1]
+        _check("cos", cos, torch.float32, (T, half))
+        _check("sin", sin, torch.float32, (T, half))
+    L.call("ib_map_qkv", proj.data_ptr(), P, T * R, R, _ptr(bias), _ptr(cos), _ptr(sin), half, 1 if interleaved else 0, positions.data_ptr(), seg_of_token.data_ptr(),
+           q_out.data_ptr(), dtype_code(q_out.dtype), C.byref(view), 1 if write_kv else 0, T, heads, maps, dim, v_dim, status.data_ptr(), _stream())
+
+
+def diff_combine(a: torch.Tensor, lam: float, eps: float, factor: float, out: torch.Tensor, v_dim: int) -> None:
+    """out[t, h] = factor * u / sqrt(mean(u^2) + eps) with u = a[t, h, 0] - lam * a[t, h, 1]; a [T, heads * 2 * v_dim], out [T, heads * v_dim]."""
+    T, n = out.shape
+    _check("out", out)
+    _check("a", a, out.dtype, (T, 2 * n))
+    if n % v_dim:
+        raise L.KernelError(f"diff_combine: rows of {n} entries are not whole heads of {v_dim}")
+    L.call("ib_diff_combine", a.data_ptr(), dtype_code(a.dtype), float(lam), float(eps), float(factor), out.data_ptr(), T * (n // v_dim), v_dim, _stream())

@@ -30,21 +30,28 @@ class WeightSpec:
     "gate_floor": lower bounds of a forget gate, used in float32; random U(0, 0.9)
     "unit":   per-channel mixing weights, used in float32; random U(0, 1)
     "log_rate": logarithms of decay rates, used in float32; random log U(0.5, 8)
+    "decay_bias": what a decay exp(-exp(z)) adds to z, used in float32; random U(-6, 0)
     "mix":    weights of an average over the n entries of the tensor's last axis, used in float32; random around 1 / n
-    "table":  integer table, int32."""
+    "table":  integer table, int32.
+    `free` lists the axes whose size the checkpoint decides (the shape's entry there is what random weights are made with)."""
     name: str
     shape: tuple[int, ...]
     role: str = "matrix"
     std: float = 0.02
+    free: tuple[int, ...] = ()
+
+    def fits(self, shape) -> bool:
+        return len(shape) == len(self.shape) and all(a == b or i in self.free for i, (a, b) in enumerate(zip(shape, self.shape)))
 
 
 # ------------------------------------------------------------------ what a mixer asks of the cache
 @dataclass(frozen=True)
 class PagedKV:
-    """Keys and values for every token (or for the last `window` tokens) of a request, in pages."""
+    """Keys and values for every token (or for the last `window` tokens and the first `keep_first`) of a request, in pages."""
     kv_heads: int
     head_dim: int
     window: Optional[int] = None
+    keep_first: int = 0     # with a window: the positions 0 .. keep_first - 1 stay for as long as the request lives
 
 
 @dataclass(frozen=True)
@@ -105,7 +112,16 @@ class NormedDelta:
     bias: Optional[torch.Tensor] = None     # float32 [H], added to the summed partial sums before the norm
 
 
+@dataclass
+class ScaledDelta:
+    """A contribution to the residual stream that is multiplied by a constant where it is added: x += scale * (sum of `delta`). What a block
+    with a residual multiplier leaves for the next norm; `Norm.takes_scaled_delta` says whether a norm can add one."""
+    delta: torch.Tensor     # float32 [P, T, H]
+    scale: float
+
+
 class Norm(Part):
+    takes_scaled_delta = False   # True: `forward` takes a `ScaledDelta` as delta
     takes_normed_delta = False   # True: `forward` takes a `NormedDelta` as delta
 
     def forward(self, ctx: "StepContext", x: torch.Tensor, delta: Optional[torch.Tensor], rows: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -128,6 +144,8 @@ class PositionEncoding(Part):
 
 class Mixer(Part):
     adds_to_residual = False   # True: forward takes `residual=` and may add its contribution there itself
+    runs_norm = False          # True: the block calls `forward_normed(ctx, norm, x, pending, cache)` instead of running its input norm and `forward`:
+                               # a mixer that reads the normed rows in more than one form (several shifted mixes of them) makes them in its own kernels
     out_bias: Optional[torch.Tensor] = None   # float32 [H], set at bind: a vector that belongs to every row of the contribution and that the
                                               # kernel which adds the contribution to the stream adds with it (only blocks that say so take such a mixer)
 

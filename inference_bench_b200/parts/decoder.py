@@ -17,6 +17,8 @@ def _build(table: dict, what: str, spec: PartSpec):
     params = dict(spec.params)
     if isinstance(params.get("position"), PartSpec):
         params["position"] = _build(base.POSITION_ENCODINGS, "position encoding", params["position"])
+    if isinstance(params.get("norm"), PartSpec):   # a norm that belongs to the part itself (an embedding's)
+        params["norm"] = _build(base.NORMS, "norm", params["norm"])
     return base.make(table, what, spec.kind, **params)
 
 
@@ -82,6 +84,8 @@ class Decoder:
             if pending.bias is not None:
                 y = y + pending.bias
             return out + pending.norm.w * (y * torch.rsqrt((y * y).mean(-1, keepdim=True) + pending.norm.eps))
+        if isinstance(pending, base.ScaledDelta):
+            return out + pending.scale * pending.delta.sum(0).index_select(0, rows)
         if pending is not None:
             for p in range(pending.shape[0]):
                 out = out + pending[p].index_select(0, rows)

@@ -9,6 +9,9 @@ plus (optionally) one shared expert that every token uses.
 that is added to s where groups and experts are chosen and left out of the weights; `group_top` n makes a group's score the sum of
 its n largest choice scores (experts of groups that do not stay cannot be chosen, whatever the sign of their scores). `weight_on="input"`: the weight scales what the expert
 reads, out = sum_e down_e(silu(gate_e (weight_e h)) * up_e (weight_e h)), which is not the same thing for a gated expert.
+`score="chosen_softmax"`: the `top` experts with the largest logits are chosen and weighted by the softmax over the chosen logits alone;
+`router_bias` names a bias of the logits. `activation="relu2"`: experts and shared expert without a gate, down_e(max(up_e h, 0)^2).
+`shared_gate` names a vector (one row): the shared expert's output is multiplied by the sigmoid of its product with the token's row.
 The step's (token, expert) pairs are regrouped by expert on the device (no trip to the host, so the step can be captured),
 the experts' products run on the regrouped rows, and the weighted sum returns them to token order.
 """
@@ -26,11 +29,15 @@ from .base import WeightSpec
 class RoutedExperts(base.FeedForward):
     def __init__(self, prefix: str, hidden: int, expert_ff: int, experts: int, top: int, route_scale: float = 1.0, groups: int = 1, groups_keep: int = 1,
                  shared_ff: int = 0, renorm: bool = False, names: tuple = ("router", "e{}", "shared", "gate", "up", "down"), score: str = "softmax",
-                 weight_on: str = "output", correction: str = "", group_top: int = 1):
+                 weight_on: str = "output", correction: str = "", group_top: int = 1, activation: str = "swiglu", router_bias: str = "", shared_gate: str = ""):
         if not 0 < top <= experts or experts % groups or not 0 < groups_keep <= groups:
             raise ValueError(f"top {top} of {experts} experts in {groups} groups of which {groups_keep} stay")
-        if score not in ("softmax", "sigmoid") or weight_on not in ("output", "input"):
-            raise ValueError(f"score {score!r} (softmax, sigmoid) or weight_on {weight_on!r} (output, input) is not known")
+        if activation not in ("swiglu", "relu2"):
+            raise ValueError(f"activation {activation!r} is not known (swiglu, relu2)")
+        self.gated, self.router_bias, self.shared_gate = activation == "swiglu", router_bias, shared_gate if shared_ff else ""
+        self.b_router = None
+        if score not in ops.ROUTE_SCORES or weight_on not in ("output", "input"):
+            raise ValueError(f"score {score!r} ({', '.join(ops.ROUTE_SCORES)}) or weight_on {weight_on!r} (output, input) is not known")
         if not 1 <= group_top <= 4:
             raise ValueError(f"a group's score is the sum of its {group_top} largest scores: 1 to 4 are built")
         self.score, self.weight_on, self.correction, self.group_top = score, weight_on, correction, int(group_top)
@@ -48,32 +55,44 @@ class RoutedExperts(base.FeedForward):
     def weight_specs(self):
         W, F = self.hidden, self.expert_ff
         specs = [WeightSpec(f"{self.prefix}.{self.names[0]}", (self.experts, W))]
+        gate = (0,) if self.gated else ()
         for k in range(self.experts):
-            specs += [WeightSpec(self._expert(k, 0), (F, W)), WeightSpec(self._expert(k, 1), (F, W)), WeightSpec(self._expert(k, 2), (W, F))]
+            specs += [WeightSpec(self._expert(k, i), (F, W)) for i in (*gate, 1)] + [WeightSpec(self._expert(k, 2), (W, F))]
+        if self.router_bias:
+            specs.append(WeightSpec(f"{self.prefix}.{self.router_bias}", (self.experts,), std=0.1))
         if self.correction:
             specs.append(WeightSpec(f"{self.prefix}.{self.correction}", (self.experts,), std=0.1))
         if self.shared_ff:
             S = self.shared_ff
-            specs += [WeightSpec(self._shared(0), (S, W)), WeightSpec(self._shared(1), (S, W)), WeightSpec(self._shared(2), (W, S))]
+            specs += [WeightSpec(self._shared(i), (S, W)) for i in (*gate, 1)] + [WeightSpec(self._shared(2), (W, S))]
+            if self.shared_gate:
+                specs.append(WeightSpec(f"{self.prefix}.{self.names[2]}.{self.shared_gate}", (1, W)))
         return specs
 
     def bind(self, weights, rt):
-        self.w_router = rt.matrix(weights[f"{self.prefix}.{self.names[0]}"])
+        router = weights[f"{self.prefix}.{self.names[0]}"]
+        if self.shared_gate:   # the shared expert's gate is one more row of the router's product
+            router = torch.cat([router, weights[f"{self.prefix}.{self.names[2]}.{self.shared_gate}"]], dim=0)
+        self.w_router = rt.matrix(router)
+        if self.router_bias:
+            self.b_router = rt.vector(weights[f"{self.prefix}.{self.router_bias}"])
         if self.correction:
             self.w_correction = rt.vector(weights[f"{self.prefix}.{self.correction}"])
         # [experts, gate rows then up rows, width] and [experts, width, inner]: one tensor each, so a tile of the grouped product finds its expert by an offset
-        self.w_gu = rt.upload(torch.stack([torch.cat([weights[self._expert(k, 0)], weights[self._expert(k, 1)]], dim=0) for k in range(self.experts)]), rt.act_dtype)
+        front = (0, 1) if self.gated else (1,)
+        self.w_gu = rt.upload(torch.stack([torch.cat([weights[self._expert(k, i)] for i in front], dim=0) for k in range(self.experts)]), rt.act_dtype)
         self.w_d = rt.upload(torch.stack([weights[self._expert(k, 2)] for k in range(self.experts)]), rt.act_dtype)
         if self.shared_ff:
-            self.shared_gu = rt.matrix(torch.cat([weights[self._shared(0)], weights[self._shared(1)]], dim=0))
+            self.shared_gu = rt.matrix(torch.cat([weights[self._shared(i)] for i in front], dim=0))
             self.shared_d = rt.matrix(weights[self._shared(2)])
 
     def forward(self, ctx, h):
         rt, T, E, top = ctx.rt, ctx.n_tokens, self.experts, self.top
         R = T * top
-        logits = rt.linear(h, self.w_router)                     # float32 partial sums [P, T, E]
+        logits = rt.linear(h, self.w_router)                     # float32 partial sums [P, T, E (+ 1)]
         idx, wt = rt.empty((T, top), torch.int32), rt.empty((T, top), torch.float32)
-        ops.moe_route(logits, self.groups, self.groups_keep, top, self.route_scale, self.renorm, idx, wt, self.score, correction=self.w_correction, group_top=self.group_top)
+        ops.moe_route(logits, self.groups, self.groups_keep, top, self.route_scale, self.renorm, idx, wt, self.score, correction=self.w_correction, group_top=self.group_top,
+                      experts=E, logit_bias=self.b_router)
         on_input = self.weight_on == "input"
         offsets, tile_start = rt.empty((E + 1,), torch.int32), rt.empty((E + 1,), torch.int32)
         row_of_pair, token_of_row = rt.empty((R,), torch.int32), rt.empty((R,), torch.int32)
@@ -81,7 +100,7 @@ class RoutedExperts(base.FeedForward):
         bn = G.grouped_token_tile(R, E, self.expert_ff, rt.sm_count)
         act = rt.empty((R, self.expert_ff))
         y = rt.empty((R, self.hidden), torch.float32)
-        if how in ("auto", "tcgen05") and rt.act_dtype == torch.bfloat16 and rt.gemm != "simt" and G.grouped_supported(self.hidden, self.expert_ff, bn):
+        if how in ("auto", "tcgen05") and rt.act_dtype == torch.bfloat16 and rt.gemm != "simt" and G.grouped_supported(self.hidden, self.expert_ff, bn, self.gated):
             # the tcgen05 kernel of the single-matrix products, its tiles taking their expert from the tile table
             ops.moe_sort(idx, E, offsets, tile_start, row_of_pair, token_of_row, tile_rows=bn)
             xs = rt.empty((R, self.hidden))
@@ -89,7 +108,7 @@ class RoutedExperts(base.FeedForward):
                 ops.scatter_scaled_rows(h, row_of_pair, wt, xs)
             else:
                 ops.gather_rows(h, token_of_row, xs)
-            G.gemm_grouped_swiglu(xs, self.w_gu, act, bn, offsets, tile_start, rt.status)
+            (G.gemm_grouped_swiglu if self.gated else G.gemm_grouped_relu2)(xs, self.w_gu, act, bn, offsets, tile_start, rt.status)
             G.gemm_grouped(act, self.w_d, y, bn, offsets, tile_start, rt.status)
         else:
             if how == "tcgen05":
@@ -100,9 +119,12 @@ class RoutedExperts(base.FeedForward):
             if on_input:   # the rows in the experts' order, each times its weight; the product then reads them as they lie
                 src, rows = rt.empty((R, self.hidden)), None
                 ops.scatter_scaled_rows(h, row_of_pair, wt, src)
-            ops.gemm_grouped(src, rows, self.w_gu, act, offsets, tile_start, gated=True, tensor_cores=tc and ops.rows_mma_fits(src, self.w_gu))
+            ops.gemm_grouped(src, rows, self.w_gu, act, offsets, tile_start, gated=self.gated, tensor_cores=tc and ops.rows_mma_fits(src, self.w_gu),
+                             act="none" if self.gated else "relu2")
             ops.gemm_grouped(act, None, self.w_d, y, offsets, tile_start, gated=False, tensor_cores=tc and ops.rows_mma_fits(act, self.w_d))
-        shared = rt.linear(rt.gate_up_act(h, self.shared_gu), self.shared_d) if self.shared_ff else None
+        shared = None
+        if self.shared_ff:
+            shared = rt.linear(rt.gate_up_act(h, self.shared_gu) if self.gated else rt.up_act(h, self.shared_gu, "relu2"), self.shared_d)
         out = rt.empty((1, T, self.hidden), torch.float32)
-        ops.moe_combine(y, row_of_pair, wt, shared, out[0], weighted=not on_input)
+        ops.moe_combine(y, row_of_pair, wt, shared, out[0], weighted=not on_input, gate=(logits, E) if self.shared_gate else None)
         return out

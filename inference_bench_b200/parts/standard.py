@@ -67,29 +67,62 @@ class RMSNorm(base.Norm):
 
 @base.register_norm("layernorm")
 class LayerNorm(base.Norm):
-    """y = w * (x - mean(x)) / sqrt(mean((x - mean)^2) + eps), no bias, float32 arithmetic, fused with the residual add that precedes
-    it. `forward` takes the extras a block may need from that kernel: a per-channel scale and a bias on the contribution it adds, a
+    """y = w * (x - mean(x)) / sqrt(mean((x - mean)^2) + eps) (+ b with `bias`: the tensor of the same name in the bias pattern), float32
+    arithmetic, fused with the residual add that precedes it; a `ScaledDelta` is multiplied by its constant as it is added. `forward` takes the extras a block may need from that kernel: a per-channel scale and a bias on the contribution it adds, a
     copy of the updated stream, and a layout of the normed rows for a convolution over time (`ops.ConvLayout`; the rows then stay
     float32 and keep their place in that layout)."""
 
     takes_layout = True   # `forward` takes the extras named above (what a block with input convolutions asks of its norms)
 
-    def __init__(self, name: str, size: int, eps: float):
-        self.name, self.size, self.eps = name, size, eps
+    takes_scaled_delta = True
+
+    def __init__(self, name: str, size: int, eps: float, bias: Optional[str] = None):
+        """bias: None, or the bias tensor's name as a pattern of the weight's ("{}.b")."""
+        self.name, self.size, self.eps, self.bias_name = name, size, eps, None if bias is None else bias.format(name)
         self.w: Optional[torch.Tensor] = None
+        self.b: Optional[torch.Tensor] = None
 
     def weight_specs(self):
-        return [WeightSpec(self.name, (self.size,), role="norm")]
+        specs = [WeightSpec(self.name, (self.size,), role="norm")]
+        return specs if self.bias_name is None else specs + [WeightSpec(self.bias_name, (self.size,), std=0.1)]
 
     def bind(self, weights, rt):
         self.w = rt.vector(weights[self.name])
+        if self.bias_name is not None:
+            self.b = rt.vector(weights[self.bias_name])
+
+    @staticmethod
+    def _contribution(delta):
+        """(partial sums, constant they are multiplied by)."""
+        return (delta.delta, delta.scale) if isinstance(delta, base.ScaledDelta) else (delta, 1.0)
+
+    @staticmethod
+    def _early(ctx) -> bool:
+        """Whether the next kernels may be scheduled while the norm runs. In a step with prompt portions the product that made the contribution may
+        still be waiting for tensor memory that an attention kernel holds; the next product must not be served before it."""
+        return ctx.fixed_shape or ctx.n_segments == ctx.n_tokens
+
+    def forward_mixes(self, ctx, x, pending, mu, state, out):
+        """The normed rows h of x (after `pending`) as several mixes with the row before: out[m, t] = h_t + (h_(t-1) - h_t) * mu[m]. state (float32
+        [slots, size]) holds every request's last normed row. One kernel where every segment of the step brings one token."""
+        delta, mult = self._contribution(pending)
+        if ctx.fixed_shape or ctx.n_segments == ctx.n_tokens:
+            ops.add_layernorm_mixes_single(x, delta, mult, self.w, self.b, self.eps, mu, state, ctx.seg_slot, out)
+            return
+        h = ctx.rt.empty((ctx.n_tokens, self.size), torch.float32)
+        ops.add_layernorm(x, delta, self.w, h, self.eps, b=self.b, delta_mult=mult, early=self._early(ctx))
+        ops.shift_mixes(h, mu, state, ctx.seg_of_token, ctx.seg_start, ctx.seg_slot, out)
 
     def forward(self, ctx, x, delta, rows=None, delta_scale=None, delta_bias=None, x_copy=None, layout=None):
+        if isinstance(delta, base.ScaledDelta):
+            out = ctx.rt.empty((x.shape[0] if rows is None else rows.shape[0], self.size))
+            ops.add_layernorm(x, delta.delta, self.w, out, self.eps, rows, b=self.b, delta_mult=delta.scale, early=self._early(ctx))
+            return out
         if layout is not None:
             out = ctx.rt.empty((layout.rows(x.shape[0]), self.size), torch.float32)
         else:
             out = ctx.rt.empty((x.shape[0] if rows is None else rows.shape[0], self.size))
-        ops.add_layernorm(x, delta, self.w, out, self.eps, rows, delta_scale, delta_bias, x_copy, layout)
+        ops.add_layernorm(x, delta, self.w, out, self.eps, rows, delta_scale, delta_bias, x_copy, layout, b=self.b)
         return out
 
 
@@ -304,7 +337,7 @@ class SwiGLU(base.FeedForward):
 class DenseXielu(base.FeedForward):
     """down(act(up h)) with the activation xIELU, whose two numbers (p, q) are a tensor of the layer:
     act(z) = softplus(p) z^2 + z / 2 for z > 0, (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 otherwise, in float32 on the product's
-    float32 sums (`Runtime.up_xielu`: in the tensor-core product's epilogue where its k-range is whole)."""
+    float32 sums (`Runtime.up_act`: in the tensor-core product's epilogue where its k-range is whole)."""
 
     def __init__(self, prefix: str, hidden: int, intermediate: int, names: tuple = ("up", "down", "act")):
         self.prefix, self.hidden, self.intermediate, self.names = prefix, hidden, intermediate, tuple(names)
@@ -323,7 +356,7 @@ class DenseXielu(base.FeedForward):
 
     def forward(self, ctx, h, residual=None):
         rt = ctx.rt
-        return rt.linear(rt.up_xielu(h, self.wu, self.pq), self.wd, add_to=residual)
+        return rt.linear(rt.up_act(h, self.wu, "xielu", self.pq), self.wd, add_to=residual)
 
 
 # ------------------------------------------------------------------------------------------ embedding and head
@@ -331,11 +364,15 @@ class DenseXielu(base.FeedForward):
 class TokenEmbedding(base.Embedding):
     """x[t] = float32(E[token_t]) * 1 (crates/kir/src/prims.rs:387)."""
 
-    def __init__(self, name: str, vocab: int, hidden: int, scale: float = 1.0, positions: Optional[str] = None, max_positions: int = 0):
-        """scale: a constant on the token's vector. positions: the name of a table [max_positions, hidden] of learned vectors, one a position,
+    def __init__(self, name: str, vocab: int, hidden: int, scale: float = 1.0, positions: Optional[str] = None, max_positions: int = 0,
+                 norm: Optional[LayerNorm] = None):
+        """norm: a layer norm of the token's vector (with neither a scale nor positions). scale: a constant on the token's vector. positions: the name of a table [max_positions, hidden] of learned vectors, one a position,
         added to it unscaled: x[t] = E[token_t] * scale + P[position_t]."""
         if positions is not None and max_positions <= 0:
             raise ValueError("a table of learned positions needs its number of positions")
+        if norm is not None and (not isinstance(norm, LayerNorm) or scale != 1.0 or positions is not None):
+            raise ValueError("an embedding's norm is a layer norm of the plain token vector")
+        self.norm = norm
         self.name, self.vocab, self.hidden, self.scale, self.positions, self.max_positions = name, vocab, hidden, float(scale), positions, max_positions
         self.table = self.pos_table = None
 
@@ -343,16 +380,20 @@ class TokenEmbedding(base.Embedding):
         specs = [WeightSpec(self.name, (self.vocab, self.hidden))]
         if self.positions is not None:
             specs.append(WeightSpec(self.positions, (self.max_positions, self.hidden)))
-        return specs
+        return specs if self.norm is None else specs + self.norm.weight_specs()
 
     def bind(self, weights, rt):
         self.table = rt.matrix(weights[self.name])
         if self.positions is not None:
             self.pos_table = rt.matrix(weights[self.positions])
+        if self.norm is not None:
+            self.norm.bind(weights, rt)
 
     def forward(self, ctx):
         x = ctx.rt.empty((ctx.n_tokens, self.hidden), torch.float32)
-        if self.pos_table is None and self.scale == 1.0:
+        if self.norm is not None:
+            ops.embed_layernorm(self.table.weight, ctx.token_ids, self.norm.w, self.norm.b, self.norm.eps, x, ctx.rt.status)
+        elif self.pos_table is None and self.scale == 1.0:
             ops.embed(self.table.weight, ctx.token_ids, x, ctx.rt.status)
         elif self.pos_table is None:
             ops.embed(self.table.weight, ctx.token_ids, x, ctx.rt.status)
@@ -368,8 +409,12 @@ class LinearHead(base.Head):
     its own (a tied model ignores lm_head.weight even when the file has it:
     crates/specrt/src/weights.rs:1396-1405)."""
 
-    def __init__(self, name: str, vocab: int, hidden: int, tied_to: Optional[str] = None, scale: float = 1.0):
-        """scale: a constant on the logits."""
+    def __init__(self, name: str, vocab: int, hidden: int, tied_to: Optional[str] = None, scale: float = 1.0,
+                 softcap: Optional[float] = None):
+        """scale: a constant on the logits. softcap c: logits <- c tanh(logits / c), after the scale."""
+        if softcap is not None and not softcap > 0:
+            raise ValueError(f"softcap must be positive, got {softcap}")
+        self.softcap = softcap
         self.name, self.vocab, self.hidden, self.tied_to, self.scale = name, vocab, hidden, tied_to, float(scale)
         self.w = None
 
@@ -385,6 +430,8 @@ class LinearHead(base.Head):
             raise RuntimeError(f"the head's product came back in {out.shape[0]} partial sums although it asked for one")
         if self.scale != 1.0:
             ops.scale_values(out[0], self.scale)
+        if self.softcap is not None:
+            ops.softcap_values(out[0], self.softcap)
         return out[0]
 
 
@@ -393,18 +440,34 @@ class LinearHead(base.Head):
 class PreNormBlock(base.Block):
     """x += mixer(norm(x)); x += feed_forward(norm(x)) (crates/specrt/graphs/decoder.toml:168-303).
     Each residual add is fused into the norm that follows it, so the feed-forward's contribution
-    is handed to the next block (or the final norm) instead of being added here."""
+    is handed to the next block (or the final norm) instead of being added here. residual_mult m: x += m * sublayer (norms that
+    take a `ScaledDelta`). A layer without a feed-forward has the first half only."""
 
-    def __init__(self, mixer_norm, mixer, feed_forward_norm, feed_forward):
+    def __init__(self, mixer_norm, mixer, feed_forward_norm, feed_forward, residual_mult: float = 1.0):
         super().__init__(mixer_norm, mixer, feed_forward_norm, feed_forward)
+        self.residual_mult = float(residual_mult)
+        self.has_ff = not isinstance(feed_forward, NoFeedForward)
+        if self.residual_mult != 1.0 and not all(n.takes_scaled_delta for n in ((mixer_norm, feed_forward_norm) if self.has_ff else (mixer_norm,))):
+            raise ValueError("a residual multiplier needs norms that add a scaled contribution")
+        if mixer.runs_norm and not hasattr(mixer_norm, "forward_mixes"):
+            raise ValueError(f"{type(mixer).__name__} runs its input norm itself, which {type(mixer_norm).__name__} does not allow")
         if getattr(mixer, "bias", False):
             raise ValueError("this arrangement does not add a mixer's output bias")
 
     def forward(self, ctx, x, pending, cache):
-        h = self.mixer_norm.forward(ctx, x, pending)
-        a = self.mixer.forward(ctx, h, cache, residual=x) if self.mixer.adds_to_residual else self.mixer.forward(ctx, h, cache)
+        plain = self.residual_mult == 1.0
+        if self.mixer.runs_norm:
+            a = self.mixer.forward_normed(ctx, self.mixer_norm, x, pending, cache)
+        else:
+            h = self.mixer_norm.forward(ctx, x, pending)
+            a = self.mixer.forward(ctx, h, cache, residual=x) if self.mixer.adds_to_residual and plain else self.mixer.forward(ctx, h, cache)
+        if not plain:
+            a = base.ScaledDelta(a, self.residual_mult)
+        if not self.has_ff:
+            return a
         h = self.feed_forward_norm.forward(ctx, x, a)
-        return self.feed_forward.forward(ctx, h, residual=x) if self.feed_forward.adds_to_residual else self.feed_forward.forward(ctx, h)
+        f = self.feed_forward.forward(ctx, h, residual=x) if self.feed_forward.adds_to_residual and plain else self.feed_forward.forward(ctx, h)
+        return f if plain else base.ScaledDelta(f, self.residual_mult)
 
 
 @base.register_block("outnorm")

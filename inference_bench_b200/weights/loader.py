@@ -103,7 +103,7 @@ class WeightStore:
         info = {n: self.ckpt.tensors[self.names[n]] for n in have}
         missing = sorted(set(wanted) - have)
         self.unexpected = sorted(have - set(wanted) - ignored)
-        wrong = [(n, info[n].shape, wanted[n].shape) for n in sorted(set(wanted) & have) if tuple(info[n].shape) != tuple(wanted[n].shape)]
+        wrong = [(n, info[n].shape, wanted[n].shape) for n in sorted(set(wanted) & have) if not wanted[n].fits(tuple(info[n].shape))]
         other = []
         for n in sorted(set(wanted) & have):
             dt = info[n].dtype

@@ -39,6 +39,8 @@ def random_tensor(spec: WeightSpec, seed: int, device="cpu", dtype=torch.bfloat1
         t = torch.rand(spec.shape, generator=g, device=device, dtype=torch.float32)
     elif spec.role == "log_rate":      # logarithms of decay rates between 0.5 and 8
         t = torch.log(0.5 + 7.5 * torch.rand(spec.shape, generator=g, device=device, dtype=torch.float32))
+    elif spec.role == "decay_bias":    # z of a decay exp(-exp(z)): decays between 0.37 and 0.998
+        t = torch.rand(spec.shape, generator=g, device=device, dtype=torch.float32) * 6.0 - 6.0
     elif spec.role == "matrix":
         t = torch.randn(spec.shape, generator=g, device=device, dtype=torch.float32) * (spec.std if std is None else std)
     else:

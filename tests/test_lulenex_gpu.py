@@ -226,10 +226,10 @@ def test_product_with_xielu_in_its_epilogue(rt16, T, N, K):
         real = L.call
         L.call = lambda name, *a: (called.append(name), real(name, *a))[1]
         try:
-            act = rt16.up_xielu(x, lw, pq_dev)
+            act = rt16.up_act(x, lw, "xielu", pq_dev)
         finally:
             L.call = real
-        if G.xielu_in_epilogue(T, N, K, rt16.sm_count):
+        if G.act_in_epilogue(T, N, K, rt16.sm_count):
             assert called in (["ib_gemm_xielu_tcgen05"], ["ib_gemm_xielu_tcgen05_2cta"])
             assert called == ["ib_gemm_xielu_tcgen05"] if T <= 128 else T < 2048 or called == ["ib_gemm_xielu_tcgen05_2cta"]
         else:
