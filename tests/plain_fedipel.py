@@ -11,6 +11,7 @@ shift, or differential attention over a window and the first tokens; feed-forwar
 """
 from __future__ import annotations
 
+import contextlib
 import math
 
 import torch
@@ -18,8 +19,31 @@ import torch
 F64 = torch.float64
 
 
+ROUND = False     # True (`rounded`): what a bfloat16 engine stores in 16 bits is rounded: the inputs of every matrix product, turned queries and keys, values,
+                  # attention outputs. How far that moves a row says how far an engine's own rounding may.
+
+
 def d(t):
     return t.to(F64)
+
+
+def rnd(t):
+    return t.to(torch.bfloat16).to(F64) if ROUND else t
+
+
+def lin(h, w):
+    """h w^T for a stored matrix [out, in]."""
+    return rnd(h) @ d(w).T
+
+
+@contextlib.contextmanager
+def rounded():
+    global ROUND
+    ROUND = True
+    try:
+        yield
+    finally:
+        ROUND = False
 
 
 # ------------------------------------------------------------------------------------------ small pieces
@@ -77,11 +101,11 @@ def retention(h, w, p, m, eps):
     H, D, V = int(m["heads"]), int(m["dim"]), int(m["vdim"])
     dims, base = int(m["rot"]["dims"]), float(m["rot"]["base"])
     pos = torch.arange(T)
-    q = rotate((h @ d(w[f"{p}.q"]).T).view(T, H, D), pos, dims, base, False)
-    k = rotate((h @ d(w[f"{p}.k"]).T).view(T, H, D), pos, dims, base, False) / math.sqrt(D)
-    v = (h @ d(w[f"{p}.v"]).T).view(T, H, V)
+    q = rotate(lin(h, w[f"{p}.q"]).view(T, H, D), pos, dims, base, False)
+    k = rotate(lin(h, w[f"{p}.k"]).view(T, H, D), pos, dims, base, False) / math.sqrt(D)
+    v = lin(h, w[f"{p}.v"]).view(T, H, V)
     o = rms_unit(retention_scan(q, k, v, [float(x) for x in m["decay"]]), eps).reshape(T, H * V)
-    return (o * silu(h @ d(w[f"{p}.g"]).T)) @ d(w[f"{p}.o"]).T
+    return lin(o * silu(lin(h, w[f"{p}.g"])), w[f"{p}.o"])
 
 
 # ------------------------------------------------------------------------------------------ the recurrence with a decay per channel
@@ -102,11 +126,11 @@ def wkv(h, w, p, m, eps):
     H, D = int(m["heads"]), int(m["dim"])
     before = torch.cat([torch.zeros_like(h[:1]), h[:-1]], 0)
     mix = {s: h + (before - h) * d(w[f"{p}.mu.{s}"]) for s in "rkvgw"}
-    r, k, v = ((mix[s] @ d(w[f"{p}.{s}"]).T).view(T, H, D) for s in "rkv")
-    gate = silu(mix["g"] @ d(w[f"{p}.g"]).T)
-    z = torch.tanh(mix["w"] @ d(w[f"{p}.w1"]).T) @ d(w[f"{p}.w2"]).T + d(w[f"{p}.w0"])
+    r, k, v = (lin(mix[s], w[f"{p}.{s}"]).view(T, H, D) for s in "rkv")
+    gate = silu(lin(mix["g"], w[f"{p}.g"]))
+    z = torch.tanh(lin(mix["w"], w[f"{p}.w1"])) @ d(w[f"{p}.w2"]).T + d(w[f"{p}.w0"])
     o = wkv_scan(r, k, v, torch.exp(-torch.exp(z)).view(T, H, D), d(w[f"{p}.u"]).view(H, D))
-    return (rms_unit(o, eps).reshape(T, H * D) * d(w[f"{p}.norm"]) * gate) @ d(w[f"{p}.o"]).T
+    return lin(rms_unit(o, eps).reshape(T, H * D) * d(w[f"{p}.norm"]) * gate, w[f"{p}.o"])
 
 
 # ------------------------------------------------------------------------------------------ differential attention
@@ -137,35 +161,35 @@ def attention_kv(h, w, p, m):
     """The keys of both maps, turned, [T, G, 2, D], and the values [T, G, V]."""
     T = h.shape[0]
     G, D, V = int(m["kv_heads"]), int(m["dim"]), int(m["vdim"])
-    k = (h @ d(w[f"{p}.k"]).T + d(w[f"{p}.k.b"])).view(T, G * 2, D)
+    k = (lin(h, w[f"{p}.k"]) + d(w[f"{p}.k.b"])).view(T, G * 2, D)
     k = rotate(k, torch.arange(T), int(m["rot"]["dims"]), float(m["rot"]["base"]), True).view(T, G, 2, D)
-    return k, (h @ d(w[f"{p}.v"]).T + d(w[f"{p}.v.b"])).view(T, G, V)
+    return rnd(k), rnd(lin(h, w[f"{p}.v"]) + d(w[f"{p}.v.b"])).view(T, G, V)
 
 
 def diff_attention(h, w, p, m, eps, kv):
     T = h.shape[0]
     H, D, V = int(m["heads"]), int(m["dim"]), int(m["vdim"])
     k, v = kv
-    q = (h @ d(w[f"{p}.q"]).T + d(w[f"{p}.q.b"])).view(T, H * 2, D)
-    q = rotate(q, torch.arange(T), int(m["rot"]["dims"]), float(m["rot"]["base"]), True).view(T, H, 2, D)
+    q = (lin(h, w[f"{p}.q"]) + d(w[f"{p}.q.b"])).view(T, H * 2, D)
+    q = rnd(rotate(q, torch.arange(T), int(m["rot"]["dims"]), float(m["rot"]["base"]), True)).view(T, H, 2, D)
     seen, scale, diff = visible(T, m["mask"]), float(m["scale"]), float(m["diff"])
-    a1, a2 = (masked_attention(q[:, :, i], k[:, :, i], v, seen, scale) for i in (0, 1))
+    a1, a2 = (rnd(masked_attention(q[:, :, i], k[:, :, i], v, seen, scale)) for i in (0, 1))
     o = rms_unit(a1 - diff_lambda(w, p, diff) * a2, eps) * (1.0 - diff)
-    return o.reshape(T, H * V) @ d(w[f"{p}.o"]).T
+    return lin(o.reshape(T, H * V), w[f"{p}.o"])
 
 
 # ------------------------------------------------------------------------------------------ feed-forwards
 def dense_ff(h, w, p):
-    return (silu(h @ d(w[f"{p}.gate"]).T) * (h @ d(w[f"{p}.up"]).T)) @ d(w[f"{p}.down"]).T
+    return lin(silu(lin(h, w[f"{p}.gate"])) * lin(h, w[f"{p}.up"]), w[f"{p}.down"])
 
 
 def relu2_ff(h, w, p):
-    return relu2(h @ d(w[f"{p}.up"]).T) @ d(w[f"{p}.down"]).T
+    return lin(relu2(lin(h, w[f"{p}.up"])), w[f"{p}.down"])
 
 
 def route(h, w, p, top):
     """[T, top] chosen experts (largest logits) and their weights (softmax over the chosen logits)."""
-    z = h @ d(w[f"{p}.router"]).T + d(w[f"{p}.router.b"])
+    z = lin(h, w[f"{p}.router"]) + d(w[f"{p}.router.b"])
     best, idx = torch.topk(z, top, dim=-1)
     return idx, torch.softmax(best, -1)
 
@@ -177,7 +201,7 @@ def experts_ff(h, w, p, f):
         weight = (wt * (idx == e)).sum(-1, keepdim=True)
         out = out + weight * relu2_ff(h, w, f"{p}.e{e}")
     if f.get("shared"):
-        out = out + torch.sigmoid(h @ d(w[f"{p}.shared.sg"]).T) * relu2_ff(h, w, f"{p}.shared")
+        out = out + torch.sigmoid(lin(h, w[f"{p}.shared.sg"])) * relu2_ff(h, w, f"{p}.shared")
     return out
 
 
@@ -211,7 +235,7 @@ def hidden_states(cfg, w, tokens):
 def logits(cfg, w, tokens):
     """Logits at every position of one sequence, float64 [T, vocab]."""
     x = hidden_states(cfg, w, tokens)[-1]
-    z = layer_norm(x, w, "final.norm", float(cfg["norm"]["eps"])) @ d(w["head"]).T
+    z = lin(layer_norm(x, w, "final.norm", float(cfg["norm"]["eps"])), w["head"])
     cap = cfg.get("logit_softcap")
     return z if not cap else float(cap) * torch.tanh(z / float(cap))
 
