@@ -604,6 +604,65 @@ def lulenex_work(z: dict, layers: int, T: int, ctx: int, batch: int) -> tuple:
     return work, lin
 
 
+# Fedipel at layer sizes that resemble small hybrid models: retention with heads of 128 x 128, differential attention with maps of 64 and values of 128
+# over a window and four kept positions, a recurrence with heads of 64 x 64, attention that reads the other attention layer's keys; every feed-forward
+# routed beside a shared expert. Beside it Busadra, the closest design (windowed attention, a matrix-state recurrence, routed experts), at equal
+# width, windows, cache rows, experts and choices.
+FEDIPEL_SIZES = {
+    "small": dict(BUSADRA_SIZES["small"], att_heads=8, att_kv_heads=2, map_dim=64, att_vdim=128, keep=4, wkv_heads=16, wkv_dim=64, decay_rank=64, shared_ff=1024),
+    "mid": dict(BUSADRA_SIZES["mid"], att_heads=16, att_kv_heads=4, map_dim=64, att_vdim=128, keep=4, wkv_heads=32, wkv_dim=64, decay_rank=64, shared_ff=2816),
+}
+DESIGN_KINDS["fedipel"] = {
+    "attention": ["ib_attention_generic", "ib_attention_decode_capped", "ib_attention_decode_stream_capped", "ib_attention_prefill_ws_capped", "ib_attention_decode_maps",
+                  "ib_attention_prefill_maps"],
+    "recurrence": ["ib_recurrence_parts", "ib_recurrence_chunks_finish", "ib_head_norm_gate"],
+    "experts": ["ib_gemm_grouped", "ib_gemm_grouped_mma", "ib_gemm_grouped_tcgen05", "ib_gemm_grouped_relu2_tcgen05", "ib_gather_rows"],
+    "route": ["ib_moe_route", "ib_moe_sort", "ib_moe_combine"],
+    "norm": ["ib_add_layernorm", "ib_add_layernorm_mixes_single", "ib_shift_mixes", "ib_decay_rows", "ib_map_qkv", "ib_diff_combine", "ib_embed_layernorm"],
+    "gemm": LEAVE_OUT["gemm"] + ["ib_gemm_relu2_tcgen05", "ib_gemm_relu2_tcgen05_2cta", "ib_relu2_rows", "ib_gemm_parts_tcgen05"]}
+
+
+def fedipel_config(z: dict, layers: int) -> dict:
+    att = {"heads": z["att_heads"], "kv_heads": z["att_kv_heads"], "dim": z["map_dim"], "vdim": z["att_vdim"], "mask": {"size": z["window"], "keep_first": z["keep"]},
+           "scale": z["map_dim"] ** -0.5, "diff": 0.5, "rot": {"base": 500000.0, "dims": z["map_dim"]}}
+    ret = {"heads": z["rec_heads"], "dim": z["rec_dim"], "vdim": z["rec_vdim"], "rot": {"base": 10000.0, "dims": z["rec_dim"]},
+           "decay": [1.0 - 0.5 ** (5 + 8 * h / z["rec_heads"]) for h in range(z["rec_heads"])]}
+    wkv = {"heads": z["wkv_heads"], "dim": z["wkv_dim"]}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]}, "shared": {"ff": z["shared_ff"]}}
+    four = [("retention", ret), ("attention", att), ("wkv", wkv), ("attention", None)]
+    ls = []
+    for i in range(layers):
+        t, m = four[i % 4]
+        ls.append({"type": t, "mixer": dict(att, kv_from=i - 2) if m is None else m, "mlp": moe})
+    return {"architecture": "Fedipel", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "residual_mult": 0.5, "logit_softcap": 30.0, "layers": ls}
+
+
+def fedipel_work(z: dict, layers: int, T: int, ctx: int, batch: int) -> tuple:
+    """As `lulenex_work`: the recurrences are float32 FMAs, their floors the bytes they must move."""
+    n_ret, n_wkv, n_own, n_read = (sum(1 for i in range(layers) if i % 4 == k) for k in (0, 2, 1, 3))
+    n_att = n_own + n_read
+    W, H, G, D, V = z["width"], z["att_heads"], z["att_kv_heads"], z["map_dim"], z["att_vdim"]
+    rh, rd, rv, C, wd = z["rec_heads"], z["rec_dim"], z["rec_vdim"], z["wkv_heads"] * z["wkv_dim"], z["wkv_dim"]
+    pairs = sum(min(t + 1, z["window"] + z["keep"]) for t in range(T))
+    seen = min(ctx, z["window"] + z["keep"])
+    ret_row = rh * (4.0 * (2 * rd + rv) + 4.0 * rv + 10.0 * rv)        # q, k, v in; o out; o and the gate in, the gated norm out
+    wkv_row = C * (4.0 * 4 + 4.0 + 10.0)                                 # r, k, v and the decays in; o out; o and the gate in, the gated norm out
+    kv_row = G * (2 * D + V)
+    norm_row = layers * W * 2 * (4.0 * 3 + 2) + n_wkv * (W * (4.0 + 10) + 4.0 * (C + z["decay_rank"])) + n_att * (H * 2 * D * (4.0 + 4) + H * V * 6.0) + n_own * kv_row * 6.0
+    lin = n_ret * (2 * rh * rd + 3 * rh * rv) * W + n_wkv * (5 * C + z["decay_rank"]) * W + n_att * (2 * H * D + H * V) * W + n_own * kv_row * W + \
+        layers * (z["experts"] + 1 + 2 * z["shared_ff"]) * W + z["vocab"] * W
+    att_flops = 2.0 * 2 * H * (D + V)                                    # per (query, key): two maps, a product of D and one of V each
+    work = {
+        "prefill": {"attention": {"flops": n_att * att_flops * pairs}, "recurrence": {"flops": 0.0, "bytes": T * (n_ret * ret_row + n_wkv * wkv_row)},
+                    "experts": {"flops": layers * 2.0 * T * z["top"] * 2 * z["expert_ff"] * W}, "norm": {"flops": 0.0, "bytes": T * norm_row}},
+        "decode": {"attention": {"flops": n_att * att_flops * batch * seen, "bytes": n_att * 2.0 * batch * seen * kv_row},
+                   "recurrence": {"flops": 0.0, "bytes": batch * (n_ret * (ret_row + rh * 8.0 * rd * rv) + n_wkv * (wkv_row + 8.0 * C * wd))},
+                   "experts": {"flops": layers * 2.0 * batch * z["top"] * 2 * z["expert_ff"] * W, "bytes": layers * 2.0 * min(batch * z["top"], z["experts"]) * 2 * z["expert_ff"] * W},
+                   "norm": {"flops": 0.0, "bytes": batch * norm_row}},
+    }
+    return work, lin
+
+
 def kernel_times(engine, entries) -> dict:
     """Milliseconds per library entry point in one step run outside a graph: every call stands between two CUDA events, and a
     long idle kernel goes first so that the whole step is queued before its first kernel starts (the events then measure the
@@ -695,7 +754,7 @@ def run_design(args) -> dict:
     layers = args.layers or 4
     steps, warmup = min(args.steps, 32), max(args.warmup, 3)
     out = {"design": args.design, "layers": layers, "peaks": pk_src, "sizes": {}}
-    sizes = {"busadra": BUSADRA_SIZES, "lulenex": LULENEX_SIZES, "ditalorn": DITALORN_SIZES}.get(args.design, DESIGN_SIZES)
+    sizes = {"busadra": BUSADRA_SIZES, "lulenex": LULENEX_SIZES, "ditalorn": DITALORN_SIZES, "fedipel": FEDIPEL_SIZES}.get(args.design, DESIGN_SIZES)
     for name in (args.size.split(",") if args.size else list(sizes)):
         z = sizes[name] if name in sizes or args.design != "lulenex" else LULENEX_EXTRA_SIZES[name]
         report = {}
@@ -705,6 +764,9 @@ def run_design(args) -> dict:
         elif args.design == "busadra":
             zb = z
             pair = (("busadra", busadra_config(z, layers)), ("qwen3", qwen3_like_busadra(z, layers)))
+        elif args.design == "fedipel":
+            zb = z
+            pair = (("fedipel", fedipel_config(z, layers)), ("busadra", busadra_config(z, layers)))
         elif args.design == "ditalorn":
             pair = (("ditalorn", ditalorn_config(z, layers)), ("zabonex", zabonex_config(z, layers)))
         else:
@@ -719,6 +781,8 @@ def run_design(args) -> dict:
                     3 * z["dense_ff"] * z["width"] + (layers - 1) * (3 * z["shared_ff"] + z["experts"]) * z["width"] + vocab * z["width"]
             elif arch == "lulenex":
                 work, lin = lulenex_work(z, layers, PROMPT, PROMPT, 8)
+            elif arch == "fedipel":
+                work, lin = fedipel_work(z, layers, PROMPT, PROMPT, 8)
             elif arch == "ditalorn":
                 work, lin = ditalorn_work(z, layers, PROMPT, PROMPT, 8)
             elif arch == "busadra":
@@ -767,6 +831,8 @@ def run_design(args) -> dict:
                 if k:
                     kinds[kind] = k
             r["kinds"] = kinds
+            if args.kernels:
+                r["kernels"] = {phase: {n: {"ms": t[0], "calls": t[1]} for n, t in sorted(times.items(), key=lambda kv: -kv[1][0])} for phase, times in (("prefill", times_p), ("decode_b8", times_d))}
             r["kernels_alone_ms"] = {"prefill": sum(t[0] for t in times_p.values()), "decode_b8": sum(t[0] for t in times_d.values())}
             report[arch] = r
             del engine
@@ -791,9 +857,10 @@ def main() -> int:
     ap.add_argument("--leave-out", default="", help="with --only decode or prefill: also time the step without each of these kinds of kernel (comma separated; "
                     "a+b leaves both out): " + ", ".join(sorted(LEAVE_OUT)))
     ap.add_argument("--only", default="", choices=["", "prefill", "decode", "mixed"], help="run one part alone (for profiling); prints a short report")
-    ap.add_argument("--design", default="", choices=["", "zabonex", "busadra", "lulenex", "ditalorn"],
-                    help="measure another design beside the closest existing one at equal size (Qwen3; for lulenex, Busadra; for ditalorn, Zabonex) instead of the benchmark (prints its own report)")
-    ap.add_argument("--size", default="", help="with --design: which of its sizes (comma separated; default all): " + ", ".join(DESIGN_SIZES) + " (zabonex); " + ", ".join(BUSADRA_SIZES) + " (busadra); " + ", ".join(LULENEX_SIZES) + " (lulenex); " + ", ".join(DITALORN_SIZES) + " (ditalorn)")
+    ap.add_argument("--design", default="", choices=["", "zabonex", "busadra", "lulenex", "ditalorn", "fedipel"],
+                    help="measure another design beside the closest existing one at equal size (Qwen3; for lulenex and fedipel, Busadra; for ditalorn, Zabonex) instead of the benchmark (prints its own report)")
+    ap.add_argument("--size", default="", help="with --design: which of its sizes (comma separated; default all): " + ", ".join(DESIGN_SIZES) + " (zabonex); " + ", ".join(BUSADRA_SIZES) + " (busadra); " + ", ".join(LULENEX_SIZES) + " (lulenex); " + ", ".join(DITALORN_SIZES) + " (ditalorn); " + ", ".join(FEDIPEL_SIZES) + " (fedipel)")
+    ap.add_argument("--kernels", action="store_true", help="with --design: also list every library entry point's time in one prefill and one decode step")
     args = ap.parse_args()
     if args.design:
         print(json.dumps(run_design(args)))

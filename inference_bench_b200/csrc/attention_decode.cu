@@ -286,31 +286,20 @@ __global__ void __launch_bounds__(kWarps * 32)
 // lane-th slice for four values of the head, and the lanes are added in order through shared memory.
 constexpr int kCombineThreads = 256;
 
+// What the combine kernels share: the merged output of one (token, head) for the values 4 * dq .. of the threads with sg == 0, and the scratch it
+// needs. Every thread of the CTA calls it; the scratch may be used again after it returns.
 template <int HD>
-__global__ void __launch_bounds__(kCombineThreads)
-    decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const int* __restrict__ dec_tokens,
-                          const int* __restrict__ positions, int window, __nv_bfloat16* __restrict__ out, int heads, int max_slices,
-                          int tiles_per_slice, unsigned* __restrict__ status, int sink, IbAttnTail tail, int keep) {
-  // sink: one more term of score 0 (or tail.sink_values[head]) and no value in the denominator; tail: factors on the output and its row length
-  constexpr int DQ = HD / 4;
-  constexpr int SG = kCombineThreads / DQ;
-  __shared__ float4 o_red[SG][DQ];
-  __shared__ float m_red[SG], l_red[SG];
-  ib::pdl_launch_dependents();
-  const int h = blockIdx.x, item = blockIdx.y;
-  const int t = dec_tokens[item];
-  const int pos = positions[t];
-  int lo, tile_lo, tps, win_tile, pre_shift;
-  slice_plan(pos, window, keep, max_slices, tiles_per_slice, lo, tile_lo, tps, win_tile, pre_shift);
-  const int s_begin = keep > 0 ? 0 : (lo / kTile - tile_lo) / tps;
-  int s_end = (pos / kTile - tile_lo) / tps + 1;
-  if (s_end > max_slices) {   // the caller's max_slices does not cover this position: nothing beyond the scratch is read, and the status says so
-    if (threadIdx.x == 0) atomicOr(status, IB_ERR_INTERNAL);
-    s_end = max_slices;
-  }
-  const size_t slot0 = ((size_t)item * heads + h) * max_slices;
+struct CombineScratch {
+  static constexpr int DQ = HD / 4, SG = kCombineThreads / DQ;
+  float4 o_red[SG][DQ];
+  float m_red[SG], l_red[SG];
+};
+
+template <int HD>
+__device__ __forceinline__ void combine_head(CombineScratch<HD>& sc, const float* __restrict__ part_o, const float* __restrict__ part_ml, size_t slot0, int s_begin, int s_end,
+                                             int sink, float sink_log2e, float4& O, float& Lsum) {
+  constexpr int DQ = HD / 4, SG = kCombineThreads / DQ;
   const int sg = threadIdx.x / DQ, dq = threadIdx.x % DQ;
-  ib::pdl_wait();
   // the thread's first slice (with up to SG slices, its only one) is requested whole before anything is waited for:
   // one trip to memory instead of two, one after the other
   const int s0 = s_begin + sg;
@@ -324,11 +313,11 @@ __global__ void __launch_bounds__(kCombineThreads)
   }
   float mx = m0;
   for (int s = s0 + SG; s < s_end; s += SG) mx = fmaxf(mx, part_ml[(slot0 + s) * 2]);
-  if (dq == 0) m_red[sg] = mx;
+  if (dq == 0) sc.m_red[sg] = mx;
   __syncthreads();
   float M = -INFINITY;
 #pragma unroll
-  for (int i = 0; i < SG; i++) M = fmaxf(M, m_red[i]);
+  for (int i = 0; i < SG; i++) M = fmaxf(M, sc.m_red[i]);
   float Lp = 0.f;
   float4 Op = make_float4(0.f, 0.f, 0.f, 0.f);
   if (have) {
@@ -345,29 +334,90 @@ __global__ void __launch_bounds__(kCombineThreads)
     Op.z += v.z * f;
     Op.w += v.w * f;
   }
-  o_red[sg][dq] = Op;
-  if (dq == 0) l_red[sg] = Lp;
+  sc.o_red[sg][dq] = Op;
+  if (dq == 0) sc.l_red[sg] = Lp;
   __syncthreads();
+  Lsum = 0.f;
+  O = make_float4(0.f, 0.f, 0.f, 0.f);
   if (sg == 0) {
-    float Lsum = 0.f;
-    float4 O = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int i = 0; i < SG; i++) {
-      Lsum += l_red[i];
-      const float4 v = o_red[i][dq];
+      Lsum += sc.l_red[i];
+      const float4 v = sc.o_red[i][dq];
       O.x += v.x;
       O.y += v.y;
       O.z += v.z;
       O.w += v.w;
     }
-    if (sink && M > -INFINITY) Lsum += exp2f((tail.sink_values ? tail.sink_values[h] * 1.4426950408889634f : 0.f) - M);
+    if (sink && M > -INFINITY) Lsum += exp2f(sink_log2e - M);
     if (!(Lsum > 0.f)) {
       O = make_float4(0.f, 0.f, 0.f, 0.f);
       Lsum = 1.f;
     }
+  }
+}
+
+// The slices of a decoded token that hold visible keys; false bits in the status when max_slices does not cover them.
+__device__ __forceinline__ void combine_range(int pos, int window, int keep, int max_slices, int tiles_per_slice, unsigned* status, int& s_begin, int& s_end) {
+  int lo, tile_lo, tps, win_tile, pre_shift;
+  slice_plan(pos, window, keep, max_slices, tiles_per_slice, lo, tile_lo, tps, win_tile, pre_shift);
+  s_begin = keep > 0 ? 0 : (lo / kTile - tile_lo) / tps;
+  s_end = (pos / kTile - tile_lo) / tps + 1;
+  if (s_end > max_slices) {   // the caller's max_slices does not cover this position: nothing beyond the scratch is read, and the status says so
+    if (threadIdx.x == 0) atomicOr(status, IB_ERR_INTERNAL);
+    s_end = max_slices;
+  }
+}
+
+template <int HD>
+__global__ void __launch_bounds__(kCombineThreads)
+    decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const int* __restrict__ dec_tokens,
+                          const int* __restrict__ positions, int window, __nv_bfloat16* __restrict__ out, int heads, int max_slices,
+                          int tiles_per_slice, unsigned* __restrict__ status, int sink, IbAttnTail tail, int keep) {
+  // sink: one more term of score 0 (or tail.sink_values[head]) and no value in the denominator; tail: factors on the output and its row length
+  __shared__ CombineScratch<HD> sc;
+  ib::pdl_launch_dependents();
+  const int h = blockIdx.x, item = blockIdx.y;
+  const int t = dec_tokens[item];
+  int s_begin, s_end;
+  combine_range(positions[t], window, keep, max_slices, tiles_per_slice, status, s_begin, s_end);
+  ib::pdl_wait();
+  float4 O;
+  float Lsum;
+  combine_head<HD>(sc, part_o, part_ml, ((size_t)item * heads + h) * max_slices, s_begin, s_end, sink, tail.sink_values ? tail.sink_values[h] * 1.4426950408889634f : 0.f, O, Lsum);
+  if ((int)threadIdx.x < HD / 4) {
     if (tail.gate || tail.out_scale != 0.f) Lsum /= ib::tail_factor(tail, t, h);
     uint2 packed = make_uint2(mt::pack_bf16(O.x / Lsum, O.y / Lsum), mt::pack_bf16(O.z / Lsum, O.w / Lsum));
-    *(uint2*)&out[(size_t)t * (tail.out_row ? tail.out_row : heads * HD) + h * HD + 4 * dq] = packed;
+    *(uint2*)&out[(size_t)t * (tail.out_row ? tail.out_row : heads * HD) + h * HD + 4 * threadIdx.x] = packed;
+  }
+}
+
+// The same for heads that come in pairs of score maps (query heads 2h and 2h + 1): out[t][h] = factor * u / sqrt(mean(u^2) + eps) with
+// u = o_2h - lambda * o_(2h+1), in float32 up to the store.
+template <int HD>
+__global__ void __launch_bounds__(kCombineThreads)
+    decode_combine_diff_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const int* __restrict__ dec_tokens,
+                               const int* __restrict__ positions, int window, __nv_bfloat16* __restrict__ out, int heads, int max_slices,
+                               int tiles_per_slice, unsigned* __restrict__ status, IbAttnTail tail, int keep) {
+  __shared__ CombineScratch<HD> sc[2];
+  ib::pdl_launch_dependents();
+  const int h = blockIdx.x, item = blockIdx.y;
+  const int t = dec_tokens[item];
+  int s_begin, s_end;
+  combine_range(positions[t], window, keep, max_slices, tiles_per_slice, status, s_begin, s_end);
+  ib::pdl_wait();
+  float4 a, b;
+  float la, lb;
+  const size_t slot0 = ((size_t)item * heads + 2 * h) * max_slices;
+  combine_head<HD>(sc[0], part_o, part_ml, slot0, s_begin, s_end, 0, 0.f, a, la);
+  combine_head<HD>(sc[1], part_o, part_ml, slot0 + max_slices, s_begin, s_end, 0, 0.f, b, lb);
+  if (threadIdx.x < 32) {   // the HD / 4 (at most 32) threads that hold the head; a lane beyond them adds nothing
+    const bool mine = (int)threadIdx.x < HD / 4;
+    const float ia = mine ? 1.f / la : 0.f, ib_ = mine ? tail.diff_lambda / lb : 0.f;
+    const float4 u = mine ? make_float4(a.x * ia - b.x * ib_, a.y * ia - b.y * ib_, a.z * ia - b.z * ib_, a.w * ia - b.w * ib_) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float ss = ib::warp_sum(u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w);
+    const float f = tail.diff_factor / sqrtf(ss / (float)HD + tail.diff_eps);
+    if (mine) *(uint2*)&out[((size_t)t * (heads / 2) + h) * HD + 4 * threadIdx.x] = make_uint2(mt::pack_bf16(u.x * f, u.y * f), mt::pack_bf16(u.z * f, u.w * f));
   }
 }
 
@@ -902,8 +952,12 @@ int launch_stream(const void* q, const RawQkv* raw, const IbKvView* kv, const in
              positions, seg_of_token, window, scale_log2e, part_o, part_ml, heads, n_dec, max_slices, tiles_per_slice, merge_cols,
              *kv_map, view_row0, ib_wait_limit_ns(), status, cap_pre, keep);
   IB_CHECK_LAUNCH("attention_decode_stream split");
-  ib::launch(decode_combine_kernel<HD>, dim3(heads, n_dec), kCombineThreads, 0, stream, part_o, part_ml, dec_tokens, positions, window, (__nv_bfloat16*)out, heads,
-             max_slices, tiles_per_slice, status, sink, tail, keep);
+  if (tail.diff)
+    ib::launch(decode_combine_diff_kernel<HD>, dim3(heads / 2, n_dec), kCombineThreads, 0, stream, part_o, part_ml, dec_tokens, positions, window, (__nv_bfloat16*)out, heads,
+               max_slices, tiles_per_slice, status, tail, keep);
+  else
+    ib::launch(decode_combine_kernel<HD>, dim3(heads, n_dec), kCombineThreads, 0, stream, part_o, part_ml, dec_tokens, positions, window, (__nv_bfloat16*)out, heads,
+               max_slices, tiles_per_slice, status, sink, tail, keep);
   IB_CHECK_LAUNCH("attention_decode_stream combine");
   return 0;
 }
@@ -925,8 +979,12 @@ int launch(const void* q, const IbKvView* kv, const int* dec_tokens, int n_dec, 
   ib::launch(decode_split_kernel<HD>, grid, kWarps * 32, smem, stream, (const __nv_bfloat16*)q, *kv, dec_tokens, positions, seg_of_token, window,
              scale_log2e, part_o, part_ml, heads, max_slices, tiles_per_slice, status, cap_pre, keep);
   IB_CHECK_LAUNCH("attention_decode split");
-  ib::launch(decode_combine_kernel<HD>, dim3(heads, n_dec), kCombineThreads, 0, stream, part_o, part_ml, dec_tokens, positions, window, (__nv_bfloat16*)out, heads,
-             max_slices, tiles_per_slice, status, sink, tail, keep);
+  if (tail.diff)
+    ib::launch(decode_combine_diff_kernel<HD>, dim3(heads / 2, n_dec), kCombineThreads, 0, stream, part_o, part_ml, dec_tokens, positions, window, (__nv_bfloat16*)out, heads,
+               max_slices, tiles_per_slice, status, tail, keep);
+  else
+    ib::launch(decode_combine_kernel<HD>, dim3(heads, n_dec), kCombineThreads, 0, stream, part_o, part_ml, dec_tokens, positions, window, (__nv_bfloat16*)out, heads,
+               max_slices, tiles_per_slice, status, sink, tail, keep);
   IB_CHECK_LAUNCH("attention_decode combine");
   return 0;
 }
@@ -966,6 +1024,10 @@ namespace {
 // The tail as the kernels take it (null: all zero), or false with the error set.
 bool read_tail(const char* who, const IbAttnTail* in, int sink, int heads, const IbKvView* kv, IbAttnTail& tail) {
   tail = in ? *in : IbAttnTail{};
+  if (tail.diff && (sink || tail.gate || tail.out_scale != 0.f || tail.out_row || heads % 2)) {
+    ib_set_error("%s: the difference of two maps takes an even number of heads and no sink, gate, scale or output row of its own", who);
+    return false;
+  }
   if ((!tail.sink_values || sink) && (tail.out_row == 0 || (kv && tail.out_row >= heads * kv->head_dim && tail.out_row % 4 == 0)) &&
       (!tail.gate || (tail.gate_parts >= 1 && tail.gate_row >= heads)))
     return true;

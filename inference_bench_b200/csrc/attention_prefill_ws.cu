@@ -422,6 +422,7 @@ extern "C" int ib_attention_prefill_ws_capped(const void* q, const IbKvView* kv,
   if (n_tiles == 0) return 0;
   IB_CHECK_ARG(keep >= 0 && (keep == 0 || window > 0), "attention_prefill_ws: %d kept positions need a window", keep);
   const IbAttnTail tail = tail_in ? *tail_in : IbAttnTail{};
+  IB_CHECK_ARG(!tail.diff, "attention_prefill_ws: the difference of two maps is not taken here");
   IB_CHECK_ARG((!tail.sink_values || sink) && (tail.out_row == 0 || (tail.out_row >= heads * (kv ? kv->head_dim : 0) && tail.out_row % 8 == 0)) &&
                    (!tail.gate || (tail.gate_parts >= 1 && tail.gate_row >= heads)),
                "attention_prefill_ws: sink scores without a sink, an output row of %d (a multiple of 8 that holds the heads), or a gate of %d parts and rows of %d",

@@ -337,8 +337,18 @@ __global__ void __launch_bounds__(256) decay_rows_kernel(const float* __restrict
   float acc[TT];
 #pragma unroll
   for (int tt = 0; tt < TT; tt++) acc[tt] = 0.f;
-#pragma unroll 4
-  for (int j = 0; j < rank; j++) {
+  constexpr int U = TT == 1 ? 16 : 8;   // rows of w2 requested before the first is used
+  int j = 0;
+  for (; j + U <= rank; j += U) {
+    float w[U];
+#pragma unroll
+    for (int e = 0; e < U; e++) w[e] = w2[(size_t)(j + e) * C + c];
+#pragma unroll
+    for (int e = 0; e < U; e++)
+#pragma unroll
+      for (int tt = 0; tt < TT; tt++) acc[tt] = __fmaf_rn(w[e], th[(j + e) * TT + tt], acc[tt]);
+  }
+  for (; j < rank; j++) {
     const float w = w2[(size_t)j * C + c];
 #pragma unroll
     for (int tt = 0; tt < TT; tt++) acc[tt] = __fmaf_rn(w, th[j * TT + tt], acc[tt]);

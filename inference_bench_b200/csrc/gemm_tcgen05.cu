@@ -50,7 +50,9 @@ template <int BN, int MT, int EPI>
 __global__ void __launch_bounds__(kThreads, 1)
     gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_x, void* __restrict__ out_, int T,
                         int N, int K, int ktiles_per_split, int second_off, unsigned long long wait_ns, int starve, unsigned* __restrict__ status,
-                        const int* __restrict__ grp_offsets, const int* __restrict__ grp_tiles, int n_groups, int grp_w_rows, const float* __restrict__ act_pq) {
+                        const int* __restrict__ grp_offsets, const int* __restrict__ grp_tiles, int n_groups, int grp_w_rows, const float* __restrict__ act_pq, int part_rows) {
+  // part_rows > 0: x holds parts of that many rows each, one after the other, and part i goes through matrix i (rows i * grp_w_rows .. of w); a
+  // tile of rows belongs to one part.
   // grp_offsets != nullptr: the rows of x are regrouped (rows grp_offsets[e] .. grp_offsets[e + 1] belong to group e, whose matrix is rows
   // e * grp_w_rows .. of w) and blockIdx.x counts token tiles over all groups: grp_tiles[e] is the first tile of group e, grp_tiles[n_groups]
   // their number (the grid is an upper bound; the CTAs beyond it leave at once). A tile never crosses a group's end: rows past it are
@@ -87,6 +89,12 @@ __global__ void __launch_bounds__(kThreads, 1)
     t0 = grp_offsets[lo] + (b - grp_tiles[lo]) * BN;
     t_end = grp_offsets[lo + 1];
     w_row0 = lo * grp_w_rows;
+  }
+  if (part_rows > 0) {
+    const int per = (part_rows + BN - 1) / BN, part = blockIdx.x / per;
+    t0 = part * part_rows + (blockIdx.x - part * per) * BN;
+    t_end = (part + 1) * part_rows;
+    w_row0 = part * grp_w_rows;
   }
   const int total_kt = (K + BK - 1) / BK;
   const int kt_begin = split * ktiles_per_split;
@@ -313,6 +321,7 @@ struct Groups {   // regrouped rows (see the kernel): nullptr offsets = one matr
   const int* offsets = nullptr;
   const int* tiles = nullptr;
   int n = 0, w_rows = 0;
+  int part_rows = 0;               // equal parts instead of groups: rows of a part
 };
 
 template <int BN, int MT, int EPI>
@@ -326,10 +335,10 @@ int launch(const CUtensorMap& tw, const CUtensorMap& tx, void* out, int T, int N
     configured = true;
   }
   const int cols_per_cta = EPI == EPI_SWIGLU_HALF ? BM / 2 : EPI == EPI_SWIGLU ? BM : BM * MT;
-  dim3 grid(grp.offsets ? T / BN + grp.n : (T + BN - 1) / BN, (N + cols_per_cta - 1) / cols_per_cta, splits);
+  dim3 grid(grp.offsets ? T / BN + grp.n : grp.part_rows ? grp.n * ((grp.part_rows + BN - 1) / BN) : (T + BN - 1) / BN, (N + cols_per_cta - 1) / cols_per_cta, splits);
   IB_CHECK_ARG(grid.y <= 65535, "gemm_tcgen05: N=%d gives more than 65535 row blocks", N);
   ib::launch(gemm_tcgen05_kernel<BN, MT, EPI>, grid, kThreads, TL::kSmemBytes, stream, tw, tx, out, T, N, K, kt_per_split, second_off, ib_wait_limit_ns(), starve, status,
-             grp.offsets, grp.tiles, grp.n, grp.w_rows, act_pq);
+             grp.offsets, grp.tiles, grp.n, grp.w_rows, act_pq, grp.part_rows);
   IB_CHECK_LAUNCH("gemm_tcgen05");
   return 0;
 }
@@ -490,6 +499,29 @@ extern "C" int ib_gemm_grouped_tcgen05(const void* x, const void* w, float* out,
     case 128: return launch<128, 1, EPI_STORE>(tw, tx, out, R, N, K, 1, total_kt, 0, status, stream, 0, g);
     case 256: return launch<256, 1, EPI_STORE>(tw, tx, out, R, N, K, 1, total_kt, 0, status, stream, 0, g);
     default: return ib_set_error("gemm_grouped_tcgen05: token tile %d is not one of 16, 32, 64, 128, 256", bn);
+  }
+}
+
+// Several products of one shape in one launch: x [parts * T, K] (part i's rows follow part i - 1's), w [parts, N, K], out [splits, parts * T, N]
+// float32 partial sums. bn: 16, 32, 64 or 128 tokens per CTA.
+extern "C" int ib_gemm_parts_tcgen05(const void* x, const void* w, float* out, int parts, int T, int N, int K, int bn, int splits, unsigned* status, cudaStream_t stream) {
+  if (T == 0 || N == 0 || parts == 0) return 0;
+  if (check_common("gemm_parts_tcgen05", x, w, T, N, K, bn)) return 1;
+  const int total_kt = (K + BK - 1) / BK;
+  IB_CHECK_ARG(parts > 0 && splits >= 1 && splits <= total_kt && splits <= 65535, "gemm_parts_tcgen05: %d parts, %d splits for %d k-tiles", parts, splits, total_kt);
+  const int per = (total_kt + splits - 1) / splits;
+  IB_CHECK_ARG((splits - 1) * per < total_kt, "gemm_parts_tcgen05: %d splits of %d k-tiles leave one empty (%d k-tiles)", splits, per, total_kt);
+  CUtensorMap tw, tx;
+  if (make_tmap(&tw, w, parts * N, K, BM)) return 1;
+  if (make_tmap(&tx, x, parts * T, K, bn)) return 1;
+  Groups g;
+  g.n = parts, g.w_rows = N, g.part_rows = T;
+  switch (bn) {
+    case 16: return launch<16, 1, EPI_STORE>(tw, tx, out, parts * T, N, K, splits, per, 0, status, stream, 0, g);
+    case 32: return launch<32, 1, EPI_STORE>(tw, tx, out, parts * T, N, K, splits, per, 0, status, stream, 0, g);
+    case 64: return launch<64, 1, EPI_STORE>(tw, tx, out, parts * T, N, K, splits, per, 0, status, stream, 0, g);
+    case 128: return launch<128, 1, EPI_STORE>(tw, tx, out, parts * T, N, K, splits, per, 0, status, stream, 0, g);
+    default: return ib_set_error("gemm_parts_tcgen05: token tile %d is not one of 16, 32, 64, 128", bn);
   }
 }
 

@@ -34,6 +34,10 @@ struct IbAttnTail {
   long long gate_stride;     // elements between consecutive parts
   float out_scale;           // 0 stands for 1
   int out_row;               // elements per output row; 0 stands for heads * head_dim
+  int diff;                  // 1 (decoded tokens only): query heads 2h and 2h + 1 are two maps of head h, whose output is diff_factor * u / sqrt(mean(u^2) +
+  float diff_lambda;         //   diff_eps) with u the first map's output minus diff_lambda times the second's; the output has heads / 2 heads
+  float diff_eps;
+  float diff_factor;
 };
 
 namespace ib {

@@ -10,6 +10,8 @@
 //    the chosen logits alone.
 //  * moe_sort: counts the (token, choice) pairs of every expert, lays the experts' rows out one after the other
 //    (offsets[e] .. offsets[e + 1]) and gives every pair a row of its expert's range; tile_start[e] is the first tile of expert e.
+//  * moe_route_sort: both in one kernel for a step of few tokens. Experts that every token uses (a shared expert cut into blocks of the routed
+//    experts' inner size) may stand behind the routed ones as further choices.
 //  * gemm_grouped: out[r] = W[e(r)] x[src(r)] for every regrouped row r: a 64 x 64 tile belongs to one expert; float32
 //    FMA chains per output (a row's result does not depend on its place among the rows). With `gated`, W holds gate
 //    rows then up rows and the output is silu(gate) * up. With `relu2` the output is the square of max(product, 0).
@@ -34,33 +36,40 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
   }
 }
 
-__global__ void moe_route_kernel(const float* __restrict__ logits, int P, size_t stride_p, int T, int E, int n_groups, int keep, int top, float route_scale,
-                                 int renorm, int* __restrict__ idx_out, float* __restrict__ wt_out, int score, const float* __restrict__ correction,
-                                 int group_top, int row, const float* __restrict__ logit_bias) {
-  // row: entries of a row of logits (the experts' are its first E). logit_bias: float32 [E] added to the logits, or null.
-  // correction: a number per expert added to its score for the choice (of groups and of experts) and left out of the weights, or null.
-  // group_top: a group's score is the sum of its `group_top` largest choice scores (1: its largest).
-  // Choice scores may be negative: what cannot be chosen counts as minus infinity.
-  extern __shared__ float sm[];   // per warp: E scores, E choice scores, then n_groups group scores
-  ib::pdl_launch_dependents();
-  ib::pdl_wait();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int t = blockIdx.x * kRouteWarps + warp;
-  if (t >= T) return;
-  float* s = sm + (size_t)warp * (2 * E + n_groups);
+struct RouteArgs {
+  const float* logits;       // float32 partial sums [P][T][row], the experts' are a row's first E
+  int P;
+  size_t stride_p;
+  int T, E, row, n_groups, keep, top;
+  float route_scale;
+  int renorm, score;
+  const float* correction;   // a number per expert added to its score for the choice (of groups and of experts) and left out of the weights, or null
+  const float* logit_bias;   // float32 [E] added to the logits, or null
+  int group_top;             // a group's score is the sum of its `group_top` largest choice scores (1: its largest)
+  int always;                // experts E .. E + always - 1 that every token uses as well: the last entries of its row of choices, weighted by
+  int gate_col;              //   the sigmoid of its logit in this column (-1: one)
+  int* idx_out;              // [T][top + always]
+  float* wt_out;
+  __device__ __forceinline__ int row_out() const { return top + always; }
+};
+
+// One warp routes token t; `s` holds 2 E + n_groups floats of shared memory of its own. Choice scores may be negative: what cannot be
+// chosen counts as minus infinity.
+__device__ __forceinline__ void route_token(const RouteArgs& a, int t, float* s, int lane) {
+  const int E = a.E;
   float* c = s + E;
   float* g = c + E;
   float mx = -INFINITY;
   for (int e = lane; e < E; e += 32) {
-    float z = logits[(size_t)t * row + e];
-    for (int p = 1; p < P; p++) z += logits[p * stride_p + (size_t)t * row + e];
-    if (logit_bias) z += logit_bias[e];
+    float z = a.logits[(size_t)t * a.row + e];
+    for (int p = 1; p < a.P; p++) z += a.logits[p * a.stride_p + (size_t)t * a.row + e];
+    if (a.logit_bias) z += a.logit_bias[e];
     s[e] = z;
     mx = fmaxf(mx, z);
   }
-  if (score == 1) {   // every expert's own sigmoid
+  if (a.score == 1) {   // every expert's own sigmoid
     for (int e = lane; e < E; e += 32) s[e] = 1.f / (1.f + expf(-s[e]));
-  } else if (score == 0) {
+  } else if (a.score == 0) {
     mx = ib::warp_max(mx);
     float sum = 0.f;
     for (int e = lane; e < E; e += 32) {
@@ -72,15 +81,15 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int P, size_t
     const float inv = 1.f / sum;
     for (int e = lane; e < E; e += 32) s[e] *= inv;
   }
-  for (int e = lane; e < E; e += 32) c[e] = correction ? s[e] + correction[e] : s[e];
+  for (int e = lane; e < E; e += 32) c[e] = a.correction ? s[e] + a.correction[e] : s[e];
   __syncwarp();
-  if (n_groups > 1 && keep < n_groups) {
-    const int per = E / n_groups;
-    for (int k = lane; k < n_groups; k += 32) {
+  if (a.n_groups > 1 && a.keep < a.n_groups) {
+    const int per = E / a.n_groups;
+    for (int k = lane; k < a.n_groups; k += 32) {
       // the group's `group_top` largest choice scores, found one after the other (ties: the lower index first, which changes no sum)
       float total = 0.f;
       int taken[4] = {-1, -1, -1, -1};
-      for (int r = 0; r < group_top && r < per; r++) {
+      for (int r = 0; r < a.group_top && r < per; r++) {
         float b = -INFINITY;
         int bi = -1;
         for (int e = k * per; e < (k + 1) * per; e++) {
@@ -93,13 +102,13 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int P, size_t
       g[k] = total;
     }
     __syncwarp();
-    for (int r = 0; r < keep; r++) {   // the best groups, one after the other; a kept group is marked in `g` by NaN
+    for (int r = 0; r < a.keep; r++) {   // the best groups, one after the other; a kept group is marked in `g` by NaN
       float bv = -INFINITY;
       int bi = 0x7fffffff;
-      for (int k = lane; k < n_groups; k += 32)
+      for (int k = lane; k < a.n_groups; k += 32)
         if (g[k] == g[k] && (bi == 0x7fffffff || g[k] > bv)) bv = g[k], bi = k;
       warp_argmax(bv, bi);
-      if (lane == 0 && bi < n_groups) g[bi] = __int_as_float(0x7fc00000);
+      if (lane == 0 && bi < a.n_groups) g[bi] = __int_as_float(0x7fc00000);
       __syncwarp();
     }
     for (int e = lane; e < E; e += 32)
@@ -107,7 +116,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int P, size_t
     __syncwarp();
   }
   float chosen_sum = 0.f, chosen_max = 0.f;
-  for (int r = 0; r < top; r++) {
+  for (int r = 0; r < a.top; r++) {
     float bv = -INFINITY;
     int bi = 0x7fffffff;
     for (int e = lane; e < E; e += 32)
@@ -116,36 +125,55 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int P, size_t
     float w = 0.f;
     if (bi >= E) {   // fewer experts that can be chosen than choices: weight zero
       bi = 0;
-    } else if (score == 2) {   // the softmax over the chosen logits: the first choice has the largest
+    } else if (a.score == 2) {   // the softmax over the chosen logits: the first choice has the largest
       if (r == 0) chosen_max = s[bi];
       w = expf(s[bi] - chosen_max);
     } else {
       w = s[bi];
     }
     if (lane == 0) {
-      idx_out[(size_t)t * top + r] = bi;
-      wt_out[(size_t)t * top + r] = w;
+      a.idx_out[(size_t)t * a.row_out() + r] = bi;
+      a.wt_out[(size_t)t * a.row_out() + r] = w;
       c[bi] = -INFINITY;
     }
     chosen_sum += w;
     __syncwarp();
   }
   if (lane == 0) {
-    const float f = renorm ? route_scale / (chosen_sum > 0.f ? chosen_sum : 1.f) : route_scale;
-    for (int r = 0; r < top; r++) wt_out[(size_t)t * top + r] *= f;
+    const float f = a.renorm ? a.route_scale / (chosen_sum > 0.f ? chosen_sum : 1.f) : a.route_scale;
+    for (int r = 0; r < a.top; r++) a.wt_out[(size_t)t * a.row_out() + r] *= f;
   }
+  for (int r = lane; r < a.always; r += 32) {
+    float w = 1.f;
+    if (a.gate_col >= 0) {
+      const float* src = a.logits + (size_t)t * a.row + a.gate_col;
+      float z = src[0];
+      for (int p = 1; p < a.P; p++) z += src[p * a.stride_p];
+      w = 1.f / (1.f + expf(-z));
+    }
+    a.idx_out[(size_t)t * a.row_out() + a.top + r] = E + r;
+    a.wt_out[(size_t)t * a.row_out() + a.top + r] = w;
+  }
+}
+
+__global__ void moe_route_kernel(RouteArgs a) {
+  extern __shared__ float sm[];   // per warp: E scores, E choice scores, then n_groups group scores
+  ib::pdl_launch_dependents();
+  ib::pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * kRouteWarps + warp;
+  if (t >= a.T) return;
+  route_token(a, t, sm + (size_t)warp * (2 * a.E + a.n_groups), lane);
 }
 
 constexpr int SM_ = 64;   // rows of a tile of the grouped product
 
-__global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ idx, int R, int top, int E, int tile_rows, int* __restrict__ offsets,
-                                                        int* __restrict__ tile_start, int* __restrict__ row_of_pair, int* __restrict__ token_of_row) {
-  extern __shared__ int si[];   // counts[E], fill[E], start[E + 1]
-  int* counts = si;
+// The regrouping by one CTA; `si` holds 3 E + 1 ints of shared memory.
+__device__ __forceinline__ void sort_pairs(const int* idx, int R, int top, int E, int tile_rows, int* __restrict__ offsets, int* __restrict__ tile_start,
+                                           int* __restrict__ row_of_pair, int* __restrict__ token_of_row, int* si) {
+  int* counts = si;   // counts[E], fill[E], start[E + 1]
   int* fill = si + E;
   int* start = si + 2 * E;
-  ib::pdl_launch_dependents();
-  ib::pdl_wait();
   for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = 0, fill[e] = 0;
   __syncthreads();
   for (int r = threadIdx.x; r < R; r += blockDim.x) {
@@ -176,6 +204,31 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ 
     row_of_pair[r] = row;
     token_of_row[row] = r / top;
   }
+}
+
+__global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ idx, int R, int top, int E, int tile_rows, int* __restrict__ offsets,
+                                                        int* __restrict__ tile_start, int* __restrict__ row_of_pair, int* __restrict__ token_of_row) {
+  extern __shared__ int si[];
+  ib::pdl_launch_dependents();
+  ib::pdl_wait();
+  sort_pairs(idx, R, top, E, tile_rows, offsets, tile_start, row_of_pair, token_of_row, si);
+}
+
+// Both for a step of few tokens: one CTA routes every token (a warp each, in rounds) and regroups the pairs.
+__global__ void __launch_bounds__(1024) moe_route_sort_kernel(RouteArgs a, int tile_rows, int* __restrict__ offsets, int* __restrict__ tile_start,
+                                                              int* __restrict__ row_of_pair, int* __restrict__ token_of_row) {
+  extern __shared__ float sm[];
+  ib::pdl_launch_dependents();
+  ib::pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const int per = 2 * a.E + a.n_groups, E = a.E + a.always;
+  for (int t = warp; t < a.T; t += warps) {
+    route_token(a, t, sm + (size_t)warp * per, lane);
+    __syncwarp();
+  }
+  __syncthreads();
+  // the choices were written by this CTA: they are read as ordinary memory, not through a read-only path
+  sort_pairs(a.idx_out, a.T * a.row_out(), a.row_out(), E, tile_rows, offsets, tile_start, row_of_pair, token_of_row, (int*)(sm + (size_t)warps * per));
 }
 
 template <typename X, typename W, typename O>
@@ -286,6 +339,8 @@ __global__ void gather_rows_kernel(const uint4* __restrict__ x, const int* __res
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < chunks; c += gridDim.y * blockDim.x) out[(size_t)r * chunks + c] = src[c];
 }
 
+// VEC: 16-byte accesses (H a multiple of 4); an output's sum runs in the same order in both forms.
+template <bool VEC>
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ row_of_pair, const float* __restrict__ wt, int top,
                                    const float* __restrict__ base, int P, size_t stride_p, float* __restrict__ out, int H, const float* __restrict__ gate,
                                    int gate_P, size_t gate_stride, int gate_row) {
@@ -299,6 +354,34 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
     float z = gr[0];
     for (int p = 1; p < gate_P; p++) z += gr[p * gate_stride];
     f = 1.f / (1.f + expf(-z));
+  }
+  if constexpr (VEC) {
+    for (int i = (blockIdx.x * blockDim.x + threadIdx.x) * 4; i < H; i += gridDim.x * blockDim.x * 4) {
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int p = 0; p < P; p++) {
+        const float4 b = *(const float4*)(base + p * stride_p + (size_t)t * H + i);
+        a.x += b.x, a.y += b.y, a.z += b.z, a.w += b.w;
+      }
+      if (gate) a.x *= f, a.y *= f, a.z *= f, a.w *= f;
+      for (int k0 = 0; k0 < top; k0 += 4) {   // four choices' rows are requested before the first is used
+        float4 v[4];
+        float c[4];
+#pragma unroll
+        for (int u = 0; u < 4; u++) {
+          if (k0 + u >= top) continue;
+          const size_t at = (size_t)t * top + k0 + u;
+          c[u] = wt ? wt[at] : 1.f;
+          v[u] = *(const float4*)(y + (size_t)row_of_pair[at] * H + i);
+        }
+#pragma unroll
+        for (int u = 0; u < 4; u++) {
+          if (k0 + u >= top) continue;
+          a.x = fmaf(c[u], v[u].x, a.x), a.y = fmaf(c[u], v[u].y, a.y), a.z = fmaf(c[u], v[u].z, a.z), a.w = fmaf(c[u], v[u].w, a.w);
+        }
+      }
+      *(float4*)(out + (size_t)t * H + i) = a;
+    }
+    return;
   }
   for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < H; i += gridDim.x * blockDim.x) {
     float a = 0.f;
@@ -328,22 +411,55 @@ __global__ void scatter_scaled_rows_kernel(const X* __restrict__ x, const int* _
 
 }  // namespace
 
+namespace {
+int check_route(const RouteArgs& a, const char* who) {
+  IB_CHECK_ARG(a.group_top >= 1 && a.group_top <= 4, "%s: a group's score is the sum of its %d largest scores (1 to 4)", who, a.group_top);
+  IB_CHECK_ARG(a.P >= 1 && a.E > 0 && a.top > 0 && a.top <= a.E, "%s: bad sizes P=%d experts=%d top=%d", who, a.P, a.E, a.top);
+  IB_CHECK_ARG(a.score >= 0 && a.score <= 2, "%s: score %d is not known (0: softmax, 1: sigmoid, 2: softmax over the chosen logits)", who, a.score);
+  IB_CHECK_ARG(a.row >= a.E && a.gate_col < a.row && a.always >= 0, "%s: rows of %d logits do not hold %d experts or column %d", who, a.row, a.E, a.gate_col);
+  IB_CHECK_ARG(a.n_groups >= 1 && a.E % a.n_groups == 0 && a.keep >= 1 && a.keep <= a.n_groups, "%s: %d experts in %d groups of which %d stay", who, a.E, a.n_groups, a.keep);
+  return 0;
+}
+RouteArgs route_args(const float* logits, int P, long long stride_p, int T, int E, int n_groups, int keep, int top, float route_scale, int renorm, int* idx_out, float* wt_out,
+                     int score, const float* correction, int group_top, int row, const float* logit_bias, int always, int gate_col) {
+  RouteArgs a;
+  a.logits = logits, a.P = P, a.stride_p = (size_t)stride_p, a.T = T, a.E = E, a.row = row > 0 ? row : E, a.n_groups = n_groups, a.keep = keep, a.top = top;
+  a.route_scale = route_scale, a.renorm = renorm || score == 2, a.score = score, a.correction = correction, a.logit_bias = logit_bias, a.group_top = group_top;
+  a.always = always, a.gate_col = gate_col, a.idx_out = idx_out, a.wt_out = wt_out;
+  return a;
+}
+}  // namespace
+
+// row: entries of a row of logits (0: E). correction, group_top, logit_bias, always, gate_col: see RouteArgs.
 extern "C" int ib_moe_route(const float* logits, int P, long long stride_p, int T, int E, int n_groups, int keep, int top, float route_scale, int renorm,
-                            int* idx_out, float* wt_out, int score, const float* correction, int group_top, int row, const float* logit_bias, cudaStream_t stream) {
-  // row: entries of a row of logits (0: E). logit_bias: see the kernel.
-  if (row <= 0) row = E;
-  // correction: float32 [E] added to the scores for the choice only, or null; group_top: how many of a group's largest choice scores make its score (1 to 4).
+                            int* idx_out, float* wt_out, int score, const float* correction, int group_top, int row, const float* logit_bias, int always, int gate_col,
+                            cudaStream_t stream) {
   if (T == 0) return 0;
-  IB_CHECK_ARG(group_top >= 1 && group_top <= 4, "moe_route: a group's score is the sum of its %d largest scores (1 to 4)", group_top);
-  IB_CHECK_ARG(P >= 1 && E > 0 && top > 0 && top <= E, "moe_route: bad sizes P=%d experts=%d top=%d", P, E, top);
-  IB_CHECK_ARG(score >= 0 && score <= 2, "moe_route: score %d is not known (0: softmax, 1: sigmoid, 2: softmax over the chosen logits)", score);
-  IB_CHECK_ARG(row >= E, "moe_route: rows of %d logits do not hold %d experts", row, E);
-  IB_CHECK_ARG(n_groups >= 1 && E % n_groups == 0 && keep >= 1 && keep <= n_groups, "moe_route: %d experts in %d groups of which %d stay", E, n_groups, keep);
+  const RouteArgs a = route_args(logits, P, stride_p, T, E, n_groups, keep, top, route_scale, renorm, idx_out, wt_out, score, correction, group_top, row, logit_bias, always, gate_col);
+  if (check_route(a, "moe_route")) return 1;
   const size_t smem = (size_t)kRouteWarps * (2 * E + n_groups) * sizeof(float);
   IB_CHECK_ARG(smem <= 48 * 1024, "moe_route: %d experts need %zu bytes of shared memory, more than 48 KiB", E, smem);
-  ib::launch(moe_route_kernel, (unsigned)((T + kRouteWarps - 1) / kRouteWarps), kRouteWarps * 32, smem, stream, logits, P, (size_t)stride_p, T, E, n_groups, keep,
-             top, route_scale, renorm || score == 2, idx_out, wt_out, score, correction, group_top, row, logit_bias);
+  ib::launch(moe_route_kernel, (unsigned)((T + kRouteWarps - 1) / kRouteWarps), kRouteWarps * 32, smem, stream, a);
   IB_CHECK_LAUNCH("moe_route");
+  return 0;
+}
+
+// ib_moe_route and ib_moe_sort (over E + always experts) in one kernel, for up to 128 tokens; ib_moe_route_sort_fits says whether the sizes allow it.
+extern "C" int ib_moe_route_sort_fits(int T, int E, int n_groups, int always) {
+  const int warps = T < 32 ? (T > 8 ? T : 8) : 32;
+  return T <= 128 && ((size_t)warps * (2 * E + n_groups) + 3 * (E + always) + 1) * 4 <= 48 * 1024;
+}
+extern "C" int ib_moe_route_sort(const float* logits, int P, long long stride_p, int T, int E, int n_groups, int keep, int top, float route_scale, int renorm,
+                                 int* idx_out, float* wt_out, int score, const float* correction, int group_top, int row, const float* logit_bias, int always, int gate_col,
+                                 int tile_rows, int* offsets, int* tile_start, int* row_of_pair, int* token_of_row, cudaStream_t stream) {
+  if (T == 0) return 0;
+  const RouteArgs a = route_args(logits, P, stride_p, T, E, n_groups, keep, top, route_scale, renorm, idx_out, wt_out, score, correction, group_top, row, logit_bias, always, gate_col);
+  if (check_route(a, "moe_route_sort")) return 1;
+  IB_CHECK_ARG(tile_rows > 0 && ib_moe_route_sort_fits(T, E, n_groups, always), "moe_route_sort: %d tokens, %d experts and tiles of %d rows do not fit one CTA", T, E, tile_rows);
+  const int warps = T < 32 ? (T > 8 ? T : 8) : 32;
+  const size_t smem = ((size_t)warps * (2 * E + n_groups) + 3 * (E + always) + 1) * 4;
+  ib::launch(moe_route_sort_kernel, 1, warps * 32, smem, stream, a, tile_rows, offsets, tile_start, row_of_pair, token_of_row);
+  IB_CHECK_LAUNCH("moe_route_sort");
   return 0;
 }
 
@@ -385,8 +501,11 @@ extern "C" int ib_moe_combine(const float* y, const int* row_of_pair, const floa
   IB_CHECK_ARG(!gate || (gate_P >= 1 && gate_row >= 1), "moe_combine: a gate of %d parts and rows of %d", gate_P, gate_row);
   IB_CHECK_ARG(T > 0 && H > 0 && top > 0 && P >= 0, "moe_combine: bad sizes T=%d H=%d top=%d P=%d", T, H, top, P);
   IB_CHECK_ARG(T <= 65535, "moe_combine: T=%d rows exceed the grid limit 65535", T);
-  dim3 grid(min((H + 255) / 256, 64), T);
-  ib::launch(moe_combine_kernel, grid, 256, 0, stream, y, row_of_pair, wt, top, base, P, (size_t)stride_p, out, H, gate, gate_P, (size_t)gate_stride, gate_row);
+  const bool vec = H % 4 == 0 && ((uintptr_t)y & 15) == 0 && ((uintptr_t)base & 15) == 0 && ((uintptr_t)out & 15) == 0 && stride_p % 4 == 0;
+  const int per = vec ? 1024 : 256;
+  dim3 grid(min((H + per - 1) / per, 64), T);
+  if (vec) ib::launch(moe_combine_kernel<true>, grid, 256, 0, stream, y, row_of_pair, wt, top, base, P, (size_t)stride_p, out, H, gate, gate_P, (size_t)gate_stride, gate_row);
+  else ib::launch(moe_combine_kernel<false>, grid, 256, 0, stream, y, row_of_pair, wt, top, base, P, (size_t)stride_p, out, H, gate, gate_P, (size_t)gate_stride, gate_row);
   IB_CHECK_LAUNCH("moe_combine");
   return 0;
 }

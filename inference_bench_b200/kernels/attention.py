@@ -172,13 +172,17 @@ def decode_fused(ctx, qkv: torch.Tensor, q_norm_w, k_norm_w, eps: float, cos, si
 
 def paged_attention(ctx, q: torch.Tensor, cache: ops.KvLayerView, heads: int, window: Optional[int], scale: float, qk_dim: Optional[int] = None,
                     v_dim: Optional[int] = None, softcap: float = 0.0, sink: bool = False, chunk: int = 0, sink_values: Optional[torch.Tensor] = None,
-                    gate: Optional[tuple] = None, out_scale: float = 1.0, out: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
+                    gate: Optional[tuple] = None, out_scale: float = 1.0, out: Optional[torch.Tensor] = None, keep_first: int = 0,
+                    diff: Optional[tuple] = None) -> torch.Tensor:
     """q [T, heads * qk_dim] (activation dtype) -> attention output [T, heads * v_dim] of the same dtype. qk_dim, v_dim: the head sizes
     (default: the cache's row); softcap > 0 caps the scores with a tanh; sink adds one to the softmax's denominator, or with sink_values
     (float32 [heads]) exp of the head's value. chunk > 0: instead of a window, a position sees the earlier positions of its own block of
     `chunk` positions, blocks counted from position 0. gate = (float32 partial sums [P, T, row], the first head's column): head h's
     output is multiplied by the sigmoid of its column; out_scale multiplies the output. out: a buffer [T, >= heads * v_dim] whose first
-    columns are written, instead of a new one. keep_first (with a window): the request's first positions, which are seen whatever the window."""
+    columns are written, instead of a new one. keep_first (with a window): the request's first positions, which are seen whatever the window.
+    diff = (lambda, eps, factor): query heads 2h and 2h + 1 are two maps of head h; returned is factor * u / sqrt(mean(u^2) + eps) with u the first map's
+    output minus lambda times the second's, [T, heads / 2 * v_dim] (in a step of decoded tokens on the tensor-core kernels from the kernel that
+    merges the slices)."""
     rt = ctx.rt
     view = cache.c_view()
     T = q.shape[0]
@@ -186,11 +190,21 @@ def paged_attention(ctx, q: torch.Tensor, cache: ops.KvLayerView, heads: int, wi
     qk_dim, v_dim = qk_dim or view.head_dim, v_dim or view.head_dim
     if chunk and window:
         raise L.KernelError("paged_attention: a window and blocks of positions exclude one another")
-    if out is None:
+    if diff is not None:
+        if heads % 2 or out is not None or sink or gate is not None or out_scale != 1.0:
+            raise L.KernelError("paged_attention: the difference of two maps takes an even number of heads and no sink, gate, scale or output buffer")
+        fits = not softcap and qk_dim == view.head_dim and v_dim == view.head_dim and has_tensor_core_kernel(q.dtype, view.head_dim, heads, view.kv_heads)
+        if not fits or _work_lists(ctx)["n_tiles"]:
+            a = paged_attention(ctx, q, cache, heads, window, scale, qk_dim, v_dim, softcap, chunk=chunk, keep_first=keep_first)
+            out = rt.empty((T, heads // 2 * v_dim), q.dtype)
+            ops.diff_combine(a, *diff, out, v_dim)
+            return out
+        out = rt.empty((T, heads // 2 * v_dim), q.dtype)
+    elif out is None:
         out = rt.empty((T, heads * v_dim), q.dtype)
     elif out.dim() != 2 or out.shape[0] != T or out.shape[1] < heads * v_dim or out.dtype != q.dtype or not out.is_contiguous():
         raise L.KernelError(f"paged_attention: out must be a contiguous [{T}, >= {heads * v_dim}] of {q.dtype}, got {tuple(out.shape)} of {out.dtype}")
-    tailed = chunk > 0 or sink_values is not None or gate is not None or out_scale != 1.0 or out.shape[1] != heads * v_dim
+    tailed = chunk > 0 or sink_values is not None or gate is not None or out_scale != 1.0 or out.shape[1] != heads * v_dim or diff is not None
     capped = softcap > 0 or sink or tailed or keep_first > 0
     generic = qk_dim != view.head_dim or v_dim != view.head_dim or not has_tensor_core_kernel(q.dtype, view.head_dim, heads, view.kv_heads)
     generic = generic or (tailed and out.shape[1] % 8 != 0)
@@ -203,7 +217,10 @@ def paged_attention(ctx, q: torch.Tensor, cache: ops.KvLayerView, heads: int, wi
         return out
     tail_ref = None
     if tailed:
-        t = L.AttnTail(sink_values=ops._ptr(sink_values), gate=None, gate_parts=0, gate_row=0, gate_stride=0, out_scale=float(out_scale), out_row=out.shape[1])
+        t = L.AttnTail(sink_values=ops._ptr(sink_values), gate=None, gate_parts=0, gate_row=0, gate_stride=0, out_scale=float(out_scale), out_row=out.shape[1], diff=0,
+                       diff_lambda=0.0, diff_eps=0.0, diff_factor=0.0)
+        if diff is not None:
+            t.diff, t.diff_lambda, t.diff_eps, t.diff_factor, t.out_scale, t.out_row = 1, float(diff[0]), float(diff[1]), float(diff[2]), 0.0, 0
         if sink_values is not None:
             ops._check("sink_values", sink_values, torch.float32, (heads,))
         if gate is not None:

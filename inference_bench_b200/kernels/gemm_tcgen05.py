@@ -31,6 +31,7 @@ L.register("ib_gemm_tcgen05_2cta_add", [L._p, L._p, L._p, L._i, L._i, L._i, L._p
 L.register("ib_gemm_qkv_tcgen05_2cta", [L._p, L._p, L._i, L._i, L._p, L._p, L._f, L._p, L._p, L._p, L._p, L._p, C.POINTER(L.KvView), L._i, L._i, L._p, L._p])
 
 L.register("ib_gemm_grouped_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._p, L._p, L._i, L._p, L._p])
+L.register("ib_gemm_parts_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._i, L._p, L._p])
 L.register("ib_gemm_grouped_relu2_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._p, L._p, L._i, L._p, L._p])
 L.register("ib_gemm_grouped_swiglu_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._p, L._p, L._i, L._p, L._p])
 
@@ -316,6 +317,21 @@ def gemm_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bn: int, o
     ops._check("w", w, torch.bfloat16, (E, N, K))
     ops._check("out", out, torch.float32, (R, N))
     L.call("ib_gemm_grouped_tcgen05", x.data_ptr(), w.data_ptr(), out.data_ptr(), R, N, K, bn, offsets.data_ptr(), tiles.data_ptr(), E, status.data_ptr(), ops._stream())
+
+
+PARTS_MAX_TOKENS = 128   # up to here several products of one shape run as one launch; above, each product fills the GPU by itself
+
+
+def gemm_parts(rt, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """x [parts, T, K], w [parts, N, K] (bfloat16) -> float32 partial sums [P, parts, T, N] of every part's product with its own matrix, in one launch."""
+    parts, T, K = x.shape
+    N = w.shape[1]
+    ops._check("x", x, torch.bfloat16)
+    ops._check("w", w, torch.bfloat16, (parts, N, K))
+    bn, splits, _ = choose(T, parts * N, K, True, rt.sm_count)
+    out = rt.empty((splits, parts, T, N), torch.float32)
+    L.call("ib_gemm_parts_tcgen05", x.data_ptr(), w.data_ptr(), out.data_ptr(), parts, T, N, K, bn, splits, rt.status.data_ptr(), ops._stream())
+    return out
 
 
 def gemm_grouped_relu2(x: torch.Tensor, w: torch.Tensor, act: torch.Tensor, bn: int, offsets: torch.Tensor, tiles: torch.Tensor, status: torch.Tensor) -> None:

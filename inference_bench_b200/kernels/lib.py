@@ -51,6 +51,10 @@ class AttnTail(C.Structure):
         ("gate_stride", C.c_longlong),
         ("out_scale", C.c_float),
         ("out_row", C.c_int),
+        ("diff", C.c_int),
+        ("diff_lambda", C.c_float),
+        ("diff_eps", C.c_float),
+        ("diff_factor", C.c_float),
     ]
 
 

@@ -501,7 +501,8 @@ def latent_attention_mma(q_full: torch.Tensor, kv: KvLayerView, positions: torch
 
 
 # ---------------------------------------------------------------- routed experts (csrc/moe.cu)
-L.register("ib_moe_route", [L._p, L._i, L._ll, L._i, L._i, L._i, L._i, L._i, L._f, L._i, L._p, L._p, L._i, L._p, L._i, L._i, L._p, L._p])
+L.register("ib_moe_route", [L._p, L._i, L._ll, L._i, L._i, L._i, L._i, L._i, L._f, L._i, L._p, L._p, L._i, L._p, L._i, L._i, L._p, L._i, L._i, L._p])
+L.register("ib_moe_route_sort", [L._p, L._i, L._ll, L._i, L._i, L._i, L._i, L._i, L._f, L._i, L._p, L._p, L._i, L._p, L._i, L._i, L._p, L._i, L._i, L._i, L._p, L._p, L._p, L._p, L._p])
 ROUTE_SCORES = {"softmax": 0, "sigmoid": 1, "chosen_softmax": 2}
 GROUPED_ACTS = {"none": 0, "swiglu": 1, "relu2": 2}
 L.register("ib_scatter_scaled_rows", [L._p, L._i, L._p, L._p, L._i, L._p, L._i, L._i, L._p])
@@ -529,10 +530,13 @@ L.register("ib_moe_combine", [L._p, L._p, L._p, L._i, L._p, L._i, L._ll, L._p, L
 
 def moe_route(logits: torch.Tensor, n_groups: int, keep: int, top: int, route_scale: float, renorm: bool, idx: torch.Tensor, wt: torch.Tensor,
               score: str = "softmax", correction: Optional[torch.Tensor] = None, group_top: int = 1, experts: Optional[int] = None,
-              logit_bias: Optional[torch.Tensor] = None) -> None:
+              logit_bias: Optional[torch.Tensor] = None, always: int = 0, gate_col: int = -1, sort: Optional[tuple] = None) -> None:
     """logits float32 [P, T, E] (partial sums) -> idx int32 [T, top], wt float32 [T, top]. score: "softmax" over all experts, "sigmoid" of every
     expert's logit on its own, or "chosen_softmax" (chosen by the logits, weighted by the softmax over the chosen ones). experts: how many
-    of a row's first entries are experts (default: all). logit_bias: float32 [E] added to the logits. correction: float32 [E] added to the scores where groups and experts are chosen (the
+    of a row's first entries are experts (default: all). logit_bias: float32 [E] added to the logits. always: experts E .. E + always - 1 that every
+    token uses as well, the last of its choices (idx and wt are then [T, top + always]), weighted by the sigmoid of its logit in column gate_col (-1: one).
+    sort = (offsets, tile_start, row_of_pair, token_of_row, tile_rows): also what `moe_sort` does for the E + always experts, in the same kernel (few
+    tokens: `moe_route_sort_fits`). correction: float32 [E] added to the scores where groups and experts are chosen (the
     weights are the scores without it). group_top: a group's score is the sum of its `group_top` largest choice scores (1: the largest)."""
     if score not in ROUTE_SCORES:
         raise L.KernelError(f"moe_route: score {score!r} is not known ({', '.join(ROUTE_SCORES)})")
@@ -541,12 +545,24 @@ def moe_route(logits: torch.Tensor, n_groups: int, keep: int, top: int, route_sc
     E = row if experts is None else int(experts)
     if logit_bias is not None:
         _check("logit_bias", logit_bias, torch.float32, (E,))
-    _check("idx", idx, torch.int32, (T, top))
-    _check("wt", wt, torch.float32, (T, top))
+    _check("idx", idx, torch.int32, (T, top + always))
+    _check("wt", wt, torch.float32, (T, top + always))
     if correction is not None:
         _check("correction", correction, torch.float32, (E,))
-    L.call("ib_moe_route", logits.data_ptr(), P, T * row, T, E, n_groups, keep, top, float(route_scale), 1 if renorm else 0, idx.data_ptr(), wt.data_ptr(),
-           ROUTE_SCORES[score], _ptr(correction), int(group_top), row, _ptr(logit_bias), _stream())
+    args = (logits.data_ptr(), P, T * row, T, E, n_groups, keep, top, float(route_scale), 1 if renorm else 0, idx.data_ptr(), wt.data_ptr(),
+            ROUTE_SCORES[score], _ptr(correction), int(group_top), row, _ptr(logit_bias), int(always), int(gate_col))
+    if sort is None:
+        L.call("ib_moe_route", *args, _stream())
+        return
+    offsets, tile_start, row_of_pair, token_of_row, tile_rows = sort
+    for name, t, n in (("offsets", offsets, E + always + 1), ("tile_start", tile_start, E + always + 1), ("row_of_pair", row_of_pair, T * (top + always)),
+                       ("token_of_row", token_of_row, T * (top + always))):
+        _check(name, t, torch.int32, (n,))
+    L.call("ib_moe_route_sort", *args, int(tile_rows), offsets.data_ptr(), tile_start.data_ptr(), row_of_pair.data_ptr(), token_of_row.data_ptr(), _stream())
+
+
+def moe_route_sort_fits(T: int, experts: int, groups: int, always: int = 0) -> bool:
+    return bool(L.load().ib_moe_route_sort_fits(int(T), int(experts), int(groups), int(always)))
 
 
 def moe_sort(idx: torch.Tensor, n_experts: int, offsets: torch.Tensor, tile_start: torch.Tensor, row_of_pair: torch.Tensor, token_of_row: torch.Tensor,

@@ -79,7 +79,6 @@ class DifferentialAttention(base.Mixer):
         q = rt.empty((T, self.heads * MAPS * MAPS * self.dim))
         ops.map_qkv(rt.linear(h, self.w_in), self.in_bias, cos, sin, getattr(self.position, "pairing", "half") == "interleaved", ctx.positions, ctx.seg_of_token, q, cache,
                     self.heads, MAPS, self.dim, self.vdim, rt.status, write_kv=self.own_kv)
-        a = attention.paged_attention(ctx, q, cache, self.heads * MAPS, self.window, self.scale, qk_dim=MAPS * self.dim, v_dim=self.vdim, keep_first=self.keep_first)
-        out = rt.empty((T, self.heads * self.vdim))
-        ops.diff_combine(a, self.lam, self.norm_eps, 1.0 - self.diff, out, self.vdim)
+        out = attention.paged_attention(ctx, q, cache, self.heads * MAPS, self.window, self.scale, qk_dim=MAPS * self.dim, v_dim=self.vdim, keep_first=self.keep_first,
+                                        diff=(self.lam, self.norm_eps, 1.0 - self.diff))
         return rt.linear(out, self.wo)

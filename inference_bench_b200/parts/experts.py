@@ -25,6 +25,10 @@ from . import base
 from .base import WeightSpec
 
 
+FEW_TOKENS = 64         # up to here the shared expert runs beside the routed ones
+ROUTE_SORT_TOKENS = 32  # up to here the choice and the regrouping are one kernel (a warp of one CTA per token)
+
+
 @base.register_feed_forward("routed_experts")
 class RoutedExperts(base.FeedForward):
     def __init__(self, prefix: str, hidden: int, expert_ff: int, experts: int, top: int, route_scale: float = 1.0, groups: int = 1, groups_keep: int = 1,
@@ -35,7 +39,7 @@ class RoutedExperts(base.FeedForward):
         if activation not in ("swiglu", "relu2"):
             raise ValueError(f"activation {activation!r} is not known (swiglu, relu2)")
         self.gated, self.router_bias, self.shared_gate = activation == "swiglu", router_bias, shared_gate if shared_ff else ""
-        self.b_router = None
+        self.b_router, self.blocks = None, 0
         if score not in ops.ROUTE_SCORES or weight_on not in ("output", "input"):
             raise ValueError(f"score {score!r} ({', '.join(ops.ROUTE_SCORES)}) or weight_on {weight_on!r} (output, input) is not known")
         if not 1 <= group_top <= 4:
@@ -80,51 +84,67 @@ class RoutedExperts(base.FeedForward):
             self.w_correction = rt.vector(weights[f"{self.prefix}.{self.correction}"])
         # [experts, gate rows then up rows, width] and [experts, width, inner]: one tensor each, so a tile of the grouped product finds its expert by an offset
         front = (0, 1) if self.gated else (1,)
-        self.w_gu = rt.upload(torch.stack([torch.cat([weights[self._expert(k, i)] for i in front], dim=0) for k in range(self.experts)]), rt.act_dtype)
-        self.w_d = rt.upload(torch.stack([weights[self._expert(k, 2)] for k in range(self.experts)]), rt.act_dtype)
-        if self.shared_ff:
-            self.shared_gu = rt.matrix(torch.cat([weights[self._shared(i)] for i in front], dim=0))
-            self.shared_d = rt.matrix(weights[self._shared(2)])
+        S, F = self.shared_ff, self.expert_ff
+        self.blocks = S // F if S and S % F == 0 and not self.gated and self.weight_on == "output" else 0
+        gu = [torch.cat([weights[self._expert(k, i)] for i in front], dim=0) for k in range(self.experts)]
+        down = [weights[self._expert(k, 2)] for k in range(self.experts)]
+        if S:
+            shared_gu, shared_d = torch.cat([weights[self._shared(i)] for i in front], dim=0), weights[self._shared(2)]
+            # the shared expert's inner channels in blocks of a routed expert's size, behind the routed experts
+            gu += list(shared_gu.split(F)) if self.blocks else []
+            down += list(shared_d.split(F, dim=1)) if self.blocks else []
+        self.w_gu, self.w_d = rt.upload(torch.stack(gu), rt.act_dtype), rt.upload(torch.stack(down), rt.act_dtype)
+        if S:
+            self.shared_gu = rt.matrix(self.w_gu[self.experts:].reshape(S, self.hidden) if self.blocks else shared_gu)   # (a view where the blocks hold it)
+            self.shared_d = rt.matrix(self.w_d[self.experts] if self.blocks == 1 else shared_d)
 
     def forward(self, ctx, h):
         rt, T, E, top = ctx.rt, ctx.n_tokens, self.experts, self.top
-        R = T * top
         logits = rt.linear(h, self.w_router)                     # float32 partial sums [P, T, E (+ 1)]
-        idx, wt = rt.empty((T, top), torch.int32), rt.empty((T, top), torch.float32)
-        ops.moe_route(logits, self.groups, self.groups_keep, top, self.route_scale, self.renorm, idx, wt, self.score, correction=self.w_correction, group_top=self.group_top,
-                      experts=E, logit_bias=self.b_router)
+        # few tokens: a shared expert that is whole blocks of the routed experts' size runs as further experts that every token uses (in float32
+        # always, so that a token's sums run in one order however many share its step)
+        always = self.blocks if T <= FEW_TOKENS or rt.act_dtype == torch.float32 else 0
+        n, used = E + always, top + always
+        R = T * used
+        idx, wt = rt.empty((T, used), torch.int32), rt.empty((T, used), torch.float32)
         on_input = self.weight_on == "input"
-        offsets, tile_start = rt.empty((E + 1,), torch.int32), rt.empty((E + 1,), torch.int32)
+        offsets, tile_start = rt.empty((n + 1,), torch.int32), rt.empty((n + 1,), torch.int32)
         row_of_pair, token_of_row = rt.empty((R,), torch.int32), rt.empty((R,), torch.int32)
         how = rt.options.expert_gemm
-        bn = G.grouped_token_tile(R, E, self.expert_ff, rt.sm_count)
+        bn = G.grouped_token_tile(R, n, self.expert_ff, rt.sm_count)
         act = rt.empty((R, self.expert_ff))
         y = rt.empty((R, self.hidden), torch.float32)
-        if how in ("auto", "tcgen05") and rt.act_dtype == torch.bfloat16 and rt.gemm != "simt" and G.grouped_supported(self.hidden, self.expert_ff, bn, self.gated):
-            # the tcgen05 kernel of the single-matrix products, its tiles taking their expert from the tile table
-            ops.moe_sort(idx, E, offsets, tile_start, row_of_pair, token_of_row, tile_rows=bn)
+        tcgen05 = how in ("auto", "tcgen05") and rt.act_dtype == torch.bfloat16 and rt.gemm != "simt" and G.grouped_supported(self.hidden, self.expert_ff, bn, self.gated)
+        if how == "tcgen05" and not tcgen05:
+            raise ValueError(f"expert_gemm = \"tcgen05\" needs bfloat16 and inner sizes that are multiples of 8 (of 64 for few tokens), got {self.hidden} and {self.expert_ff}")
+        tile_rows = bn if tcgen05 else ops.moe_tile_rows()
+        one = T <= ROUTE_SORT_TOKENS and ops.moe_route_sort_fits(T, E, self.groups, always)     # the choice and the regrouping in one kernel
+        ops.moe_route(logits, self.groups, self.groups_keep, top, self.route_scale, self.renorm, idx, wt, self.score, correction=self.w_correction, group_top=self.group_top,
+                      experts=E, logit_bias=self.b_router, always=always, gate_col=E if self.shared_gate and always else -1,
+                      sort=(offsets, tile_start, row_of_pair, token_of_row, tile_rows) if one else None)
+        if not one:
+            ops.moe_sort(idx, n, offsets, tile_start, row_of_pair, token_of_row, tile_rows=tile_rows)
+        w_gu, w_d = self.w_gu[:n], self.w_d[:n]
+        if tcgen05:   # the tcgen05 kernel of the single-matrix products, its tiles taking their expert from the tile table
             xs = rt.empty((R, self.hidden))
             if on_input:
                 ops.scatter_scaled_rows(h, row_of_pair, wt, xs)
             else:
                 ops.gather_rows(h, token_of_row, xs)
-            (G.gemm_grouped_swiglu if self.gated else G.gemm_grouped_relu2)(xs, self.w_gu, act, bn, offsets, tile_start, rt.status)
-            G.gemm_grouped(act, self.w_d, y, bn, offsets, tile_start, rt.status)
+            (G.gemm_grouped_swiglu if self.gated else G.gemm_grouped_relu2)(xs, w_gu, act, bn, offsets, tile_start, rt.status)
+            G.gemm_grouped(act, w_d, y, bn, offsets, tile_start, rt.status)
         else:
-            if how == "tcgen05":
-                raise ValueError(f"expert_gemm = \"tcgen05\" needs bfloat16 and inner sizes that are multiples of 8 (of 64 for few tokens), got {self.hidden} and {self.expert_ff}")
             tc = how != "simt"
-            ops.moe_sort(idx, E, offsets, tile_start, row_of_pair, token_of_row)
             src, rows = h, token_of_row
             if on_input:   # the rows in the experts' order, each times its weight; the product then reads them as they lie
                 src, rows = rt.empty((R, self.hidden)), None
                 ops.scatter_scaled_rows(h, row_of_pair, wt, src)
-            ops.gemm_grouped(src, rows, self.w_gu, act, offsets, tile_start, gated=self.gated, tensor_cores=tc and ops.rows_mma_fits(src, self.w_gu),
+            ops.gemm_grouped(src, rows, w_gu, act, offsets, tile_start, gated=self.gated, tensor_cores=tc and ops.rows_mma_fits(src, w_gu),
                              act="none" if self.gated else "relu2")
-            ops.gemm_grouped(act, None, self.w_d, y, offsets, tile_start, gated=False, tensor_cores=tc and ops.rows_mma_fits(act, self.w_d))
+            ops.gemm_grouped(act, None, w_d, y, offsets, tile_start, gated=False, tensor_cores=tc and ops.rows_mma_fits(act, w_d))
         shared = None
-        if self.shared_ff:
+        if self.shared_ff and not always:
             shared = rt.linear(rt.gate_up_act(h, self.shared_gu) if self.gated else rt.up_act(h, self.shared_gu, "relu2"), self.shared_d)
         out = rt.empty((1, T, self.hidden), torch.float32)
-        ops.moe_combine(y, row_of_pair, wt, shared, out[0], weighted=not on_input, gate=(logits, E) if self.shared_gate else None)
+        ops.moe_combine(y, row_of_pair, wt, shared, out[0], weighted=not on_input, gate=(logits, E) if self.shared_gate and shared is not None else None)
         return out

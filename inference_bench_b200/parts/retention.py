@@ -86,7 +86,6 @@ class WkvMixer(base.Mixer):
             raise ValueError(f"heads {heads} and dim {dim} (at most 512) must be positive")
         self.prefix, self.hidden, self.heads, self.dim, self.norm_eps, self.decay_rank, self.names = prefix, hidden, heads, dim, norm_eps, int(decay_rank), tuple(names)
         self.mu = self.w_rkvg = self.stacked = self.w1 = self.w2 = self.w0 = self.u = self.norm_w = self.wo = None
-        self._tables: dict = {}     # tokens of a step -> row ranges of the four products run as one
 
     def cache_need(self):
         return Several((FixedState((self.heads, self.dim, self.dim), torch.float32), FixedState((self.hidden,), torch.float32)))
@@ -105,7 +104,8 @@ class WkvMixer(base.Mixer):
 
     def bind(self, weights, rt):
         self.mu = rt.vector(torch.stack([weights[self._mu(s)] for s in self.MIXES]))                      # [5, W], in the order of MIXES
-        self.w_rkvg = [rt.matrix(weights[self._n(i)]) for i in range(1, 5)]
+        self.stacked = rt.upload(torch.stack([weights[self._n(i)] for i in range(1, 5)]), rt.act_dtype)      # [4, C, W]: r, k, v, g
+        self.w_rkvg = [rt.matrix(w) for w in self.stacked]
         w1, w2 = weights[self._n(5)], weights[self._n(6)]
         if w1.shape[0] != w2.shape[1]:
             raise ValueError(f"{self._n(5)} has {w1.shape[0]} rows, {self._n(6)} has {w2.shape[1]} columns")
@@ -123,7 +123,11 @@ class WkvMixer(base.Mixer):
 
     def _mix(self, ctx, mixes, state):
         rt, T, H, D = ctx.rt, ctx.n_tokens, self.heads, self.dim
-        r, k, v, g = (ops.Parts.columns(rt.linear(mixes[i], w)) for i, w in enumerate(self.w_rkvg))
+        if T <= G.PARTS_MAX_TOKENS and rt.mode == "bfloat16" and rt.gemm != "simt" and G.supports(self.hidden):   # few tokens: the four products as one launch
+            z = G.gemm_parts(rt, mixes[:4], self.stacked)
+            r, k, v, g = (ops.Parts(z, z.shape[0], 4 * T * H * D, H * D, i * T * H * D) for i in range(4))
+        else:
+            r, k, v, g = (ops.Parts.columns(rt.linear(mixes[i], w)) for i, w in enumerate(self.w_rkvg))
         decay = rt.empty((T, H * D), torch.float32)
         ops.decay_rows(rt.linear(mixes[4], self.w1), self.w2, self.w0, decay)
         o = rt.empty((T, H, D), torch.float32)
