@@ -26,9 +26,10 @@
 namespace {
 
 constexpr int kChunk = 16;   // tokens prepared at a time
+constexpr int kLoads = 4;    // values a thread requests at a time while it prepares tokens
+constexpr int kGroup = 8;    // tokens whose outputs are reduced together
 
 // RPT: rows of S a thread holds (for each of its two columns); kCols: value columns per CTA (32, or 16 where a thread holds sixteen rows)
-// BONUS: form 3
 struct RecurrenceExtras {
   const float* cos_t;   // form 2: float32 [T][rot_half], the angles of the first 2 * rot_half entries of q and k (entry i with i + rot_half), or null
   const float* sin_t;
@@ -37,8 +38,9 @@ struct RecurrenceExtras {
   const float* decay;   // form 3: float32 [T][heads * D]
 };
 
-template <int RPT, int kCols, bool BONUS>
-__global__ void __launch_bounds__(kCols * 16) gated_recurrence_kernel(const float* __restrict__ q_src, const float* __restrict__ f_src, const float* __restrict__ v_src,
+// FIXED: forms 1 and 2 (one decay a head, kept in a register), BONUS: form 3
+template <int RPT, int kCols, bool FIXED, bool BONUS, int MAXT>
+__global__ void __launch_bounds__(MAXT, MAXT == 256 && RPT == 8 ? 3 : 1) gated_recurrence_kernel(const float* __restrict__ q_src, const float* __restrict__ f_src, const float* __restrict__ v_src,
                                         int P, size_t stride_p, int R, const float* __restrict__ f_bias,
                                         const float* __restrict__ lower, float* __restrict__ state, size_t slot_stride, const int* __restrict__ seg_start,
                                         const int* __restrict__ seg_slot, float* __restrict__ o_out, int heads, int D, int V, int DS,
@@ -83,6 +85,7 @@ __global__ void __launch_bounds__(kCols * 16) gated_recurrence_kernel(const floa
     st[r][1] = (!chunks && d < D && j + 1 < V) ? S[(size_t)d * V + j + 1] : 0.f;
   }
   const int q_off = a * D, v_off = a * V + j0;
+  const float fixed = FIXED ? lower[a] : 0.f;
   float u[BONUS ? RPT : 1];
   if constexpr (BONUS) {
 #pragma unroll
@@ -91,82 +94,140 @@ __global__ void __launch_bounds__(kCols * 16) gated_recurrence_kernel(const floa
   for (int c0 = t0; c0 < t1; c0 += kChunk) {
     const int n = min(kChunk, t1 - c0);
     __syncthreads();
-    if (!BONUS && form == 2) {   // a thread takes a pair of entries that are turned together, or one that is not
-      const int half = ex.rot_half, per = D - half;
-      for (int i = tid; i < n * per; i += blockDim.x) {
-        const int tt = i / per, w = i % per;
-        const size_t row = (size_t)(c0 + tt) * R + q_off;
-        const int d = w < half ? w : w + half, d2 = w + half;
-        float zq = q_src[row + d], zk = f_src[row + d];
-        for (int p = 1; p < P; p++) zq += q_src[p * stride_p + row + d], zk += f_src[p * stride_p + row + d];
-        if (w < half) {
-          float yq = q_src[row + d2], yk = f_src[row + d2];
-          for (int p = 1; p < P; p++) yq += q_src[p * stride_p + row + d2], yk += f_src[p * stride_p + row + d2];
-          const float c = ex.cos_t[(size_t)(c0 + tt) * half + w], s = ex.sin_t[(size_t)(c0 + tt) * half + w];
-          sq[tt * D + d2] = yq * c + zq * s;
-          sg[tt * D + d2] = (yk * c + zk * s) * ex.k_scale;
-          sf[tt * D + d2] = lower[a];
-          zq = zq * c - yq * s, zk = zk * c - yk * s;
+    // The sixteen tokens' rows into shared memory: every thread requests its values of kLoads items before it uses the first.
+    const int step = kLoads * blockDim.x;
+    if (FIXED && form == 2) {   // an item is a pair of entries that are turned together, or one that is not
+      const int half = ex.rot_half, per = D - half, items = n * per;
+      for (int i0 = tid; i0 < items; i0 += step) {
+        float zq[kLoads], zk[kLoads], yq[kLoads], yk[kLoads], c[kLoads], sn[kLoads];
+#pragma unroll
+        for (int e = 0; e < kLoads; e++) {
+          const int i = i0 + e * (int)blockDim.x;
+          zq[e] = zk[e] = yq[e] = yk[e] = c[e] = sn[e] = 0.f;
+          if (i >= items) continue;
+          const int tt = i / per, w = i % per;
+          const size_t at = (size_t)(c0 + tt) * R + q_off + (w < half ? w : w + half);
+          zq[e] = q_src[at], zk[e] = f_src[at];
+          if (w < half) {
+            yq[e] = q_src[at + half], yk[e] = f_src[at + half];
+            c[e] = ex.cos_t[(size_t)(c0 + tt) * half + w], sn[e] = ex.sin_t[(size_t)(c0 + tt) * half + w];
+          }
         }
-        sq[tt * D + d] = zq;
-        sg[tt * D + d] = zk * ex.k_scale;
-        sf[tt * D + d] = lower[a];
+        for (int p = 1; p < P; p++) {
+#pragma unroll
+          for (int e = 0; e < kLoads; e++) {
+            const int i = i0 + e * (int)blockDim.x;
+            if (i >= items) continue;
+            const int tt = i / per, w = i % per;
+            const size_t at = p * stride_p + (size_t)(c0 + tt) * R + q_off + (w < half ? w : w + half);
+            zq[e] += q_src[at], zk[e] += f_src[at];
+            if (w < half) yq[e] += q_src[at + half], yk[e] += f_src[at + half];
+          }
+        }
+#pragma unroll
+        for (int e = 0; e < kLoads; e++) {
+          const int i = i0 + e * (int)blockDim.x;
+          if (i >= items) continue;
+          const int tt = i / per, w = i % per;
+          float q = zq[e], k = zk[e];
+          if (w < half) {
+            sq[tt * D + w + half] = yq[e] * c[e] + zq[e] * sn[e];
+            sg[tt * D + w + half] = (yk[e] * c[e] + zk[e] * sn[e]) * ex.k_scale;
+            q = zq[e] * c[e] - yq[e] * sn[e], k = zk[e] * c[e] - yk[e] * sn[e];
+          }
+          const int d = w < half ? w : w + half;
+          sq[tt * D + d] = q;
+          sg[tt * D + d] = k * ex.k_scale;
+        }
       }
-    } else
-    for (int i = tid; i < n * D; i += blockDim.x) {
-      const int tt = i / D, d = i % D;
-      const size_t row = (size_t)(c0 + tt) * R + q_off + d;
-      float zq = q_src[row], zf = f_src[row];
-      for (int p = 1; p < P; p++) zq += q_src[p * stride_p + row], zf += f_src[p * stride_p + row];
-      if constexpr (BONUS) {
-        sq[i] = zq;
-        sg[i] = zf;
-        sf[i] = ex.decay[(size_t)(c0 + tt) * heads * D + q_off + d];
-        continue;
-      }
-      sq[i] = zq / (1.f + expf(-zq));
-      if (form == 1) {
-        sf[i] = lower[a];
-        sg[i] = zf / (1.f + expf(-zf));
-      } else {
-        zf += f_bias[a * D + d];
-        const float lo = lower[a * D + d];
-        const float sig = 1.f / (1.f + expf(-zf));
-        const float f = __fmaf_rn(1.f - lo, sig, lo);
-        sf[i] = f;
-        sg[i] = 1.f - f;
+    } else {
+      const int items = n * D;
+      for (int i0 = tid; i0 < items; i0 += step) {
+        float zq[kLoads], zf[kLoads], dc[kLoads];
+#pragma unroll
+        for (int e = 0; e < kLoads; e++) {
+          const int i = i0 + e * (int)blockDim.x;
+          zq[e] = zf[e] = dc[e] = 0.f;
+          if (i >= items) continue;
+          const int tt = i / D, d = i % D;
+          const size_t at = (size_t)(c0 + tt) * R + q_off + d;
+          zq[e] = q_src[at], zf[e] = f_src[at];
+          if (BONUS) dc[e] = ex.decay[(size_t)(c0 + tt) * heads * D + q_off + d];
+        }
+        for (int p = 1; p < P; p++) {
+#pragma unroll
+          for (int e = 0; e < kLoads; e++) {
+            const int i = i0 + e * (int)blockDim.x;
+            if (i >= items) continue;
+            const size_t at = p * stride_p + (size_t)(c0 + i / D) * R + q_off + i % D;
+            zq[e] += q_src[at], zf[e] += f_src[at];
+          }
+        }
+#pragma unroll
+        for (int e = 0; e < kLoads; e++) {
+          const int i = i0 + e * (int)blockDim.x;
+          if (i >= items) continue;
+          if constexpr (BONUS) {
+            sq[i] = zq[e];
+            sg[i] = zf[e];
+            sf[i] = dc[e];
+          } else if constexpr (FIXED) {
+            sq[i] = zq[e] / (1.f + expf(-zq[e]));
+            sg[i] = zf[e] / (1.f + expf(-zf[e]));
+          } else {
+            sq[i] = zq[e] / (1.f + expf(-zq[e]));
+            const int d = i % D;
+            const float z = zf[e] + f_bias[a * D + d];
+            const float lo = lower[a * D + d];
+            const float sig = 1.f / (1.f + expf(-z));
+            const float f = __fmaf_rn(1.f - lo, sig, lo);
+            sf[i] = f;
+            sg[i] = 1.f - f;
+          }
+        }
       }
     }
-    for (int i = tid; i < n * kCols; i += blockDim.x) {
-      const int tt = i / kCols, c = i % kCols;
-      float z = 0.f;
-      if (j0 + c < V) {
-        const float* src = v_src + (size_t)(c0 + tt) * R + v_off + c;
-        z = src[0];
-        for (int p = 1; p < P; p++) z += src[p * stride_p];
-        if (form == 1) z = z / (1.f + expf(-z));
+    for (int i0 = tid; i0 < n * kCols; i0 += step) {
+      float z[kLoads];
+#pragma unroll
+      for (int e = 0; e < kLoads; e++) {
+        const int i = i0 + e * (int)blockDim.x, c = i % kCols;
+        z[e] = (i < n * kCols && j0 + c < V) ? v_src[(size_t)(c0 + i / kCols) * R + v_off + c] : 0.f;
       }
-      sv[i] = z;
+      for (int p = 1; p < P; p++) {
+#pragma unroll
+        for (int e = 0; e < kLoads; e++) {
+          const int i = i0 + e * (int)blockDim.x, c = i % kCols;
+          if (i < n * kCols && j0 + c < V) z[e] += v_src[p * stride_p + (size_t)(c0 + i / kCols) * R + v_off + c];
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < kLoads; e++) {
+        const int i = i0 + e * (int)blockDim.x;
+        if (i < n * kCols) sv[i] = FIXED && form == 1 ? z[e] / (1.f + expf(-z[e])) : z[e];
+      }
     }
     __syncthreads();
     if (chunks && blockIdx.z == 0) {   // q times the decay since the chunk's start, for the pass that adds the incoming state's share
       for (int d = tid; d < D; d += blockDim.x) {
         float r = run[d];
         for (int tt = 0; tt < n; tt++) {
-          if (!BONUS) r *= sf[tt * D + d];
+          if (!BONUS) r *= FIXED ? fixed : sf[tt * D + d];
           qa_out[((size_t)(c0 + tt) * heads + a) * D + d] = sq[tt * D + d] * r;
           if (BONUS) r *= sf[tt * D + d];   // the current token's decay comes after its output
         }
         run[d] = r;
       }
     }
-    for (int tt = 0; tt < n; tt++) {
+    // one token: the thread's rows of the state advance, acc0 and acc1 receive its share of o for its two columns
+    auto advance = [&](int tt, float& acc0, float& acc1) {
       const float v0 = sv[tt * kCols + col], v1 = sv[tt * kCols + col + 1];
       float f[RPT], g[RPT], q[RPT];
       if (d4 && d0 + RPT <= D) {   // this thread's rows are whole groups of four: 16-byte reads
 #pragma unroll
         for (int r = 0; r < RPT; r += 4) {
-          const float4 a = *(const float4*)(sf + tt * D + d0 + r), b = *(const float4*)(sg + tt * D + d0 + r), c = *(const float4*)(sq + tt * D + d0 + r);
+          const float4 b = *(const float4*)(sg + tt * D + d0 + r), c = *(const float4*)(sq + tt * D + d0 + r);
+          const float4 a = FIXED ? make_float4(fixed, fixed, fixed, fixed) : *(const float4*)(sf + tt * D + d0 + r);
           f[r] = a.x, f[r + 1] = a.y, f[r + 2] = a.z, f[r + 3] = a.w;
           g[r] = b.x, g[r + 1] = b.y, g[r + 2] = b.z, g[r + 3] = b.w;
           q[r] = c.x, q[r + 1] = c.y, q[r + 2] = c.z, q[r + 3] = c.w;
@@ -176,10 +237,10 @@ __global__ void __launch_bounds__(kCols * 16) gated_recurrence_kernel(const floa
         for (int r = 0; r < RPT; r++) {
           const int d = d0 + r;
           const bool in = d < D;
-          f[r] = in ? sf[tt * D + d] : 0.f, g[r] = in ? sg[tt * D + d] : 0.f, q[r] = in ? sq[tt * D + d] : 0.f;
+          f[r] = FIXED ? fixed : in ? sf[tt * D + d] : 0.f, g[r] = in ? sg[tt * D + d] : 0.f, q[r] = in ? sq[tt * D + d] : 0.f;
         }
       }
-      float acc0 = 0.f, acc1 = 0.f;
+      acc0 = acc1 = 0.f;
       if constexpr (BONUS) {
         float own = 0.f;   // this thread's rows of r . (u k)
 #pragma unroll
@@ -192,14 +253,51 @@ __global__ void __launch_bounds__(kCols * 16) gated_recurrence_kernel(const floa
         }
         acc0 = __fmaf_rn(own, v0, acc0);
         acc1 = __fmaf_rn(own, v1, acc1);
-      } else
+      } else {
 #pragma unroll
-      for (int r = 0; r < RPT; r++) {   // rows beyond D have f = g = q = 0: their state stays zero
-        st[r][0] = __fmaf_rn(f[r], st[r][0], g[r] * v0);
-        st[r][1] = __fmaf_rn(f[r], st[r][1], g[r] * v1);
-        acc0 = __fmaf_rn(st[r][0], q[r], acc0);
-        acc1 = __fmaf_rn(st[r][1], q[r], acc1);
+        for (int r = 0; r < RPT; r++) {   // rows beyond D have f = g = q = 0: their state stays zero
+          st[r][0] = __fmaf_rn(f[r], st[r][0], g[r] * v0);
+          st[r][1] = __fmaf_rn(f[r], st[r][1], g[r] * v1);
+          acc0 = __fmaf_rn(st[r][0], q[r], acc0);
+          acc1 = __fmaf_rn(st[r][1], q[r], acc1);
+        }
       }
+    };
+    int tt = 0;
+    // Eight tokens at a time: their sixteen sums per thread are reduced over the DS threads of the column pair together, each exchange halving
+    // what a lane still holds (15 shuffles for eight tokens and DS = 16 instead of 64; the pairs that are added, and so the bits, are those of
+    // the token-by-token reduction).
+    for (; tt + kGroup <= n; tt += kGroup) {
+      float acc[2 * kGroup];
+#pragma unroll
+      for (int k = 0; k < kGroup; k++) advance(tt + k, acc[2 * k], acc[2 * k + 1]);
+      int o = DS >> 1, first = 0;   // first: number of the sum that acc[0] ends up with
+#pragma unroll
+      for (int half = kGroup; half >= 1; half >>= 1) {
+        if (o > 0) {
+          const bool up = ds & o;
+#pragma unroll
+          for (int i = 0; i < half; i++) {
+            const float give = up ? acc[i] : acc[i + half], keep = up ? acc[i + half] : acc[i];
+            acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+          }
+          first += up ? half : 0;
+          o >>= 1;
+        }
+      }
+      for (; o > 0; o >>= 1) acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], o);   // more lanes than sums
+      if (DS <= 2 * kGroup || (ds & (DS / (2 * kGroup) - 1)) == 0) {
+        const int held = DS >= 2 * kGroup ? 1 : 2 * kGroup / DS;
+#pragma unroll
+        for (int i = 0; i < kGroup; i++) {   // DS >= 2: at most kGroup sums a lane
+          const int m = first + i, c = m & 1;
+          if (i < held && j + c < V) o_out[((size_t)(c0 + tt + (m >> 1)) * heads + a) * V + j + c] = acc[i];
+        }
+      }
+    }
+    for (; tt < n; tt++) {
+      float acc0, acc1;
+      advance(tt, acc0, acc1);
       for (int o = DS >> 1; o > 0; o >>= 1) {
         acc0 += __shfl_xor_sync(0xffffffffu, acc0, o);
         acc1 += __shfl_xor_sync(0xffffffffu, acc1, o);
@@ -258,44 +356,57 @@ __global__ void chunk_carry_kernel(const int* __restrict__ long_segs, const int*
   }
 }
 
-// o[t][j] += sum_d qa[t][d] * S_in[d][j] for the rows of one chunk: a CTA of 256 threads takes 64 rows x 32 columns, 32 values of d at a time.
+// o[t][j] += sum_d qa[t][d] * S_in[d][j] for the rows of one chunk: a CTA of 256 threads takes 64 rows x 64 columns, 32 values of d at a time; a
+// thread owns 4 x 4 outputs, so a value of d costs it two 16-byte reads of shared memory for sixteen FMAs.
 __global__ void __launch_bounds__(256) chunk_apply_kernel(const int* __restrict__ chunks, const float* __restrict__ chunk_state, const float* __restrict__ qa,
                                                           float* __restrict__ o_out, int heads, int D, int V) {
-  __shared__ float s_in[32][33];
-  __shared__ float s_q[64][33];
+  __shared__ __align__(16) float s_in[32][64];
+  __shared__ __align__(16) float s_q[32][68];   // [d][row]
   ib::pdl_launch_dependents();
   ib::pdl_wait();
   const int t0 = chunks[2 * blockIdx.x], n = chunks[2 * blockIdx.x + 1];
-  const int a = blockIdx.y, j0 = blockIdx.z * 32;
-  const int tx = threadIdx.x & 31, ty = threadIdx.x >> 5;
+  const int a = blockIdx.y, j0 = blockIdx.z * 64;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;   // columns 4 tx .., rows 4 ty ..
   const float* Sin = chunk_state + ((size_t)blockIdx.x * heads + a) * D * V;
-  float acc[8];
+  float acc[4][4];
 #pragma unroll
-  for (int r = 0; r < 8; r++) acc[r] = 0.f;
+  for (int r = 0; r < 4; r++)
+#pragma unroll
+    for (int c = 0; c < 4; c++) acc[r][c] = 0.f;
   for (int d0 = 0; d0 < D; d0 += 32) {
-    __syncthreads();
-    for (int i = threadIdx.x; i < 32 * 32; i += 256) {
-      const int dd = i >> 5, c = i & 31;
-      s_in[dd][c] = (d0 + dd < D && j0 + c < V) ? Sin[(size_t)(d0 + dd) * V + j0 + c] : 0.f;
+    float in[8], q[8];
+#pragma unroll
+    for (int e = 0; e < 8; e++) {   // all sixteen values are requested before the first is stored
+      const int i = threadIdx.x + e * 256, dd = i >> 6, c = i & 63, tt = i >> 5, qd = i & 31;
+      in[e] = (d0 + dd < D && j0 + c < V) ? Sin[(size_t)(d0 + dd) * V + j0 + c] : 0.f;
+      q[e] = (tt < n && d0 + qd < D) ? qa[((size_t)(t0 + tt) * heads + a) * D + d0 + qd] : 0.f;
     }
-    for (int i = threadIdx.x; i < 64 * 32; i += 256) {
-      const int tt = i >> 5, dd = i & 31;
-      s_q[tt][dd] = (tt < n && d0 + dd < D) ? qa[((size_t)(t0 + tt) * heads + a) * D + d0 + dd] : 0.f;
+    __syncthreads();
+#pragma unroll
+    for (int e = 0; e < 8; e++) {
+      const int i = threadIdx.x + e * 256;
+      s_in[i >> 6][i & 63] = in[e];
+      s_q[i & 31][i >> 5] = q[e];
     }
     __syncthreads();
 #pragma unroll 8
     for (int dd = 0; dd < 32; dd++) {
-      const float sv = s_in[dd][tx];
+      const float4 v = *(const float4*)&s_in[dd][4 * tx], w = *(const float4*)&s_q[dd][4 * ty];
+      const float qv[4] = {w.x, w.y, w.z, w.w}, sv[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
-      for (int r = 0; r < 8; r++) acc[r] = __fmaf_rn(s_q[ty * 8 + r][dd], sv, acc[r]);
+      for (int r = 0; r < 4; r++)
+#pragma unroll
+        for (int c = 0; c < 4; c++) acc[r][c] = __fmaf_rn(qv[r], sv[c], acc[r][c]);
     }
   }
-  if (j0 + tx < V) {
 #pragma unroll
-    for (int r = 0; r < 8; r++) {
-      const int tt = ty * 8 + r;
-      if (tt < n) o_out[((size_t)(t0 + tt) * heads + a) * V + j0 + tx] += acc[r];
-    }
+  for (int r = 0; r < 4; r++) {
+    const int tt = 4 * ty + r;
+    if (tt >= n) continue;
+    float* dst = o_out + ((size_t)(t0 + tt) * heads + a) * V + j0 + 4 * tx;
+#pragma unroll
+    for (int c = 0; c < 4; c++)
+      if (j0 + 4 * tx + c < V) dst[c] += acc[r][c];
   }
 }
 
@@ -410,10 +521,15 @@ int launch_recurrence(const float* q_src, const float* f_src, const float* v_src
     ib::launch(kernel, grid, kCols / 2 * DS, smem, stream, q_src, f_src, v_src, P, (size_t)stride_p, R, f_bias, lower, state, (size_t)slot_stride, seg_start, seg_slot, o_out,
                heads, D, V, DS, seg_list, chunks, chunk_state, chunk_decay, qa, form, ex);
   };
-  if (rpt == 8 && form == 3) go(gated_recurrence_kernel<8, 32, true>);
-  else if (rpt == 8) go(gated_recurrence_kernel<8, 32, false>);
-  else if (form == 3) go(gated_recurrence_kernel<16, 16, true>);
-  else go(gated_recurrence_kernel<16, 16, false>);
+  auto pick = [&](auto fixed, auto bonus) {
+    constexpr bool F = decltype(fixed)::value, B = decltype(bonus)::value;
+    if (rpt == 8 && DS <= 16) go(gated_recurrence_kernel<8, 32, F, B, 256>);
+    else if (rpt == 8) go(gated_recurrence_kernel<8, 32, F, B, 512>);
+    else go(gated_recurrence_kernel<16, 16, F, B, 256>);
+  };
+  if (form == 3) pick(std::false_type(), std::true_type());
+  else if (form == 0) pick(std::false_type(), std::false_type());
+  else pick(std::true_type(), std::false_type());
   IB_CHECK_LAUNCH("recurrence");
   return 0;
 }
@@ -458,7 +574,7 @@ extern "C" int ib_recurrence_chunks_finish(const int* long_segs, int n_long, con
   ib::launch(chunk_carry_kernel, dim3((unsigned)n_long, (unsigned)heads, (unsigned)min((D * V + 255) / 256, 64)), 256, 0, stream, long_segs, seg_slot, state,
              (size_t)slot_stride, chunk_state, chunk_decay, heads, D, V);
   IB_CHECK_LAUNCH("recurrence chunk_carry");
-  ib::launch(chunk_apply_kernel, dim3((unsigned)n_chunks, (unsigned)heads, (unsigned)((V + 31) / 32)), 256, 0, stream, chunks, (const float*)chunk_state, qa, o_out, heads, D, V);
+  ib::launch(chunk_apply_kernel, dim3((unsigned)n_chunks, (unsigned)heads, (unsigned)((V + 63) / 64)), 256, 0, stream, chunks, (const float*)chunk_state, qa, o_out, heads, D, V);
   IB_CHECK_LAUNCH("recurrence chunk_apply");
   return 0;
 }
