@@ -420,13 +420,13 @@ DESIGN_SIZES = {
 }
 DESIGN_KINDS = {   # kinds of kernel by the library entry points that launch them
     "zabonex": {"attention": ["ib_latent_attention", "ib_latent_attention_mma"], "experts": ["ib_gemm_grouped", "ib_gemm_grouped_mma", "ib_gemm_grouped_tcgen05", "ib_gemm_grouped_swiglu_tcgen05", "ib_gather_rows"],
-                "heads": ["ib_gemm_heads", "ib_gemm_heads_mma"], "route": ["ib_moe_route", "ib_moe_sort", "ib_moe_combine"],
+                "heads": ["ib_gemm_heads", "ib_gemm_heads_mma"], "route": ["ib_moe_route", "ib_moe_sort", "ib_moe_route_sort", "ib_moe_combine"],
                 "norm": ["ib_norm_residual", "ib_latent_prepare", "ib_cast_rows"], "gemm": LEAVE_OUT["gemm"]},
     "qwen3": {"attention": LEAVE_OUT["attention"], "norm": LEAVE_OUT["norm"] + LEAVE_OUT["qk"], "gemm": LEAVE_OUT["gemm"] + LEAVE_OUT["qkv"]},
     "busadra": {"attention": ["ib_attention_generic", "ib_attention_decode_capped", "ib_attention_decode_stream_capped", "ib_attention_prefill_ws_capped"],
                 "recurrence": ["ib_gated_recurrence", "ib_recurrence_chunks_finish", "ib_head_rmsnorm"],
                 "experts": ["ib_gemm_grouped", "ib_gemm_grouped_mma", "ib_gemm_grouped_tcgen05", "ib_gemm_grouped_swiglu_tcgen05", "ib_scatter_scaled_rows"],
-                "route": ["ib_moe_route", "ib_moe_sort", "ib_moe_combine"],
+                "route": ["ib_moe_route", "ib_moe_sort", "ib_moe_route_sort", "ib_moe_combine"],
                 "norm": ["ib_add_layernorm", "ib_causal_conv_rows", "ib_add_layernorm_conv_single", "ib_depth_average", "ib_qk_norm_rope_kv"], "gemm": LEAVE_OUT["gemm"]},
     "lulenex": {"attention": ["ib_attention_generic", "ib_attention_decode_capped", "ib_attention_decode_stream_capped", "ib_attention_prefill_ws_capped"],
                 "recurrence": ["ib_gated_recurrence", "ib_recurrence_chunks_finish", "ib_gated_rmsnorm"],
@@ -443,7 +443,7 @@ DITALORN_SIZES = {
 DESIGN_KINDS["ditalorn"] = {
     "attention": ["ib_latent_attention", "ib_latent_attention_mma"], "sigmoid": ["ib_sigmoid_attention", "ib_sigmoid_attention_mma"],
     "experts": ["ib_gemm_grouped", "ib_gemm_grouped_mma", "ib_gemm_grouped_tcgen05", "ib_gemm_grouped_swiglu_tcgen05", "ib_gather_rows"],
-    "heads": ["ib_gemm_heads", "ib_gemm_heads_mma"], "route": ["ib_moe_route", "ib_moe_sort", "ib_moe_combine"],
+    "heads": ["ib_gemm_heads", "ib_gemm_heads_mma"], "route": ["ib_moe_route", "ib_moe_sort", "ib_moe_route_sort", "ib_moe_combine"],
     "norm": ["ib_add_rmsnorm", "ib_post_norm", "ib_latent_down", "ib_latent_prepare", "ib_qkv_conv", "ib_embed_pos"], "gemm": LEAVE_OUT["gemm"]}
 
 
@@ -613,11 +613,10 @@ FEDIPEL_SIZES = {
     "mid": dict(BUSADRA_SIZES["mid"], att_heads=16, att_kv_heads=4, map_dim=64, att_vdim=128, keep=4, wkv_heads=32, wkv_dim=64, decay_rank=64, shared_ff=2816),
 }
 DESIGN_KINDS["fedipel"] = {
-    "attention": ["ib_attention_generic", "ib_attention_decode_capped", "ib_attention_decode_stream_capped", "ib_attention_prefill_ws_capped", "ib_attention_decode_maps",
-                  "ib_attention_prefill_maps"],
+    "attention": ["ib_attention_generic", "ib_attention_decode_capped", "ib_attention_decode_stream_capped", "ib_attention_prefill_ws_capped"],
     "recurrence": ["ib_recurrence_parts", "ib_recurrence_chunks_finish", "ib_head_norm_gate"],
     "experts": ["ib_gemm_grouped", "ib_gemm_grouped_mma", "ib_gemm_grouped_tcgen05", "ib_gemm_grouped_relu2_tcgen05", "ib_gather_rows"],
-    "route": ["ib_moe_route", "ib_moe_sort", "ib_moe_combine"],
+    "route": ["ib_moe_route", "ib_moe_sort", "ib_moe_route_sort", "ib_moe_combine"],
     "norm": ["ib_add_layernorm", "ib_add_layernorm_mixes_single", "ib_shift_mixes", "ib_decay_rows", "ib_map_qkv", "ib_diff_combine", "ib_embed_layernorm"],
     "gemm": LEAVE_OUT["gemm"] + ["ib_gemm_relu2_tcgen05", "ib_gemm_relu2_tcgen05_2cta", "ib_relu2_rows", "ib_gemm_parts_tcgen05"]}
 
