@@ -459,6 +459,7 @@ __global__ void __launch_bounds__((kWarps + 1) * 32, 2)
                          float* __restrict__ part_ml, int heads, int n_dec, int max_slices, int tiles_per_slice, int merge_cols,
                          const __grid_constant__ CUtensorMap kv_map, long long view_row0, unsigned long long wait_ns, unsigned* __restrict__ status,
                          float cap_pre, int keep) {
+  if constexpr (FUSED) keep = 0;   // (the launcher refuses anything else)
   constexpr int CPR = HD / 8;
   constexpr int TILE = kTile * HD * 2;
   constexpr int HB = HD / 64;

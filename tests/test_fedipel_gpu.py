@@ -208,6 +208,79 @@ def test_the_difference_of_two_maps(rt32, dtype, T, heads, vdim):
     assert torch.allclose(out.cpu().double().view(T, heads, vdim), want, **(dict(atol=2e-6) if dtype == torch.float32 else dict(rtol=2.0 ** -7, atol=1e-6)))
 
 
+@pytest.mark.parametrize("heads,kv_heads,dim,page,window,keep", [(4, 2, 64, 16, 48, 5), (16, 1, 128, 16, 100, 20), (6, 3, 128, 64, 1000, 3), (2, 1, 64, 64, None, 0), (4, 2, 24, 8, 13, 40)])
+@pytest.mark.parametrize("portion", [0, 5])
+def test_the_difference_of_two_maps_where_the_slices_are_merged(rt16, heads, kv_heads, dim, page, window, keep, portion):
+    """Decoded tokens from the first positions to a long context, alone (the merge kernel takes the difference and the norm) and beside a prompt
+    portion (a kernel of its own does)."""
+    from inference_bench_b200.kernels import attention
+    from inference_bench_b200.kernels.ops import KvLayerView
+    n_ctx, scale, lam, eps, factor = 700, 0.3, 0.6, 1e-5, 0.45
+    g = torch.Generator().manual_seed(heads + dim)
+    runs = [(0, 1), (1, 1), (keep + 60, 1), (333, 1), (699, 1)] + ([(20, portion)] if portion else [])
+    positions = [p0 + i for p0, n in runs for i in range(n)]
+    n_pages = -(-n_ctx // page)
+    perm = torch.randperm(n_pages, generator=g)
+    k, v, q = (torch.randn((n_ctx, h, dim), generator=g).to(torch.bfloat16).double() for h in (kv_heads, kv_heads, heads))
+    pool = torch.zeros((1, n_pages, 2, kv_heads, page, dim), dtype=torch.bfloat16, device=DEV)
+    for j in range(n_ctx):
+        pool[0, perm[j // page], 0, :, j % page] = k[j].to(torch.bfloat16)
+        pool[0, perm[j // page], 1, :, j % page] = v[j].to(torch.bfloat16)
+    a = P.masked_attention(q, k, v, P.visible(n_ctx, None if window is None else {"size": window, "keep_first": keep}), scale)[positions].view(len(positions), heads // 2, 2, dim)
+    want = P.rms_unit(a[:, :, 0] - lam * a[:, :, 1], eps) * factor
+    ctx = _ctx(rt16, runs)
+    view = KvLayerView(pool, 0, perm.to(torch.int32).reshape(1, -1).repeat(len(runs), 1).contiguous().to(DEV))
+    out = attention.paged_attention(ctx, q[positions].reshape(len(positions), heads * dim).to(DEV, torch.bfloat16).contiguous(), view, heads, window, scale, keep_first=keep,
+                                    diff=(lam, eps, factor))
+    err = (out.cpu().double().view(want.shape) - want).abs().amax(dim=(1, 2))
+    assert err.max().item() < 4e-2, f"positions {[positions[i] for i in torch.nonzero(err >= 4e-2).flatten().tolist()]}: {err.max().item():.2e}"
+    rt16.check_status()
+
+
+@pytest.mark.parametrize("parts,T,N,K", [(4, 1, 192, 192), (4, 8, 1024, 1024), (3, 17, 60, 72), (2, 128, 130, 520), (4, 64, 2048, 2048)])
+def test_several_products_in_one_launch(rt16, parts, T, N, K):
+    from inference_bench_b200.kernels import gemm_tcgen05 as G
+    g = torch.Generator().manual_seed(T + N)
+    x, w = (torch.randn(s, generator=g).to(torch.bfloat16) for s in ((parts, T, K), (parts, N, K)))
+    out = G.gemm_parts(rt16, x.to(DEV), w.to(DEV)).sum(0).cpu().double()
+    want = torch.einsum("ptk,pnk->ptn", x.double(), w.double())
+    assert (out - want).abs().max().item() < 1e-4 * want.abs().max().item()
+    rt16.check_status()
+
+
+@pytest.mark.parametrize("T,E,groups,keep,top,score,always", [(1, 1, 1, 1, 1, "chosen_softmax", 1), (8, 64, 1, 1, 6, "chosen_softmax", 2), (32, 16, 4, 2, 3, "sigmoid", 0), (5, 40, 1, 1, 40, "softmax", 3),
+                                                              (31, 6, 1, 1, 2, "chosen_softmax", 0)])
+def test_choice_and_regrouping_in_one_kernel(rt32, T, E, groups, keep, top, score, always):
+    """The same choices and weights as the router's own kernel, and rows that lie in their expert's range, each pair in one of its own."""
+    from inference_bench_b200.kernels import ops
+    g = torch.Generator().manual_seed(T + E)
+    logits, bias = _f32(torch.randn((2, T, E + 1), generator=g)), _f32(torch.randn((E,), generator=g))
+    R, n = T * (top + always), E + always
+    new = lambda *shape: torch.empty(shape, dtype=torch.int32, device=DEV)
+    got = []
+    for fused in (False, True):
+        idx, wt, off, tiles, row, tok = new(T, top + always), torch.empty((T, top + always), device=DEV), new(n + 1), new(n + 1), new(R), new(R)
+        ops.moe_route(logits, groups, keep, top, 1.5, score == "softmax", idx, wt, score, experts=E, logit_bias=bias, always=always, gate_col=E if always else -1,
+                      sort=(off, tiles, row, tok, 16) if fused else None)
+        if not fused:
+            ops.moe_sort(idx, n, off, tiles, row, tok, tile_rows=16)
+        got.append([t.cpu() for t in (idx, wt, off, tiles)])
+        idx, off, row, tok = idx.cpu().flatten(), off.cpu(), row.cpu(), tok.cpu()
+        assert sorted(row.tolist()) == list(range(R)) and int(off[-1]) == R
+        for pair in range(R):
+            e = int(idx[pair])
+            assert off[e] <= row[pair] < off[e + 1] and int(tok[row[pair]]) == pair // (top + always)
+    for a, b in zip(*got):
+        assert torch.equal(a, b)
+    z = logits.cpu().double().sum(0)
+    if always:
+        assert torch.allclose(got[0][1][:, top:].double(), torch.sigmoid(z[:, E:]).expand(T, always), atol=1e-6)
+    if score == "chosen_softmax":
+        best = torch.topk(z[:, :E] + bias.cpu().double(), top).values
+        assert torch.allclose(got[0][1][:, :top].double(), 1.5 * torch.softmax(best, -1), atol=1e-5)
+    rt32.check_status()
+
+
 # ------------------------------------------------------------------------------------------ recurrences over portions and slots
 def _walk_part(rt, plan, part, mixer, want_fn, W, caches, zero, run, tol):
     g = torch.Generator().manual_seed(W)
