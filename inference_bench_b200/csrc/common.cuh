@@ -37,6 +37,7 @@ int ib_set_error(const char* fmt, ...);
 // that an earlier kernel writes, nor write memory at all.
 extern "C" int ib_pdl_enabled();
 extern "C" void ib_set_pdl(int on);
+extern "C" void ib_pdl_skip_next();   // the next kernel is launched without it: it starts when everything before it in the stream is done
 
 // How long a bounded wait inside a kernel (on an mbarrier) may last before the kernel gives up, sets
 // IB_ERR_WAIT_TIMEOUT in the status word and unwinds. Launchers pass it to their kernels as an argument.
@@ -94,6 +95,16 @@ __device__ __forceinline__ float xielu(float z, float ap, float an) {
 __device__ __forceinline__ float relu2(float z) {   // the square of max(z, 0)
   const float r = fmaxf(z, 0.f);
   return r * r;
+}
+
+// A gated pair with clamped halves: g' sigmoid(slope g') (u' + 1) with g' = min(g, limit) and u' = u cut to [-limit, limit]. FAST: the
+// approximate exponential and division (results that are rounded to bfloat16).
+template <bool FAST>
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit, float slope) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit) + 1.f;
+  if constexpr (FAST) return __fdividef(g, 1.f + __expf(-slope * g)) * u;
+  else return g / (1.f + expf(-slope * g)) * u;
 }
 
 __device__ __forceinline__ float warp_sum(float v) {

@@ -21,7 +21,15 @@ int ib_set_error(const char* fmt, ...) {
 }
 
 static int g_pdl = 1;
-extern "C" int ib_pdl_enabled() { return g_pdl; }
+static int g_pdl_skip = 0;
+extern "C" int ib_pdl_enabled() {
+  if (g_pdl_skip) {
+    g_pdl_skip = 0;
+    return 0;
+  }
+  return g_pdl;
+}
+extern "C" void ib_pdl_skip_next() { g_pdl_skip = 1; }
 extern "C" void ib_set_pdl(int on) { g_pdl = on ? 1 : 0; }
 
 static unsigned long long g_wait_limit_ns = 2000000000ull;  // 2 s
@@ -245,10 +253,10 @@ __global__ void __launch_bounds__(128) add_rmsnorm_rows_kernel(float* __restrict
 }
 
 // ---------------------------------------------------------------- rotation tables
-// cos/sin[t][i] of angle = float(position[t]) * inv_freq[i], float32 throughout
+// amplitude times cos/sin[t][i] of angle = float(position[t]) * inv_freq[i], float32 throughout
 // (crates/kir/tests/golden/attention/RopeKvWrite_bf16x2_sm120.cu:32-35).
 __global__ void rope_table_kernel(const int* __restrict__ positions, const float* __restrict__ inv_freq, float* __restrict__ cos_t,
-                                  float* __restrict__ sin_t, int T, int half) {
+                                  float* __restrict__ sin_t, int T, int half, float amplitude) {
   ib::pdl_launch_dependents();
   ib::pdl_wait();
   int idx = blockIdx.x * blockDim.x + threadIdx.x;
@@ -257,14 +265,15 @@ __global__ void rope_table_kernel(const int* __restrict__ positions, const float
   float ang = (float)positions[t] * inv_freq[i];
   float s, c;
   sincosf(ang, &s, &c);
-  cos_t[idx] = c;
-  sin_t[idx] = s;
+  cos_t[idx] = c * amplitude;
+  sin_t[idx] = s * amplitude;
 }
 
 // ---------------------------------------------------------------- SiLU-mul
-// gu[p][t][0:I] = gate, gu[p][t][I:2I] = up (partials summed first); act = g / (1 + exp(-g)) * u.
+// gu[p][t][0:I] = gate, gu[p][t][I:2I] = up (partials summed first); act = g / (1 + exp(-g)) * u, or with a limit the
+// pair with clamped halves (ib::clamped_glu).
 template <typename O>
-__global__ void silu_mul_kernel(const float* __restrict__ gu, int P, size_t stride, O* __restrict__ act, int I) {
+__global__ void silu_mul_kernel(const float* __restrict__ gu, int P, size_t stride, O* __restrict__ act, int I, const float* __restrict__ limit, float slope) {
   ib::pdl_launch_dependents();
   ib::pdl_wait();
   int t = blockIdx.y;
@@ -275,7 +284,7 @@ __global__ void silu_mul_kernel(const float* __restrict__ gu, int P, size_t stri
       g += row[p * stride + i];
       u += row[p * stride + I + i];
     }
-    act[(size_t)t * I + i] = ib::from_f32<O>((g / (1.f + expf(-g))) * u);
+    act[(size_t)t * I + i] = ib::from_f32<O>(limit ? ib::clamped_glu<false>(g, u, limit[0], slope) : (g / (1.f + expf(-g))) * u);
   }
 }
 
@@ -449,26 +458,26 @@ extern "C" int ib_add_rmsnorm(float* x, const float* delta, int P, long long del
   return 0;
 }
 
-extern "C" int ib_rope_table(const int* positions, const float* inv_freq, float* cos_t, float* sin_t, int T, int half,
+extern "C" int ib_rope_table(const int* positions, const float* inv_freq, float* cos_t, float* sin_t, int T, int half, float amplitude,
                              cudaStream_t stream) {
   if (T == 0 || half == 0) return 0;
   IB_CHECK_ARG(T > 0 && half > 0, "rope_table: bad sizes T=%d half=%d", T, half);
   long long n = (long long)T * half;
-  ib::launch(rope_table_kernel, (unsigned)((n + 255) / 256), 256, 0, stream, positions, inv_freq, cos_t, sin_t, T, half);
+  ib::launch(rope_table_kernel, (unsigned)((n + 255) / 256), 256, 0, stream, positions, inv_freq, cos_t, sin_t, T, half, amplitude);
   IB_CHECK_LAUNCH("rope_table");
   return 0;
 }
 
-extern "C" int ib_silu_mul(const float* gu, int P, long long stride, void* act, int act_dtype, int T, int I, cudaStream_t stream) {
+extern "C" int ib_silu_mul(const float* gu, int P, long long stride, void* act, int act_dtype, int T, int I, const float* limit, float slope, cudaStream_t stream) {
   if (T == 0) return 0;
   IB_CHECK_ARG(T > 0 && I > 0 && P >= 1, "silu_mul: bad sizes T=%d I=%d P=%d", T, I, P);
   IB_CHECK_ARG(T <= 65535, "silu_mul: T=%d rows exceed the grid limit 65535", T);
   dim3 grid((I + 255) / 256, T);
   if (grid.x > 64) grid.x = 64;
   if (act_dtype == IB_F32)
-    ib::launch(silu_mul_kernel<float>, grid, 256, 0, stream, gu, P, (size_t)stride, (float*)act, I);
+    ib::launch(silu_mul_kernel<float>, grid, 256, 0, stream, gu, P, (size_t)stride, (float*)act, I, limit, slope);
   else if (act_dtype == IB_BF16)
-    ib::launch(silu_mul_kernel<__nv_bfloat16>, grid, 256, 0, stream, gu, P, (size_t)stride, (__nv_bfloat16*)act, I);
+    ib::launch(silu_mul_kernel<__nv_bfloat16>, grid, 256, 0, stream, gu, P, (size_t)stride, (__nv_bfloat16*)act, I, limit, slope);
   else
     return ib_set_error("silu_mul: unknown output dtype %d", act_dtype);
   IB_CHECK_LAUNCH("silu_mul");

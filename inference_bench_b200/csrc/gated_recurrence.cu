@@ -16,6 +16,12 @@
 //  * Other forms of the same walk: a fixed decay per head with a key (form 1: q, k, v behind a SiLU; form 2: q and k turned by the token's
 //    angles, the key scaled, v as it is), and a decay per channel and token with a bonus for the current token (form 3:
 //    o = (S + diag(u) k v^T)^T r before S <- diag(w) S + k v^T).
+//  * Form 4, the matrix memory with exponential gates (mLSTM): log gates i, f per head and token, a running maximum m_t = max(f + m_(t-1), i), and
+//    S <- e^(f + m_(t-1) - m_t) S + e^(i - m_t) k v^T. The normaliser n (the same with k alone) is one more column of S whose value is always one,
+//    so a head's state is [D][V + 1] and o's last entry is n . q. memory_gates makes the two factors and e^(-m_t) for whole segments (the running
+//    maximum is a scan over pairs m -> max(m + a, b), so a CTA takes 256 tokens at a time); in a step of single tokens every CTA of the walk makes
+//    its own from the state's m, which memory_out then moves on.
+//  * memory_out: o / (max(|n . q|, e^(-m)) + 1e-6), the norm over the head, a weight per channel of all heads, the sigmoid of the gate.
 //  * decay_rows: the decays of form 3, exp(-exp(w0 + W2 tanh(low))), from the float32 sums of the low-rank projection.
 //  * head_norm_gate: out[t, a, :] = w * o / sqrt(mean(o^2) + eps) * silu(gate), the weight (optional) and the gate per channel of all heads.
 //  * head_rmsnorm: out[t, a, :] = w * o[t, a, :] / sqrt(mean(o^2) + eps), into the activation dtype.
@@ -23,11 +29,36 @@
 
 #include "common.cuh"
 
+// Where form 4's gates come from: float32 partial sums of the gates' pre-activations (rows of `row` entries, P of them stride apart, offset to the
+// first head's column), a bias a head, the cap (cap tanh(z / cap)), and the running maxima float32 [slots][heads], m_stride apart.
+struct IbMemoryGates {
+  const float* i_src;
+  const float* f_src;
+  int P, row;
+  size_t stride;
+  const float* i_bias;
+  const float* f_bias;
+  float cap;
+  float* m_state;
+  size_t m_stride;
+};
+
 namespace {
 
 constexpr int kChunk = 16;   // tokens prepared at a time
 constexpr int kLoads = 4;    // values a thread requests at a time while it prepares tokens
 constexpr int kGroup = 8;    // tokens whose outputs are reduced together
+
+// (log input gate, log forget gate) of token t and head a: cap tanh(z / cap), and logsigmoid(cap tanh(z / cap)) = -log(1 + e^(-x)).
+__device__ __forceinline__ float2 log_gates(const IbMemoryGates& g, int t, int a) {
+  const float* si = g.i_src + (size_t)t * g.row + a;
+  const float* sf = g.f_src + (size_t)t * g.row + a;
+  float zi = si[0], zf = sf[0];
+  for (int p = 1; p < g.P; p++) zi += si[p * g.stride], zf += sf[p * g.stride];
+  zi = g.cap * tanhf((zi + g.i_bias[a]) / g.cap);
+  zf = g.cap * tanhf((zf + g.f_bias[a]) / g.cap);
+  return make_float2(zi, fminf(zf, 0.f) - log1pf(expf(-fabsf(zf))));
+}
 
 // RPT: rows of S a thread holds (for each of its two columns); kCols: value columns per CTA (32, or 16 where a thread holds sixteen rows)
 struct RecurrenceExtras {
@@ -36,10 +67,12 @@ struct RecurrenceExtras {
   int rot_half;
   float k_scale;        // form 2: factor on the key after the rotation
   const float* decay;   // form 3: float32 [T][heads * D]
+  const float2* gates;  // form 4: per token and head (factor on the state, factor on the key), or null: one token a segment, gates made here from
+  IbMemoryGates mg;       //   mg and the states' running maxima
 };
 
-// FIXED: forms 1 and 2 (one decay a head, kept in a register), BONUS: form 3
-template <int RPT, int kCols, bool FIXED, bool BONUS, int MAXT>
+// FIXED: forms 1 and 2 (one decay a head, kept in a register), BONUS: form 3, both: form 4 (one decay a head and token, in shared memory)
+template <int RPT, int kCols, bool FIXED_, bool BONUS_, int MAXT>
 __global__ void __launch_bounds__(MAXT, MAXT == 256 && RPT == 8 ? 3 : 1) gated_recurrence_kernel(const float* __restrict__ q_src, const float* __restrict__ f_src, const float* __restrict__ v_src,
                                         int P, size_t stride_p, int R, const float* __restrict__ f_bias,
                                         const float* __restrict__ lower, float* __restrict__ state, size_t slot_stride, const int* __restrict__ seg_start,
@@ -50,9 +83,12 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && RPT == 8 ? 3 : 1) gated_r
   // form 0: the gated form above (q, z_f, v). form 1: a fixed decay per head and a key:
   // S <- lower[a] S + k v^T with q, k, v = silu of q_src, f_src, v_src (f_bias is not read; lower holds one decay a head).
   // form 2: the same with q and k turned by ex's angles, k times ex.k_scale, and no SiLU anywhere.
+  // form 4 (GATED): S <- g.x S + g.y k v^T with g = ex.gates[t][a] and q times ex.k_scale; V counts the column of ones, which v_src does not have.
   // form 3 (BONUS): r, k, v as they are, decays ex.decay, lower = u [heads * D]: o = (S + diag(u) k v^T)^T r, then S <- diag(decay) S + k v^T.
   // seg_list: the segments this launch walks (null: all). chunks != null: blockIdx.x is a chunk (first row, rows) that starts from a zero
   // state and leaves its closing state in chunk_state[chunk][head], its decay in chunk_decay[chunk][head] and q * decay in qa_out[row][head].
+  constexpr bool GATED = FIXED_ && BONUS_, FIXED = FIXED_, BONUS = BONUS_ && !FIXED_;
+  __shared__ float s_keep[GATED ? kChunk : 1], s_take[GATED ? kChunk : 1];
   extern __shared__ float sm[];   // q[kChunk][D], f[kChunk][D], g[kChunk][D], v[kChunk][kCols], running decay [D]
   float* sq = sm;
   float* sf = sq + kChunk * D;
@@ -84,8 +120,9 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && RPT == 8 ? 3 : 1) gated_r
     st[r][0] = (!chunks && d < D && j < V) ? S[(size_t)d * V + j] : 0.f;
     st[r][1] = (!chunks && d < D && j + 1 < V) ? S[(size_t)d * V + j + 1] : 0.f;
   }
-  const int q_off = a * D, v_off = a * V + j0;
-  const float fixed = FIXED ? lower[a] : 0.f;
+  const int v_cols = GATED ? V - 1 : V;   // columns the values' source has
+  const int q_off = a * D, v_off = a * v_cols + j0;
+  const float fixed = FIXED && !GATED ? lower[a] : 0.f;
   float u[BONUS ? RPT : 1];
   if constexpr (BONUS) {
 #pragma unroll
@@ -94,6 +131,19 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && RPT == 8 ? 3 : 1) gated_r
   for (int c0 = t0; c0 < t1; c0 += kChunk) {
     const int n = min(kChunk, t1 - c0);
     __syncthreads();
+    if constexpr (GATED) {
+      if (tid < n) {
+        if (ex.gates) {
+          const float2 g = ex.gates[(size_t)(c0 + tid) * heads + a];
+          s_keep[tid] = g.x, s_take[tid] = g.y;
+        } else {
+          const float m = ex.mg.m_state[(size_t)seg_slot[seg_list ? seg_list[blockIdx.x] : blockIdx.x] * ex.mg.m_stride + a];
+          const float2 g = log_gates(ex.mg, c0 + tid, a);
+          const float next = fmaxf(g.y + m, g.x);
+          s_keep[tid] = expf(g.y + m - next), s_take[tid] = expf(g.x - next);
+        }
+      }
+    }
     // The sixteen tokens' rows into shared memory: every thread requests its values of kLoads items before it uses the first.
     const int step = kLoads * blockDim.x;
     if (FIXED && form == 2) {   // an item is a pair of entries that are turned together, or one that is not
@@ -171,6 +221,9 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && RPT == 8 ? 3 : 1) gated_r
             sq[i] = zq[e];
             sg[i] = zf[e];
             sf[i] = dc[e];
+          } else if constexpr (GATED) {
+            sq[i] = zq[e] * ex.k_scale;
+            sg[i] = zf[e];
           } else if constexpr (FIXED) {
             sq[i] = zq[e] / (1.f + expf(-zq[e]));
             sg[i] = zf[e] / (1.f + expf(-zf[e]));
@@ -192,19 +245,19 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && RPT == 8 ? 3 : 1) gated_r
 #pragma unroll
       for (int e = 0; e < kLoads; e++) {
         const int i = i0 + e * (int)blockDim.x, c = i % kCols;
-        z[e] = (i < n * kCols && j0 + c < V) ? v_src[(size_t)(c0 + i / kCols) * R + v_off + c] : 0.f;
+        z[e] = (i < n * kCols && j0 + c < v_cols) ? v_src[(size_t)(c0 + i / kCols) * R + v_off + c] : 0.f;
       }
       for (int p = 1; p < P; p++) {
 #pragma unroll
         for (int e = 0; e < kLoads; e++) {
           const int i = i0 + e * (int)blockDim.x, c = i % kCols;
-          if (i < n * kCols && j0 + c < V) z[e] += v_src[p * stride_p + (size_t)(c0 + i / kCols) * R + v_off + c];
+          if (i < n * kCols && j0 + c < v_cols) z[e] += v_src[p * stride_p + (size_t)(c0 + i / kCols) * R + v_off + c];
         }
       }
 #pragma unroll
       for (int e = 0; e < kLoads; e++) {
         const int i = i0 + e * (int)blockDim.x;
-        if (i < n * kCols) sv[i] = FIXED && form == 1 ? z[e] / (1.f + expf(-z[e])) : z[e];
+        if (i < n * kCols) sv[i] = GATED ? (j0 + i % kCols == v_cols ? 1.f : z[e]) : FIXED && form == 1 ? z[e] / (1.f + expf(-z[e])) : z[e];
       }
     }
     __syncthreads();
@@ -212,7 +265,7 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && RPT == 8 ? 3 : 1) gated_r
       for (int d = tid; d < D; d += blockDim.x) {
         float r = run[d];
         for (int tt = 0; tt < n; tt++) {
-          if (!BONUS) r *= FIXED ? fixed : sf[tt * D + d];
+          if (!BONUS) r *= GATED ? s_keep[GATED ? tt : 0] : FIXED ? fixed : sf[tt * D + d];
           qa_out[((size_t)(c0 + tt) * heads + a) * D + d] = sq[tt * D + d] * r;
           if (BONUS) r *= sf[tt * D + d];   // the current token's decay comes after its output
         }
@@ -221,13 +274,14 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && RPT == 8 ? 3 : 1) gated_r
     }
     // one token: the thread's rows of the state advance, acc0 and acc1 receive its share of o for its two columns
     auto advance = [&](int tt, float& acc0, float& acc1) {
-      const float v0 = sv[tt * kCols + col], v1 = sv[tt * kCols + col + 1];
+      const float take = GATED ? s_take[GATED ? tt : 0] : 1.f, keep = GATED ? s_keep[GATED ? tt : 0] : fixed;
+      const float v0 = GATED ? take * sv[tt * kCols + col] : sv[tt * kCols + col], v1 = GATED ? take * sv[tt * kCols + col + 1] : sv[tt * kCols + col + 1];
       float f[RPT], g[RPT], q[RPT];
       if (d4 && d0 + RPT <= D) {   // this thread's rows are whole groups of four: 16-byte reads
 #pragma unroll
         for (int r = 0; r < RPT; r += 4) {
           const float4 b = *(const float4*)(sg + tt * D + d0 + r), c = *(const float4*)(sq + tt * D + d0 + r);
-          const float4 a = FIXED ? make_float4(fixed, fixed, fixed, fixed) : *(const float4*)(sf + tt * D + d0 + r);
+          const float4 a = FIXED ? make_float4(keep, keep, keep, keep) : *(const float4*)(sf + tt * D + d0 + r);
           f[r] = a.x, f[r + 1] = a.y, f[r + 2] = a.z, f[r + 3] = a.w;
           g[r] = b.x, g[r + 1] = b.y, g[r + 2] = b.z, g[r + 3] = b.w;
           q[r] = c.x, q[r + 1] = c.y, q[r + 2] = c.z, q[r + 3] = c.w;
@@ -237,7 +291,7 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && RPT == 8 ? 3 : 1) gated_r
         for (int r = 0; r < RPT; r++) {
           const int d = d0 + r;
           const bool in = d < D;
-          f[r] = FIXED ? fixed : in ? sf[tt * D + d] : 0.f, g[r] = in ? sg[tt * D + d] : 0.f, q[r] = in ? sq[tt * D + d] : 0.f;
+          f[r] = FIXED ? keep : in ? sf[tt * D + d] : 0.f, g[r] = in ? sg[tt * D + d] : 0.f, q[r] = in ? sq[tt * D + d] : 0.f;
         }
       }
       acc0 = acc1 = 0.f;
@@ -494,6 +548,92 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
   }
 }
 
+// The gates of form 4 for whole segments: a CTA per (segment, head) walks its tokens 256 at a time. A token maps m to max(m + f, i); maps compose as
+// (a, b) then (a', b') = (a + a', max(b + a', b')), so the running maxima are an inclusive scan (shuffles inside a warp, then over the warps).
+// gates[t][head] = (e^(f + m_(t-1) - m_t), e^(i - m_t)), bound[t][head] = e^(-m_t); the state's m becomes the segment's last.
+constexpr int kGateTokens = 256;
+
+__global__ void __launch_bounds__(kGateTokens) memory_gates_kernel(IbMemoryGates g, const int* __restrict__ seg_start, const int* __restrict__ seg_slot,
+                                                                   float2* __restrict__ gates, float* __restrict__ bound, int heads) {
+  __shared__ float2 total[kGateTokens / 32];
+  __shared__ float m_all[kGateTokens + 1];
+  ib::pdl_launch_dependents();
+  ib::pdl_wait();
+  const int s = blockIdx.x, a = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int t0 = seg_start[s], t1 = seg_start[s + 1];
+  float* m_slot = g.m_state + (size_t)seg_slot[s] * g.m_stride + a;
+  float m_in = *m_slot;
+  for (int c0 = t0; c0 < t1; c0 += kGateTokens) {
+    const int t = c0 + tid;
+    const bool in = t < t1;
+    const float2 z = in ? log_gates(g, t, a) : make_float2(-INFINITY, 0.f);   // beyond the end: the map that changes nothing
+    float A = z.y, B = z.x;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float pa = __shfl_up_sync(0xffffffffu, A, o), pb = __shfl_up_sync(0xffffffffu, B, o);
+      if (lane >= o) {
+        B = fmaxf(pb + A, B);
+        A = pa + A;
+      }
+    }
+    if (lane == 31) total[warp] = make_float2(A, B);
+    if (tid == 0) m_all[0] = m_in;
+    __syncthreads();
+    float m0 = m_in;   // the running maximum before this warp's first token
+    for (int w = 0; w < warp; w++) m0 = fmaxf(m0 + total[w].x, total[w].y);
+    const float m = fmaxf(m0 + A, B);
+    m_all[tid + 1] = m;
+    __syncthreads();
+    if (in) {
+      gates[(size_t)t * heads + a] = make_float2(expf(z.y + m_all[tid] - m), expf(z.x - m));
+      bound[(size_t)t * heads + a] = expf(-m);
+    }
+    m_in = m_all[min(kGateTokens, t1 - c0)];
+    __syncthreads();
+  }
+  if (tid == 0 && t1 > t0) *m_slot = m_in;
+}
+
+// A warp per (token, head): o float32 [T][heads][V + 1] with n . q as its last entry. bound: e^(-m) of memory_gates, or null in a step whose row t is
+// segment t: m is then moved on here, from the state, as the walk did.
+template <typename O>
+__global__ void memory_out_kernel(const float* __restrict__ o, const float* __restrict__ bound, IbMemoryGates g, const int* __restrict__ seg_slot,
+                                  const float* __restrict__ w, float eps, const float* __restrict__ gate, int gate_P, size_t gate_stride, int gate_row,
+                                  O* __restrict__ out, long long items, int heads, int V) {
+  ib::pdl_launch_dependents();
+  ib::pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + warp;
+  if (item >= items) return;
+  const long long t = item / heads;
+  const int a = (int)(item - t * heads);
+  float floor_;
+  if (bound) {
+    floor_ = bound[item];
+  } else {
+    float* m_slot = g.m_state + (size_t)seg_slot[t] * g.m_stride + a;
+    const float2 z = log_gates(g, (int)t, a);
+    const float m = fmaxf(z.y + *m_slot, z.x);
+    __syncwarp();
+    if (lane == 0) *m_slot = m;
+    floor_ = expf(-m);
+  }
+  const float* src = o + item * (V + 1);
+  const float* gr = gate + t * gate_row + a * V;
+  const float div = 1.f / (fmaxf(fabsf(src[V]), floor_) + 1e-6f);
+  float ss = 0.f;
+  for (int i = lane; i < V; i += 32) {
+    const float v = src[i] * div;
+    ss = __fmaf_rn(v, v, ss);
+  }
+  const float inv = 1.f / sqrtf(ib::warp_sum(ss) / (float)V + eps);
+  for (int i = lane; i < V; i += 32) {
+    float z = gr[i];
+    for (int p = 1; p < gate_P; p++) z += gr[p * gate_stride + i];
+    out[item * V + i] = ib::from_f32<O>(w[a * V + i] * (src[i] * div * inv) / (1.f + expf(-z)));
+  }
+}
+
 }  // namespace
 
 // seg_list: int32 [n_segments] of the segments to walk (null: segments 0 .. n_segments - 1).
@@ -528,6 +668,7 @@ int launch_recurrence(const float* q_src, const float* f_src, const float* v_src
     else go(gated_recurrence_kernel<16, 16, F, B, 256>);
   };
   if (form == 3) pick(std::false_type(), std::true_type());
+  else if (form == 4) pick(std::true_type(), std::true_type());
   else if (form == 0) pick(std::false_type(), std::false_type());
   else pick(std::true_type(), std::false_type());
   IB_CHECK_LAUNCH("recurrence");
@@ -548,6 +689,45 @@ extern "C" int ib_recurrence_parts(const float* q, const float* k, const float* 
   RecurrenceExtras ex = {cos_t, sin_t, rot_half, k_scale, decay};
   return launch_recurrence(q, k, v, P, stride_p, row, nullptr, head_param, state, slot_stride, seg_start, seg_slot, n_segments, o_out, heads, D, V, seg_list, chunks, chunk_state,
                            chunk_decay, qa, form, ex, stream);
+}
+
+// The matrix memory (form 4). g: see IbMemoryGates; V: a value head's size; state float32 [slots][heads][D][V + 1], o_out [T][heads][V + 1]. gates
+// [T][heads][2] from ib_memory_gates, or null where every segment walked here brings one token. q_scale multiplies the queries.
+extern "C" int ib_memory_walk(const float* q, const float* k, const float* v, int P, long long stride_p, int row, const IbMemoryGates* g, const float* gates, float q_scale,
+                              float* state, long long slot_stride, const int* seg_start, const int* seg_slot, int n_segments, float* o_out, int heads, int D, int V,
+                              const int* seg_list, const int* chunks, float* chunk_state, float* chunk_decay, float* qa, cudaStream_t stream) {
+  if (n_segments == 0) return 0;
+  IB_CHECK_ARG(q && k && v && (gates || (g && !chunks)), "memory_walk: a part or the gates are missing");
+  RecurrenceExtras ex = {};
+  ex.k_scale = q_scale, ex.gates = (const float2*)gates;
+  if (g) ex.mg = *g;
+  return launch_recurrence(q, k, v, P, stride_p, row, nullptr, nullptr, state, slot_stride, seg_start, seg_slot, n_segments, o_out, heads, D, V + 1, seg_list, chunks, chunk_state,
+                           chunk_decay, qa, 4, ex, stream);
+}
+
+extern "C" int ib_memory_gates(const IbMemoryGates* g, const int* seg_start, const int* seg_slot, int n_segments, float* gates, float* bound, int heads, cudaStream_t stream) {
+  if (n_segments == 0) return 0;
+  IB_CHECK_ARG(n_segments > 0 && heads > 0 && heads <= 65535 && g && g->P >= 1 && g->cap > 0.f, "memory_gates: bad sizes segments=%d heads=%d", n_segments, heads);
+  ib::launch(memory_gates_kernel, dim3((unsigned)n_segments, (unsigned)heads), kGateTokens, 0, stream, *g, seg_start, seg_slot, (float2*)gates, bound, heads);
+  IB_CHECK_LAUNCH("memory_gates");
+  return 0;
+}
+
+// gate: float32 partial sums [gate_P][T][gate_row], offset to the first head's first column; out [T][heads * V].
+extern "C" int ib_memory_out(const float* o, const float* bound, const IbMemoryGates* g, const int* seg_slot, const float* w, float eps, const float* gate, int gate_P,
+                             long long gate_stride, int gate_row, void* out, int out_dtype, int T, int heads, int V, cudaStream_t stream) {
+  if (T == 0) return 0;
+  IB_CHECK_ARG(T > 0 && heads > 0 && V > 0 && gate && gate_P >= 1 && gate_row >= heads * V && w && g, "memory_out: bad sizes T=%d heads=%d V=%d", T, heads, V);
+  const long long items = (long long)T * heads;
+  const unsigned grid = (unsigned)((items + 3) / 4);
+  if (out_dtype == IB_F32)
+    ib::launch(memory_out_kernel<float>, grid, 128, 0, stream, o, bound, *g, seg_slot, w, eps, gate, gate_P, (size_t)gate_stride, gate_row, (float*)out, items, heads, V);
+  else if (out_dtype == IB_BF16)
+    ib::launch(memory_out_kernel<__nv_bfloat16>, grid, 128, 0, stream, o, bound, *g, seg_slot, w, eps, gate, gate_P, (size_t)gate_stride, gate_row, (__nv_bfloat16*)out, items,
+               heads, V);
+  else return ib_set_error("memory_out: unknown output dtype %d", out_dtype);
+  IB_CHECK_LAUNCH("memory_out");
+  return 0;
 }
 
 extern "C" int ib_gated_recurrence(const float* proj, int P, long long stride_p, const float* f_bias, const float* lower, float* state, long long slot_stride,

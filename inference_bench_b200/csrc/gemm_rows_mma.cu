@@ -36,6 +36,8 @@ struct RowsArgs {
   const float* gate;
   int gate_P, gate_row;
   long long gate_stride;
+  const float* limits;   // grouped mode with a gate half: null for silu(gate) * up, else clamped halves with one limit a group
+  float slope;
   int relu2;     // grouped mode without a gate half: the output is the square of max(product, 0)
 };
 
@@ -156,6 +158,7 @@ __global__ void __launch_bounds__(128) gemm_rows_mma_kernel(RowsArgs p) {
     }
   }
   O* out = (O*)p.out;
+  const float limit = GATED && p.limits ? p.limits[group] : 0.f;
 #pragma unroll
   for (int m = 0; m < 2; m++)
 #pragma unroll
@@ -177,7 +180,7 @@ __global__ void __launch_bounds__(128) gemm_rows_mma_kernel(RowsArgs p) {
           const int n = n0 + wn * 32 + nt * 8 + 2 * t4 + c;
           if (n >= N) continue;
           float v = acc[m][nt][2 * h + c];
-          if constexpr (GATED) v = (v / (1.f + expf(-v))) * acu[m][nt][2 * h + c];
+          if constexpr (GATED) v = p.limits ? ib::clamped_glu<false>(v, acu[m][nt][2 * h + c], limit, p.slope) : (v / (1.f + expf(-v))) * acu[m][nt][2 * h + c];
           else if (p.relu2) v = ib::relu2(v);
           dst[n] = ib::from_f32<O>(v * f);
         }
@@ -205,15 +208,17 @@ int launch_rows(const RowsArgs& a, dim3 grid, int gated, int out_dtype, cudaStre
 }  // namespace
 
 extern "C" int ib_gemm_grouped_mma(const void* x, const int* src_row, const void* w, void* out, int out_dtype, const int* offsets, const int* tile_start, int R, int E,
-                                   int N, int K, int act, cudaStream_t stream) {
-  // act: 0 the product, 1 silu(gate) * up (w holds gate rows, then up rows), 2 the square of max(product, 0)
+                                   int N, int K, int act, const float* limits, float slope, cudaStream_t stream) {
+  // act: 0 the product, 1 silu(gate) * up (w holds gate rows, then up rows), 2 the square of max(product, 0), 3 as 1 with clamped halves
+  // (limits: float32 [E], slope: the sigmoid's)
   if (R == 0 || N == 0) return 0;
-  IB_CHECK_ARG(act >= 0 && act <= 2, "gemm_grouped_mma: activation %d is not known", act);
-  const int gated = act == 1;
+  IB_CHECK_ARG(act >= 0 && act <= 3 && (act != 3 || limits), "gemm_grouped_mma: activation %d is not known", act);
+  const int gated = act == 1 || act == 3;
   IB_CHECK_ARG(R > 0 && E > 0 && N > 0 && K > 0, "gemm_grouped_mma: bad sizes rows=%d experts=%d N=%d K=%d", R, E, N, K);
   RowsArgs a = {};
   a.x = (const __nv_bfloat16*)x, a.w = (const __nv_bfloat16*)w, a.out = out, a.src_row = src_row, a.offsets = offsets, a.tile_start = tile_start;
   a.n_groups = E, a.N = N, a.K = K, a.grouped = 1, a.relu2 = act == 2;
+  if (act == 3) a.limits = limits, a.slope = slope;
   return launch_rows(a, dim3((N + TN - 1) / TN, R / TM + E, 1), gated, out_dtype, stream, "gemm_grouped_mma");
 }
 

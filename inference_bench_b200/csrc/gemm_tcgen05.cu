@@ -31,6 +31,9 @@ constexpr int EPI_SWIGLU = 1;  // accumulator 0 = gate, accumulator 1 = up -> bf
 constexpr int EPI_XIELU = 3;   // one or two accumulators of plain rows -> bfloat16 xielu(product) with the two numbers of act_pq
 constexpr int EPI_RELU2 = 4;   // the same with the square of max(product, 0)
 constexpr int EPI_SWIGLU_HALF = 2;  // one accumulator: rows 0-63 = 64 gate rows, rows 64-127 = the matching 64 up rows -> bfloat16 silu(gate) * up
+constexpr int EPI_CLAMPED = 5, EPI_CLAMPED_HALF = 6;   // EPI_SWIGLU and EPI_SWIGLU_HALF with clamped halves instead (ib::clamped_glu)
+constexpr bool epi_half(int epi) { return epi == EPI_SWIGLU_HALF || epi == EPI_CLAMPED_HALF; }
+constexpr bool epi_pair(int epi) { return epi == EPI_SWIGLU || epi == EPI_CLAMPED; }
 // (for a handful of tokens: as many CTAs as the plain product has, I / 64, so the weights stream as fast, and neither the
 // float32 [T, 2I] intermediate nor the SiLU-mul kernel exists)
 
@@ -50,7 +53,8 @@ template <int BN, int MT, int EPI>
 __global__ void __launch_bounds__(kThreads, 1)
     gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_x, void* __restrict__ out_, int T,
                         int N, int K, int ktiles_per_split, int second_off, unsigned long long wait_ns, int starve, unsigned* __restrict__ status,
-                        const int* __restrict__ grp_offsets, const int* __restrict__ grp_tiles, int n_groups, int grp_w_rows, const float* __restrict__ act_pq, int part_rows) {
+                        const int* __restrict__ grp_offsets, const int* __restrict__ grp_tiles, int n_groups, int grp_w_rows, const float* __restrict__ act_pq, int part_rows, float act_slope) {
+  // EPI_CLAMPED and its half form: act_pq holds the limit of every group (of the one matrix without groups), act_slope the sigmoid's slope.
   // part_rows > 0: x holds parts of that many rows each, one after the other, and part i goes through matrix i (rows i * grp_w_rows .. of w); a
   // tile of rows belongs to one part.
   // grp_offsets != nullptr: the rows of x are regrouped (rows grp_offsets[e] .. grp_offsets[e + 1] belong to group e, whose matrix is rows
@@ -73,9 +77,9 @@ __global__ void __launch_bounds__(kThreads, 1)
   // first output column of this CTA, and the W row where each accumulator's block starts
   // (token tiles vary fastest in the grid: the CTAs that share a block of W run together, so W comes
   // from memory once and the much smaller x stays in L2)
-  const int n0 = blockIdx.y * (EPI == EPI_SWIGLU_HALF ? BM / 2 : EPI == EPI_SWIGLU ? BM : BM * MT);
+  const int n0 = blockIdx.y * (epi_half(EPI) ? BM / 2 : epi_pair(EPI) ? BM : BM * MT);
   const int split = blockIdx.z;
-  int t0 = blockIdx.x * BN, t_end = T, w_row0 = 0;
+  int t0 = blockIdx.x * BN, t_end = T, w_row0 = 0, group = 0;
   if (grp_offsets) {
     ib::pdl_wait();   // the table is the work of the kernels before
     const int b = blockIdx.x;
@@ -89,6 +93,7 @@ __global__ void __launch_bounds__(kThreads, 1)
     t0 = grp_offsets[lo] + (b - grp_tiles[lo]) * BN;
     t_end = grp_offsets[lo + 1];
     w_row0 = lo * grp_w_rows;
+    group = lo;
   }
   if (part_rows > 0) {
     const int per = (part_rows + BN - 1) / BN, part = blockIdx.x / per;
@@ -126,7 +131,7 @@ __global__ void __launch_bounds__(kThreads, 1)
       // The weights do not depend on earlier kernels: fill the pipeline with them before waiting
       // for the kernel that produces x, then send the x tiles after.
       auto load_w = [&](uint8_t* a, int kt, uint64_t* bar) {   // this CTA's rows of W for k-tile kt
-        if constexpr (EPI == EPI_SWIGLU_HALF) {   // tmap_w's box has 64 rows here: gate rows, then the up rows second_off further on
+        if constexpr (epi_half(EPI)) {   // tmap_w's box has 64 rows here: gate rows, then the up rows second_off further on
           sm100::tma_load_2d(a, &tmap_w, kt * BK, w_row0 + n0, bar);
           sm100::tma_load_2d(a + TL::kABytes / 2, &tmap_w, kt * BK, w_row0 + n0 + second_off, bar);
         } else {
@@ -194,6 +199,12 @@ __global__ void __launch_bounds__(kThreads, 1)
     ok = __all_sync(0xffffffffu, ok);
     constexpr int CH = BN < 32 ? 16 : 32;
     const uint32_t lane_addr = tmem + ((uint32_t)(q * 32) << 16);
+    constexpr bool kClamped = EPI == EPI_CLAMPED || EPI == EPI_CLAMPED_HALF;
+    const float limit = kClamped ? act_pq[group] : 0.f;
+    auto gated = [&](float gv, float uv) {
+      if constexpr (kClamped) return __float2bfloat16_rn(ib::clamped_glu<true>(gv, uv, limit, act_slope));
+      else return __float2bfloat16_rn(__fdividef(gv, 1.f + __expf(-gv)) * uv);
+    };
     if (ok && (EPI == EPI_STORE || EPI == EPI_XIELU || EPI == EPI_RELU2)) {
       float* dst = (float*)out_ + (size_t)split * T * N;
       __nv_bfloat16* dst_act = (__nv_bfloat16*)out_;   // EPI_XIELU: the whole k-range is this CTA's, the activation is applied here
@@ -232,7 +243,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         }
       }
     }
-    if (ok && EPI == EPI_SWIGLU) {
+    if (ok && epi_pair(EPI)) {
       __nv_bfloat16* dst = (__nv_bfloat16*)out_;
       const int n = n0 + q * 32 + lane;
 #pragma unroll 1
@@ -251,12 +262,12 @@ __global__ void __launch_bounds__(kThreads, 1)
           for (int c = 0; c < CH; c++) {
             const int t = t0 + c0 + c;
             const float gv = __uint_as_float(g[c]), uv = __uint_as_float(u[c]);
-            if (t < t_end) dst[(size_t)t * N + n] = __float2bfloat16_rn(__fdividef(gv, 1.f + __expf(-gv)) * uv);
+            if (t < t_end) dst[(size_t)t * N + n] = gated(gv, uv);
           }
         }
       }
     }
-    if constexpr (EPI == EPI_SWIGLU_HALF) {
+    if constexpr (epi_half(EPI)) {
       // Lanes 0-63 of the accumulator (warps with q = 0, 1) hold gate rows, lanes 64-127 (q = 2, 3) the matching up rows. The up
       // half goes through shared memory (the pipeline's stages are free once the accumulator is complete) to the warps that
       // hold the gate half, which apply the activation and store. All four warps meet at a barrier of their own, whatever ok says.
@@ -285,7 +296,7 @@ __global__ void __launch_bounds__(kThreads, 1)
             for (int c = 0; c < CH; c++) {
               const int t = t0 + c0 + c;
               const float gv = __uint_as_float(r[c]), uv = up_s[(c0 + c) * 64 + q * 32 + lane];
-              if (t < t_end) dst[(size_t)t * N + n] = __float2bfloat16_rn(__fdividef(gv, 1.f + __expf(-gv)) * uv);
+              if (t < t_end) dst[(size_t)t * N + n] = gated(gv, uv);
             }
           }
         }
@@ -326,7 +337,8 @@ struct Groups {   // regrouped rows (see the kernel): nullptr offsets = one matr
 
 template <int BN, int MT, int EPI>
 int launch(const CUtensorMap& tw, const CUtensorMap& tx, void* out, int T, int N, int K, int splits, int kt_per_split, int second_off,
-           unsigned* status, cudaStream_t stream, int starve = 0, Groups grp = Groups(), const float* act_pq = nullptr) {
+           unsigned* status, cudaStream_t stream, int starve = 0, Groups grp = Groups(), const float* act_pq = nullptr,
+           float act_slope = 0.f) {
   using TL = Tile<BN, MT>;
   static bool configured = false;
   if (!configured) {
@@ -334,11 +346,11 @@ int launch(const CUtensorMap& tw, const CUtensorMap& tx, void* out, int T, int N
     IB_CHECK_ARG(e == cudaSuccess, "gemm_tcgen05: cannot reserve %d bytes of shared memory: %s", TL::kSmemBytes, cudaGetErrorString(e));
     configured = true;
   }
-  const int cols_per_cta = EPI == EPI_SWIGLU_HALF ? BM / 2 : EPI == EPI_SWIGLU ? BM : BM * MT;
+  const int cols_per_cta = epi_half(EPI) ? BM / 2 : epi_pair(EPI) ? BM : BM * MT;
   dim3 grid(grp.offsets ? T / BN + grp.n : grp.part_rows ? grp.n * ((grp.part_rows + BN - 1) / BN) : (T + BN - 1) / BN, (N + cols_per_cta - 1) / cols_per_cta, splits);
   IB_CHECK_ARG(grid.y <= 65535, "gemm_tcgen05: N=%d gives more than 65535 row blocks", N);
   ib::launch(gemm_tcgen05_kernel<BN, MT, EPI>, grid, kThreads, TL::kSmemBytes, stream, tw, tx, out, T, N, K, kt_per_split, second_off, ib_wait_limit_ns(), starve, status,
-             grp.offsets, grp.tiles, grp.n, grp.w_rows, act_pq, grp.part_rows);
+             grp.offsets, grp.tiles, grp.n, grp.w_rows, act_pq, grp.part_rows, act_slope);
   IB_CHECK_LAUNCH("gemm_tcgen05");
   return 0;
 }
@@ -455,7 +467,8 @@ extern "C" int ib_gemm_relu2_tcgen05(const void* x, const void* w, void* act, in
 // SwiGLU front half in one kernel: w [2*I, K] = gate rows then up rows; act [T, I] bfloat16 =
 // silu(x gate^T) * (x up^T). bn: 16 or 32 tokens per CTA, or 64 with half != 0 (64 gate rows and their 64 up rows in one
 // accumulator: I must be a multiple of 64), or 64, 128 or 256 (128 gate rows and 128 up rows in two accumulators).
-extern "C" int ib_gemm_swiglu_tcgen05(const void* x, const void* w, void* act, int T, int I, int K, int bn, int half, unsigned* status,
+// limit null: that; else clamped halves, with one limit (float32 on the device) and the sigmoid's slope.
+extern "C" int ib_gemm_swiglu_tcgen05(const void* x, const void* w, void* act, int T, int I, int K, int bn, int half, const float* limit, float slope, unsigned* status,
                                       cudaStream_t stream) {
   if (T == 0 || I == 0) return 0;
   if (check_common("gemm_swiglu_tcgen05", x, w, T, I, K, bn)) return 1;
@@ -465,12 +478,25 @@ extern "C" int ib_gemm_swiglu_tcgen05(const void* x, const void* w, void* act, i
     IB_CHECK_ARG(I % 64 == 0, "gemm_swiglu_tcgen05: with %d tokens per CTA the intermediate size must be a multiple of 64, not %d", bn, I);
     if (make_tmap(&tw, w, 2 * I, K, BM / 2)) return 1;
     if (make_tmap(&tx, x, T, K, bn)) return 1;
+    if (limit) {
+      if (bn == 16) return launch<16, 1, EPI_CLAMPED_HALF>(tw, tx, act, T, I, K, 1, total_kt, I, status, stream, 0, Groups(), limit, slope);
+      if (bn == 32) return launch<32, 1, EPI_CLAMPED_HALF>(tw, tx, act, T, I, K, 1, total_kt, I, status, stream, 0, Groups(), limit, slope);
+      return launch<64, 1, EPI_CLAMPED_HALF>(tw, tx, act, T, I, K, 1, total_kt, I, status, stream, 0, Groups(), limit, slope);
+    }
     if (bn == 16) return launch<16, 1, EPI_SWIGLU_HALF>(tw, tx, act, T, I, K, 1, total_kt, I, status, stream);
     if (bn == 32) return launch<32, 1, EPI_SWIGLU_HALF>(tw, tx, act, T, I, K, 1, total_kt, I, status, stream);
     return launch<64, 1, EPI_SWIGLU_HALF>(tw, tx, act, T, I, K, 1, total_kt, I, status, stream);
   }
   if (make_tmap(&tw, w, 2 * I, K, BM)) return 1;
   if (make_tmap(&tx, x, T, K, bn)) return 1;
+  if (limit) {
+    switch (bn) {
+      case 64: return launch<64, 2, EPI_CLAMPED>(tw, tx, act, T, I, K, 1, total_kt, I, status, stream, 0, Groups(), limit, slope);
+      case 128: return launch<128, 2, EPI_CLAMPED>(tw, tx, act, T, I, K, 1, total_kt, I, status, stream, 0, Groups(), limit, slope);
+      case 256: return launch<256, 2, EPI_CLAMPED>(tw, tx, act, T, I, K, 1, total_kt, I, status, stream, 0, Groups(), limit, slope);
+      default: return ib_set_error("gemm_swiglu_tcgen05: token tile %d is not one of 16, 32, 64, 128, 256", bn);
+    }
+  }
   switch (bn) {
     case 64: return launch<64, 2, EPI_SWIGLU>(tw, tx, act, T, I, K, 1, total_kt, I, status, stream);
     case 128: return launch<128, 2, EPI_SWIGLU>(tw, tx, act, T, I, K, 1, total_kt, I, status, stream);
@@ -549,8 +575,9 @@ extern "C" int ib_gemm_grouped_relu2_tcgen05(const void* x, const void* w, void*
 
 // w [E, 2 I, K]: every expert's gate rows then its up rows; act [R, I] bfloat16 = silu(x gate^T) * (x up^T) per expert.
 // bn 16 or 32: 64 gate rows and their up rows in one accumulator (I a multiple of 64); bn 64, 128 or 256: two accumulators.
+// limits null: that; else clamped halves with one limit an expert (float32 [E] on the device) and the sigmoid's slope.
 extern "C" int ib_gemm_grouped_swiglu_tcgen05(const void* x, const void* w, void* act, int R, int I, int K, int bn, const int* offsets, const int* tiles, int E,
-                                              unsigned* status, cudaStream_t stream) {
+                                              const float* limits, float slope, unsigned* status, cudaStream_t stream) {
   if (R == 0 || I == 0) return 0;
   if (check_common("gemm_grouped_swiglu_tcgen05", x, w, R, I, K, bn)) return 1;
   IB_CHECK_ARG(E > 0 && offsets && tiles, "gemm_grouped_swiglu_tcgen05: the groups' tables are missing");
@@ -562,10 +589,20 @@ extern "C" int ib_gemm_grouped_swiglu_tcgen05(const void* x, const void* w, void
   if (bn == 16 || bn == 32) {
     IB_CHECK_ARG(I % 64 == 0, "gemm_grouped_swiglu_tcgen05: with %d tokens per CTA the inner size must be a multiple of 64, not %d", bn, I);
     if (make_tmap(&tw, w, E * 2 * I, K, BM / 2)) return 1;
+    if (limits && bn == 16) return launch<16, 1, EPI_CLAMPED_HALF>(tw, tx, act, R, I, K, 1, total_kt, I, status, stream, 0, g, limits, slope);
+    if (limits) return launch<32, 1, EPI_CLAMPED_HALF>(tw, tx, act, R, I, K, 1, total_kt, I, status, stream, 0, g, limits, slope);
     if (bn == 16) return launch<16, 1, EPI_SWIGLU_HALF>(tw, tx, act, R, I, K, 1, total_kt, I, status, stream, 0, g);
     return launch<32, 1, EPI_SWIGLU_HALF>(tw, tx, act, R, I, K, 1, total_kt, I, status, stream, 0, g);
   }
   if (make_tmap(&tw, w, E * 2 * I, K, BM)) return 1;
+  if (limits) {
+    switch (bn) {
+      case 64: return launch<64, 2, EPI_CLAMPED>(tw, tx, act, R, I, K, 1, total_kt, I, status, stream, 0, g, limits, slope);
+      case 128: return launch<128, 2, EPI_CLAMPED>(tw, tx, act, R, I, K, 1, total_kt, I, status, stream, 0, g, limits, slope);
+      case 256: return launch<256, 2, EPI_CLAMPED>(tw, tx, act, R, I, K, 1, total_kt, I, status, stream, 0, g, limits, slope);
+      default: return ib_set_error("gemm_grouped_swiglu_tcgen05: token tile %d is not one of 16, 32, 64, 128, 256", bn);
+    }
+  }
   switch (bn) {
     case 64: return launch<64, 2, EPI_SWIGLU>(tw, tx, act, R, I, K, 1, total_kt, I, status, stream, 0, g);
     case 128: return launch<128, 2, EPI_SWIGLU>(tw, tx, act, R, I, K, 1, total_kt, I, status, stream, 0, g);

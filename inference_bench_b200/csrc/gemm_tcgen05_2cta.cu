@@ -28,6 +28,8 @@ constexpr int UMMA_K = 16;
 constexpr int kThreads = 192;
 constexpr int EPI_STORE = 0, EPI_SWIGLU = 1, EPI_ADD = 2;   // float32 out; bfloat16 silu(gate) * up; float32 out += product
 constexpr int EPI_QKV = 3;   // the q/k/v projection finished in the epilogue: per-head norm, rotation, queries out, keys and values into the cache
+constexpr int EPI_CLAMPED = 6;   // EPI_SWIGLU with clamped halves (ib::clamped_glu): the limit in QkvEpi::act_pq[0], the slope in QkvEpi::act_slope
+constexpr bool epi_gated(int epi) { return epi == EPI_SWIGLU || epi == EPI_CLAMPED; }
 constexpr int EPI_RELU2 = 5;   // bfloat16 max(product, 0)^2
 constexpr int EPI_XIELU = 4;   // bfloat16 xielu(product) with the activation's two numbers (QkvEpi::act_pq)
 constexpr int kQkvHead = 128;   // head size of the EPI_QKV form: a head is 128 accumulator columns
@@ -110,7 +112,8 @@ struct QkvEpi {
   IbKvView kv;
   int write_kv;
   int heads;
-  const float* act_pq;   // EPI_XIELU only: the activation's two numbers (p, q), float32 on the device
+  const float* act_pq;   // EPI_XIELU: the activation's two numbers (p, q); EPI_CLAMPED: the limit; float32 on the device
+  float act_slope;       // EPI_CLAMPED
 };
 
 // Persistent: each CTA pair walks tiles pair, pair + n_pairs, ... (token tiles vary fastest, so the
@@ -139,7 +142,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   const uint32_t rank = cluster_rank();          // 0 = leader
   const int pair = blockIdx.x >> 1, n_pairs = gridDim.x >> 1;
   const int nkt = (K + BK - 1) / BK;
-  constexpr int kColsPerPair = EPI == EPI_SWIGLU ? 2 * BM : 2 * BM * MT;
+  constexpr int kColsPerPair = epi_gated(EPI) ? 2 * BM : 2 * BM * MT;
 
   ib::pdl_launch_dependents();
   if (threadIdx.x == 0) {
@@ -173,7 +176,7 @@ __global__ void __launch_bounds__(kThreads, 1)
   // SwiGLU takes gate rows and, second_off on, up rows
   auto w_row = [&](int rb, int m) {
     const int n_pair = rb * kColsPerPair;
-    return EPI == EPI_SWIGLU ? n_pair + (int)rank * BM + m * second_off : n_pair + m * 2 * BM + (int)rank * BM;
+    return epi_gated(EPI) ? n_pair + (int)rank * BM + m * second_off : n_pair + m * 2 * BM + (int)rank * BM;
   };
 
   if (warp == 0) {
@@ -381,6 +384,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         }
       } else {
         __nv_bfloat16* dst = (__nv_bfloat16*)out_;
+        const float limit = EPI == EPI_CLAMPED ? qe.act_pq[0] : 0.f;
         const int n = n_pair + (int)rank * BM + q * 32 + lane;
 #pragma unroll 1
         for (int c0 = 0; c0 < BN; c0 += 32) {
@@ -393,7 +397,9 @@ __global__ void __launch_bounds__(kThreads, 1)
             for (int c = 0; c < 32; c++) {
               const int t = t0 + c0 + c;
               const float gv = __uint_as_float(g[c]), uv = __uint_as_float(u[c]);
-              if (t < T) dst[(size_t)t * N + n] = __float2bfloat16_rn(__fdividef(gv, 1.f + __expf(-gv)) * uv);
+              if (t >= T) continue;
+              if constexpr (EPI == EPI_CLAMPED) dst[(size_t)t * N + n] = __float2bfloat16_rn(ib::clamped_glu<true>(gv, uv, limit, qe.act_slope));
+              else dst[(size_t)t * N + n] = __float2bfloat16_rn(__fdividef(gv, 1.f + __expf(-gv)) * uv);
             }
           }
         }
@@ -441,7 +447,7 @@ int launch(const void* x, const void* w, void* out, int T, int N, int K, int w_r
   CUtensorMap tw, tx;
   if (make_tmap(&tw, w, w_rows, K, BM)) return 1;
   if (make_tmap(&tx, x, T, K, BN / 2)) return 1;
-  const int cols_per_pair = EPI == EPI_SWIGLU ? 2 * BM : 2 * BM * MT;
+  const int cols_per_pair = epi_gated(EPI) ? 2 * BM : 2 * BM * MT;
   const int token_tiles = (T + BN - 1) / BN, row_blocks = (N + cols_per_pair - 1) / cols_per_pair;
   const int total_tiles = token_tiles * row_blocks;
   static int sm_count = 0;
@@ -501,8 +507,14 @@ extern "C" int ib_gemm_xielu_tcgen05_2cta(const void* x, const void* w, void* ac
 }
 
 // w [2*I, K] = gate rows then up rows -> act [T, I] bfloat16 = silu(x gate^T) * (x up^T), on CTA pairs.
-extern "C" int ib_gemm_swiglu_tcgen05_2cta(const void* x, const void* w, void* act, int T, int I, int K, unsigned* status, cudaStream_t stream) {
+// limit: null, or one float32 on the device: clamped halves instead, with the sigmoid's slope.
+extern "C" int ib_gemm_swiglu_tcgen05_2cta(const void* x, const void* w, void* act, int T, int I, int K, const float* limit, float slope, unsigned* status, cudaStream_t stream) {
   if (T == 0 || I == 0) return 0;
+  if (limit) {
+    QkvEpi qe{};
+    qe.act_pq = limit, qe.act_slope = slope;
+    return launch<2, EPI_CLAMPED, 128>(x, w, act, T, I, K, 2 * I, I, status, stream, qe);
+  }
   return launch<2, EPI_SWIGLU, 128>(x, w, act, T, I, K, 2 * I, I, status, stream);
 }
 

@@ -13,7 +13,7 @@
 //    the two per-head products above.
 //  * latent_attention: a CTA per (token, eight heads, slice of the keys): key tiles of 32 rows go through shared memory
 //    once for all heads of the CTA; a warp owns a head, a lane a key for the scores and output columns for the sum.
-//    Scores, softmax weights and sums are float32. With slices, unnormalised partial results go to scratch and
+//    Scores, softmax weights and sums are float32. A sink adds exp(sink[head]) to the denominator, once, after all keys. With slices, unnormalised partial results go to scratch and
 //    latent_combine merges them.
 #include <type_traits>
 
@@ -216,7 +216,8 @@ __global__ void __launch_bounds__(kAttnWarps * 32) latent_attention_kernel(const
                                                                            const int* __restrict__ seg_of_token, float scale, O* __restrict__ out,
                                                                            float* __restrict__ part_o, float* __restrict__ part_ml, int T, int H,
                                                                            int rank, int D, int n_slices, int slice_keys,
-                                                                           unsigned* __restrict__ status, int window) {
+                                                                           unsigned* __restrict__ status, int window, const float* __restrict__ sink) {
+  // sink: a score per head that has no key and no value (with slices latent_combine counts it), or null
   // window > 0: a token sees itself and the window - 1 positions before it; the slices then cut that range.
   extern __shared__ __align__(16) float smem[];
   __shared__ long long koff[kKeyTile];
@@ -287,7 +288,11 @@ __global__ void __launch_bounds__(kAttnWarps * 32) latent_attention_kernel(const
   }
   if (!live) return;
   if (n_slices == 1) {
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    if (sink) {
+      const float z = sink[h], top = fmaxf(m, z), f = expf(m - top);
+      inv = f / (l * f + expf(z - top));
+    }
     O* o = out + ((size_t)t * H + h) * rank;
 #pragma unroll
     for (int r = 0; r < NR; r++) {
@@ -311,13 +316,18 @@ __global__ void __launch_bounds__(kAttnWarps * 32) latent_attention_kernel(const
 
 template <typename O>
 __global__ void latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, O* __restrict__ out, int rank,
-                                      int n_slices) {
+                                      int n_slices, const float* __restrict__ sink, int H) {
   ib::pdl_launch_dependents();
   ib::pdl_wait();
   const size_t unit0 = (size_t)blockIdx.x * n_slices;   // blockIdx.x = token * H + head
   float m = -INFINITY;
   for (int s = 0; s < n_slices; s++) m = fmaxf(m, part_ml[2 * (unit0 + s)]);
   float L = 0.f;
+  if (sink) {   // a score without key or value
+    const float z = sink[blockIdx.x % H];
+    m = fmaxf(m, z);
+    L = expf(z - m);
+  }
   for (int s = 0; s < n_slices; s++) {
     const float ms = part_ml[2 * (unit0 + s)];
     if (ms != -INFINITY) L += part_ml[2 * (unit0 + s) + 1] * expf(ms - m);
@@ -414,10 +424,11 @@ extern "C" int ib_gemm_heads(const void* x, int x_dtype, long long x_row, long l
 extern "C" int ib_latent_attention_max_rank() { return 1024; }
 
 // out[row] = the slices' unnormalised partial results of (token, head) `row`, merged and normalised.
-extern "C" int ib_latent_combine(const float* part_o, const float* part_ml, void* out, int out_dtype, int rows, int rank, int n_slices, cudaStream_t stream) {
+extern "C" int ib_latent_combine(const float* part_o, const float* part_ml, void* out, int out_dtype, int rows, int rank, int n_slices, const float* sink, int heads,
+                                 cudaStream_t stream) {
   if (rows == 0) return 0;
-  if (out_dtype == IB_F32) ib::launch(latent_combine_kernel<float>, (unsigned)rows, 128, 0, stream, part_o, part_ml, (float*)out, rank, n_slices);
-  else if (out_dtype == IB_BF16) ib::launch(latent_combine_kernel<__nv_bfloat16>, (unsigned)rows, 128, 0, stream, part_o, part_ml, (__nv_bfloat16*)out, rank, n_slices);
+  if (out_dtype == IB_F32) ib::launch(latent_combine_kernel<float>, (unsigned)rows, 128, 0, stream, part_o, part_ml, (float*)out, rank, n_slices, sink, heads);
+  else if (out_dtype == IB_BF16) ib::launch(latent_combine_kernel<__nv_bfloat16>, (unsigned)rows, 128, 0, stream, part_o, part_ml, (__nv_bfloat16*)out, rank, n_slices, sink, heads);
   else return ib_set_error("latent_combine: unknown output dtype %d", out_dtype);
   IB_CHECK_LAUNCH("latent_combine");
   return 0;
@@ -425,7 +436,8 @@ extern "C" int ib_latent_combine(const float* part_o, const float* part_ml, void
 
 extern "C" int ib_latent_attention(const float* q, const IbKvView* kv, const int* positions, const int* seg_of_token, float scale, void* out,
                                    int out_dtype, float* part_o, float* part_ml, int T, int heads, int rank, int n_slices, int slice_keys,
-                                   unsigned* status, int window, cudaStream_t stream) {
+                                   unsigned* status, int window, const float* sink, cudaStream_t stream) {
+  // sink: float32 [heads], scores without key or value, or null
   if (T == 0) return 0;
   if (check_rows_view("latent_attention", kv)) return 1;
   const int D = kv->head_dim;
@@ -439,7 +451,7 @@ extern "C" int ib_latent_attention(const float* q, const IbKvView* kv, const int
   auto go = [&](auto kernel, auto* o) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     ib::launch(kernel, grid, kAttnWarps * 32, smem, stream, q, *kv, positions, seg_of_token, scale, o, part_o, part_ml, T, heads, rank, D, n_slices, slice_keys,
-               status, window);
+               status, window, sink);
   };
   auto pick = [&](auto c_tag, auto* o) {
     using C = decltype(c_tag);
@@ -454,6 +466,6 @@ extern "C" int ib_latent_attention(const float* q, const IbKvView* kv, const int
   else if (out_dtype == IB_BF16 && kv->dtype == IB_BF16) pick(__nv_bfloat16(), (__nv_bfloat16*)out);
   else return ib_set_error("latent_attention: output dtype %d and cache dtype %d must match", out_dtype, kv->dtype);
   IB_CHECK_LAUNCH("latent_attention");
-  if (n_slices > 1) return ib_latent_combine(part_o, part_ml, out, out_dtype, T * heads, rank, n_slices, stream);
+  if (n_slices > 1) return ib_latent_combine(part_o, part_ml, out, out_dtype, T * heads, rank, n_slices, sink, heads, stream);
   return 0;
 }

@@ -30,7 +30,8 @@ __global__ void __launch_bounds__(kWarps * 32) latent_attention_mma_kernel(const
                                                                            const int* __restrict__ seg_of_token, const int2* __restrict__ units, float scale,
                                                                            __nv_bfloat16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml,
                                                                            int H, int rank, int D, int n_slices, int slice_keys, unsigned* __restrict__ status,
-                                                                           int window) {
+                                                                           int window, const float* __restrict__ sink) {
+  // sink: a score per head that has no key and no value (with slices latent_combine counts it), or null
   // window > 0: a token sees itself and the window - 1 positions before it; the CTA's keys start where its first token's window does.
   constexpr int R = 16 * MT;                                 // query rows of the CTA
   extern __shared__ __align__(128) unsigned char smem[];
@@ -283,7 +284,11 @@ __global__ void __launch_bounds__(kWarps * 32) latent_attention_mma_kernel(const
       if (row_tok[a][rr] < 0) continue;
       const size_t th = (size_t)row_tok[a][rr] * H + row_head[a][rr];
       if (n_slices == 1) {
-        const float inv = l[a][rr] > 0.f ? 1.f / l[a][rr] : 0.f;
+        float inv = l[a][rr] > 0.f ? 1.f / l[a][rr] : 0.f;
+        if (sink) {
+          const float z = sink[row_head[a][rr]], top = fmaxf(m[a][rr], z), f = expf(m[a][rr] - top);
+          inv = f / (l[a][rr] * f + expf(z - top));
+        }
         __nv_bfloat16* dst = out + th * rank;
 #pragma unroll
         for (int i = 0; i < NCH; i++) {
@@ -318,7 +323,7 @@ size_t latent_mma_smem(int D, int mt) {
 
 }  // namespace
 
-extern "C" int ib_latent_combine(const float* part_o, const float* part_ml, void* out, int out_dtype, int rows, int rank, int n_slices, cudaStream_t stream);
+extern "C" int ib_latent_combine(const float* part_o, const float* part_ml, void* out, int out_dtype, int rows, int rank, int n_slices, const float* sink, int heads, cudaStream_t stream);
 
 // 1 when the tensor-core kernel takes these sizes (bfloat16 cache rows of D values of which the first `rank` are the latent).
 extern "C" int ib_latent_attention_mma_supports(int rank, int D) { return rank > 0 && rank % 16 == 0 && D % 16 == 0 && rank <= D && rank <= 512 && D <= 576; }
@@ -336,7 +341,7 @@ extern "C" int ib_latent_attention_mma_rows(int rank, int D, int rows_wanted) {
 
 extern "C" int ib_latent_attention_mma(const float* q, const IbKvView* kv, const int* positions, const int* seg_of_token, const int* units, int n_units, int rows,
                                        float scale, void* out, float* part_o, float* part_ml, int T, int heads, int rank, int n_slices, int slice_keys,
-                                       unsigned* status, int window, cudaStream_t stream) {
+                                       unsigned* status, int window, const float* sink, cudaStream_t stream) {
   if (T == 0 || n_units == 0) return 0;
   IB_CHECK_ARG(kv && kv->base && kv->block_table && kv->kv_heads == 1 && kv->dtype == IB_BF16, "latent_attention_mma: a bfloat16 cache of one row per token is needed");
   const int D = kv->head_dim;
@@ -355,7 +360,7 @@ extern "C" int ib_latent_attention_mma(const float* q, const IbKvView* kv, const
   auto go = [&](auto kernel) {
     if (smem > 40 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     ib::launch(kernel, grid, kWarps * 32, smem, stream, q, *kv, positions, seg_of_token, (const int2*)units, scale, (__nv_bfloat16*)out, part_o, part_ml, heads, rank, D,
-               n_slices, slice_keys, status, window);
+               n_slices, slice_keys, status, window, sink);
   };
   auto pick = [&](auto nch) {
     constexpr int NCH = decltype(nch)::value;
@@ -367,6 +372,6 @@ extern "C" int ib_latent_attention_mma(const float* q, const IbKvView* kv, const
   else if (rank <= 256) pick(std::integral_constant<int, 2>());
   else pick(std::integral_constant<int, 4>());
   IB_CHECK_LAUNCH("latent_attention_mma");
-  if (n_slices > 1) return ib_latent_combine(part_o, part_ml, out, IB_BF16, T * heads, rank, n_slices, stream);
+  if (n_slices > 1) return ib_latent_combine(part_o, part_ml, out, IB_BF16, T * heads, rank, n_slices, sink, heads, stream);
   return 0;
 }

@@ -3,6 +3,7 @@
 // All arithmetic is float32; only a stored activation may be bfloat16.
 //
 //  * add_layernorm: v = x[t] + scale * (sum_p delta[p][t] + bias)   (scale, bias: per channel, optional; partial sums added in order)
+//                   (+ the partial sums of a second contribution, where two sublayers ran side by side on one normed input)
 //                   x[t] = v (optional), x_copy[t] = v (optional)
 //                   out = w * (v - mean(v)) / sqrt(mean((v - mean)^2) + eps) [+ b]
 //    With `halo` > 0 the output rows are laid out for the convolution that follows: segment s (tokens a..b of the flat batch) owns
@@ -29,6 +30,9 @@ struct LnExtras {
   const float* wb;   // the norm's bias per channel, or null
   float mult;        // factor on the contribution where there is no per-channel scale
   int early;         // 1: the kernels that follow may be scheduled while this one runs; 0: only when it is done (for the reason given in causal_conv_rows_kernel)
+  const float* delta2;   // add_layernorm: a second contribution of P2 partial sums (stride2 apart), added after the first; P2 = 0: none
+  int P2;
+  size_t stride2;
 };
 
 template <typename O>
@@ -63,8 +67,13 @@ __global__ void __launch_bounds__(kLnThreads) add_layernorm_kernel(float* __rest
         d = dbias ? a + d : a;
       }
       v = __fmaf_rn(dscale ? dscale[i] : ex.mult, d, v);
-      if (write_x) xr[i] = v;
     }
+    if (ex.P2 > 0) {
+      float a = ex.delta2[(size_t)t * H + i];
+      for (int p = 1; p < ex.P2; p++) a += ex.delta2[p * ex.stride2 + (size_t)t * H + i];
+      v += a;
+    }
+    if (write_x && (P > 0 || dbias || ex.P2 > 0)) xr[i] = v;
     if (x_copy) x_copy[(size_t)t * H + i] = v;
     row[i] = v;
     sum += v;
@@ -181,8 +190,13 @@ __global__ void __launch_bounds__(kLnThreads) add_layernorm_vec_kernel(float* __
         d = dbias ? add4(a, d) : a;
       }
       v = fma4(dscale ? ld4(dscale + i) : make_float4(ex.mult, ex.mult, ex.mult, ex.mult), d, v);
-      if (write_x) st4(xr + i, v);
     }
+    if (ex.P2 > 0) {
+      float4 a = ld4(ex.delta2 + (size_t)t * H + i);
+      for (int p = 1; p < ex.P2; p++) a = add4(a, ld4(ex.delta2 + p * ex.stride2 + (size_t)t * H + i));
+      v = add4(v, a);
+    }
+    if (write_x && (P > 0 || dbias || ex.P2 > 0)) st4(xr + i, v);
     if (x_copy) st4(x_copy + (size_t)t * H + i, v);
     st4(row + i, v);
     sum += (v.x + v.y) + (v.z + v.w);
@@ -491,10 +505,12 @@ __global__ void scale_values_kernel(float* __restrict__ v, size_t n, float s) {
 extern "C" int ib_add_layernorm(float* x, const float* delta, int P, long long delta_stride, const float* dscale, const float* dbias, const float* w, void* out,
                                 int out_dtype, const int* rows, int n_rows, int H, float eps, int write_x, float* x_copy, int halo, const int* seg_of_token,
                                 const int* seg_start, const int* seg_slot, int n_segments, const float* state, long long slot_stride, const float* wb,
-                                float mult, int early, cudaStream_t stream) {
+                                float mult, int early, const float* delta2, int P2, long long stride2, cudaStream_t stream) {
+  // delta2, P2, stride2: a second contribution (see LnExtras), P2 = 0 for none
   // wb: the norm's bias per channel, or null; mult: factor on the contribution where dscale is null; early: see LnExtras
   if (n_rows == 0) return 0;
-  const LnExtras ex = {wb, mult, early};
+  const LnExtras ex = {wb, mult, early, delta2, P2, (size_t)stride2};
+  IB_CHECK_ARG(P2 >= 0 && (P2 == 0 || delta2), "add_layernorm: a second contribution of %d partial sums is missing", P2);
   IB_CHECK_ARG(n_rows > 0 && H > 0 && P >= 0 && halo >= 0, "add_layernorm: bad sizes rows=%d H=%d P=%d halo=%d", n_rows, H, P, halo);
   IB_CHECK_ARG(!(halo && rows), "add_layernorm: gathered rows have no layout for a convolution");
   IB_CHECK_ARG(!halo || (seg_of_token && seg_start && seg_slot && state && n_segments > 0), "add_layernorm: the convolution's layout needs the step's segments and the state");
@@ -507,7 +523,8 @@ extern "C" int ib_add_layernorm(float* x, const float* delta, int P, long long d
                seg_start, seg_slot, state, (size_t)slot_stride, ex);
   };
   auto al = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
-  const bool vec = H % 4 == 0 && al(wb) && al(x) && al(delta) && delta_stride % 4 == 0 && al(dscale) && al(dbias) && al(w) && al(out) && al(x_copy) && al(state) && slot_stride % 4 == 0;
+  const bool vec = H % 4 == 0 && al(wb) && al(x) && al(delta) && delta_stride % 4 == 0 && al(dscale) && al(dbias) && al(w) && al(out) && al(x_copy) && al(state) && slot_stride % 4 == 0 &&
+                   al(delta2) && stride2 % 4 == 0;
   if (out_dtype != IB_F32 && out_dtype != IB_BF16) return ib_set_error("add_layernorm: unknown output dtype %d", out_dtype);
   if (vec && out_dtype == IB_F32) go(add_layernorm_vec_kernel<float>, (float*)out);
   else if (vec) go(add_layernorm_vec_kernel<__nv_bfloat16>, (__nv_bfloat16*)out);
@@ -625,7 +642,7 @@ extern "C" int ib_add_layernorm_mixes_single(float* x, const float* delta, int P
   if (T == 0) return 0;
   const size_t smem = (size_t)H * sizeof(float);
   IB_CHECK_ARG(T > 0 && H > 0 && P >= 0 && M > 0 && smem <= 200 * 1024, "add_layernorm_mixes_single: bad sizes T=%d H=%d P=%d mixes=%d", T, H, P, M);
-  const LnExtras ex = {wb, mult, early};
+  const LnExtras ex = {wb, mult, early, nullptr, 0, 0};
   auto go = [&](auto kernel, auto* o) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     ib::launch(kernel, (unsigned)T, kLnThreads, smem, stream, x, delta, P, (size_t)delta_stride, w, eps, mu, M, o, T, H, seg_slot, state, (size_t)slot_stride, ex);

@@ -140,7 +140,7 @@ __device__ __forceinline__ void route_token(const RouteArgs& a, int t, float* s,
     __syncwarp();
   }
   if (lane == 0) {
-    const float f = a.renorm ? a.route_scale / (chosen_sum > 0.f ? chosen_sum : 1.f) : a.route_scale;
+    const float f = a.renorm ? a.route_scale / (chosen_sum + 1e-20f) : a.route_scale;
     for (int r = 0; r < a.top; r++) a.wt_out[(size_t)t * a.row_out() + r] *= f;
   }
   for (int r = lane; r < a.always; r += 32) {
@@ -234,9 +234,10 @@ __global__ void __launch_bounds__(1024) moe_route_sort_kernel(RouteArgs a, int t
 template <typename X, typename W, typename O>
 __global__ void __launch_bounds__(256) gemm_grouped_kernel(const X* __restrict__ x, const int* __restrict__ src_row, const W* __restrict__ w,
                                                            O* __restrict__ out, const int* __restrict__ offsets, const int* __restrict__ tile_start, int E,
-                                                           int N, int K, int act) {
-  // act: 0 the product, 1 silu(gate) * up (w holds gate rows, then up rows), 2 the square of max(product, 0)
-  const bool gated = act == 1;
+                                                           int N, int K, int act, const float* __restrict__ limits, float slope) {
+  // act: 0 the product, 1 silu(gate) * up (w holds gate rows, then up rows), 2 the square of max(product, 0), 3 as 1 with clamped halves
+  // (limits: one an expert, slope: the sigmoid's)
+  const bool gated = act == 1 || act == 3;
   constexpr int BK = 16;
   __shared__ float xs[BK][SM_ + 1];
   __shared__ float ws[BK][64 + 1];
@@ -321,7 +322,7 @@ __global__ void __launch_bounds__(256) gemm_grouped_kernel(const X* __restrict__
       if (n >= N) continue;
       float v = acc[i][j];
       if (gated) {
-        v = (v / (1.f + expf(-v))) * acu[i][j];
+        v = act == 3 ? ib::clamped_glu<false>(v, acu[i][j], limits[e], slope) : (v / (1.f + expf(-v))) * acu[i][j];
       } else if (act == 2) {
         v = ib::relu2(v);
       }
@@ -479,13 +480,13 @@ extern "C" int ib_moe_sort(const int* idx, int R, int top, int E, int tile_rows,
 }
 
 extern "C" int ib_gemm_grouped(const void* x, int x_dtype, const int* src_row, const void* w, int w_dtype, void* out, int out_dtype, const int* offsets,
-                               const int* tile_start, int R, int E, int N, int K, int act, cudaStream_t stream) {
+                               const int* tile_start, int R, int E, int N, int K, int act, const float* limits, float slope, cudaStream_t stream) {
   if (R == 0 || N == 0) return 0;
-  IB_CHECK_ARG(act >= 0 && act <= 2, "gemm_grouped: activation %d is not known (0: none, 1: gated SiLU, 2: squared ReLU)", act);
+  IB_CHECK_ARG(act >= 0 && act <= 3 && (act != 3 || limits), "gemm_grouped: activation %d is not known (0: none, 1: gated SiLU, 2: squared ReLU, 3: gated, clamped)", act);
   IB_CHECK_ARG(R > 0 && E > 0 && N > 0 && K > 0, "gemm_grouped: bad sizes rows=%d experts=%d N=%d K=%d", R, E, N, K);
   dim3 grid((N + 63) / 64, R / SM_ + E);   // no more tiles than this, whatever the counts
   IB_CHECK_ARG(grid.y <= 65535, "gemm_grouped: %d rows exceed the grid limit", R);
-  auto go = [&](auto kernel, auto* xp, auto* wp, auto* op) { ib::launch(kernel, grid, 256, 0, stream, xp, src_row, wp, op, offsets, tile_start, E, N, K, act); };
+  auto go = [&](auto kernel, auto* xp, auto* wp, auto* op) { ib::launch(kernel, grid, 256, 0, stream, xp, src_row, wp, op, offsets, tile_start, E, N, K, act, limits, slope); };
   using bf = __nv_bfloat16;
   if (x_dtype == IB_F32 && w_dtype == IB_F32 && out_dtype == IB_F32) go(gemm_grouped_kernel<float, float, float>, (const float*)x, (const float*)w, (float*)out);
   else if (x_dtype == IB_BF16 && w_dtype == IB_BF16 && out_dtype == IB_F32) go(gemm_grouped_kernel<bf, bf, float>, (const bf*)x, (const bf*)w, (float*)out);

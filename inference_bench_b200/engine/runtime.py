@@ -61,6 +61,12 @@ class Runtime:
         self.lib.ib_set_pdl(1 if self.options.pdl else 0)
         self.lib.ib_set_wait_limit_ms(int(self.options.wait_limit_ms))
 
+    def next_in_order(self, ctx) -> None:
+        """In a step with prompt portions: the next kernel starts only when everything before it is done. For a place where a third kernel in a
+        row would ask for tensor memory: while the first still holds it and the second waits for it, the third must not be served first."""
+        if not ctx.fixed_shape and ctx.n_segments != ctx.n_tokens:
+            self.lib.ib_pdl_skip_next()
+
     # ---------------------------------------------------------------- memory
     def empty(self, shape, dtype=None) -> torch.Tensor:
         return torch.empty(shape, dtype=dtype or self.act_dtype, device=self.device)
@@ -103,8 +109,8 @@ class Runtime:
         ops.gemm_simt(x, lw.weight, out[0])
         return out
 
-    def gate_up_act(self, x: torch.Tensor, lw: LinearWeights) -> torch.Tensor:
-        """x [T, K] -> silu(x gate^T) * (x up^T) in the activation dtype, [T, I], for a matrix
+    def gate_up_act(self, x: torch.Tensor, lw: LinearWeights, clamp: Optional[ops.Clamp] = None) -> torch.Tensor:
+        """x [T, K] -> silu(x gate^T) * (x up^T) (with `clamp` the pair with clamped halves) in the activation dtype, [T, I], for a matrix
         [2I, K] of gate rows then up rows. Enough bfloat16 tokens run as one tensor-core kernel
         whose epilogue applies the activation; otherwise the product and the SiLU-mul kernel."""
         T, inter = x.shape[0], lw.n // 2
@@ -112,11 +118,11 @@ class Runtime:
             from ..kernels import gemm_tcgen05
             if self.options.swiglu_epilogue and gemm_tcgen05.swiglu_supported(T, lw.k, inter):
                 act = self.empty((T, inter))
-                gemm_tcgen05.gemm_swiglu(x, lw.weight, act, self.status, pair_min_tokens=self.options.pair_min_tokens)
+                gemm_tcgen05.gemm_swiglu(x, lw.weight, act, self.status, pair_min_tokens=self.options.pair_min_tokens, clamp=clamp)
                 return act
         gu = self.linear(x, lw)
         act = self.empty((T, inter))
-        ops.silu_mul(gu, act)
+        ops.silu_mul(gu, act, clamp)
         return act
 
     def up_act(self, x: torch.Tensor, lw: LinearWeights, kind: str, pq: Optional[torch.Tensor] = None) -> torch.Tensor:

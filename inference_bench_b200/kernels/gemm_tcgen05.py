@@ -20,9 +20,9 @@ FITTED_SM_COUNT = 148   # the part the cost model below was fitted on; every fun
 TOKEN_TILES = (16, 32, 64, 128, 256)
 
 L.register("ib_gemm_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._i, L._p, L._p])
-L.register("ib_gemm_swiglu_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p, L._p])
+L.register("ib_gemm_swiglu_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p, L._f, L._p, L._p])
 L.register("ib_gemm_tcgen05_2cta", [L._p, L._p, L._p, L._i, L._i, L._i, L._p, L._p])
-L.register("ib_gemm_swiglu_tcgen05_2cta", [L._p, L._p, L._p, L._i, L._i, L._i, L._p, L._p])
+L.register("ib_gemm_swiglu_tcgen05_2cta", [L._p, L._p, L._p, L._i, L._i, L._i, L._p, L._f, L._p, L._p])
 L.register("ib_gemm_xielu_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p, L._p, L._p])
 L.register("ib_gemm_xielu_tcgen05_2cta", [L._p, L._p, L._p, L._i, L._i, L._i, L._p, L._p, L._p])
 L.register("ib_gemm_relu2_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p, L._p])
@@ -33,7 +33,7 @@ L.register("ib_gemm_qkv_tcgen05_2cta", [L._p, L._p, L._i, L._i, L._p, L._p, L._f
 L.register("ib_gemm_grouped_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._p, L._p, L._i, L._p, L._p])
 L.register("ib_gemm_parts_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._i, L._p, L._p])
 L.register("ib_gemm_grouped_relu2_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._p, L._p, L._i, L._p, L._p])
-L.register("ib_gemm_grouped_swiglu_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._p, L._p, L._i, L._p, L._p])
+L.register("ib_gemm_grouped_swiglu_tcgen05", [L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._p, L._p, L._i, L._p, L._f, L._p, L._p])
 
 # Runtime options that steer the choice (config/runtime_options.py): `pair_min_tokens` (129: the fused gate/up product runs on the
 # persistent CTA-pair kernel, csrc/gemm_tcgen05_2cta.cu, from here on whatever its size), `pair_always_tokens` (2,048: every
@@ -237,8 +237,8 @@ def half_swiglu(T: int, inter: int) -> bool:
 
 
 def gemm_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, status: torch.Tensor, bn: int | None = None, pair_min_tokens: int = 129,
-                half: bool | None = None) -> None:
-    """act [T, I] bfloat16 = silu(x gate^T) * (x up^T) with w_gate_up [2I, K] = gate rows then up rows."""
+                half: bool | None = None, clamp: Optional["ops.Clamp"] = None) -> None:
+    """act [T, I] bfloat16 = silu(x gate^T) * (x up^T) (or the clamped pair) with w_gate_up [2I, K] = gate rows then up rows."""
     T, K = x.shape
     I = w_gate_up.shape[0] // 2
     ops._check("x", x, torch.bfloat16)
@@ -249,11 +249,11 @@ def gemm_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, sta
     if half is None:
         half = bn in (16, 32)
     if bn is None and (T >= pair_min_tokens or (T > 32 and -(-I // 256) >= PAIR_SWIGLU_MIN_TILES)):
-        L.call("ib_gemm_swiglu_tcgen05_2cta", x.data_ptr(), w_gate_up.data_ptr(), act.data_ptr(), T, I, K, status.data_ptr(), ops._stream())
+        L.call("ib_gemm_swiglu_tcgen05_2cta", x.data_ptr(), w_gate_up.data_ptr(), act.data_ptr(), T, I, K, *ops._clamp_args(clamp), status.data_ptr(), ops._stream())
         return
     if bn is None:
         bn = 64 if T <= 64 else (128 if T <= 128 else 256)
-    L.call("ib_gemm_swiglu_tcgen05", x.data_ptr(), w_gate_up.data_ptr(), act.data_ptr(), T, I, K, bn, 1 if half else 0, status.data_ptr(), ops._stream())
+    L.call("ib_gemm_swiglu_tcgen05", x.data_ptr(), w_gate_up.data_ptr(), act.data_ptr(), T, I, K, bn, 1 if half else 0, *ops._clamp_args(clamp), status.data_ptr(), ops._stream())
 
 
 ACT_MIN_ROW_BLOCKS = 32   # 128-row blocks of the matrix from which up to 128 tokens keep the whole k-range in one CTA (that many CTAs fill the memory system)
@@ -344,12 +344,13 @@ def gemm_grouped_relu2(x: torch.Tensor, w: torch.Tensor, act: torch.Tensor, bn: 
     L.call("ib_gemm_grouped_relu2_tcgen05", x.data_ptr(), w.data_ptr(), act.data_ptr(), R, N, K, bn, offsets.data_ptr(), tiles.data_ptr(), E, status.data_ptr(), ops._stream())
 
 
-def gemm_grouped_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, bn: int, offsets: torch.Tensor, tiles: torch.Tensor, status: torch.Tensor) -> None:
-    """act [R, I] bfloat16 = silu(gate_e x) * (up_e x) per expert, w_gate_up [E, 2 I, K] = every expert's gate rows then its up rows."""
+def gemm_grouped_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, bn: int, offsets: torch.Tensor, tiles: torch.Tensor, status: torch.Tensor,
+                        clamp: Optional["ops.Clamp"] = None) -> None:
+    """act [R, I] bfloat16 = silu(gate_e x) * (up_e x) (or the clamped pair, one limit an expert) per expert, w_gate_up [E, 2 I, K] = every expert's gate rows then its up rows."""
     R, K = x.shape
     E, I2, _ = w_gate_up.shape
     ops._check("x", x, torch.bfloat16)
     ops._check("w_gate_up", w_gate_up, torch.bfloat16, (E, I2, K))
     ops._check("act", act, torch.bfloat16, (R, I2 // 2))
     L.call("ib_gemm_grouped_swiglu_tcgen05", x.data_ptr(), w_gate_up.data_ptr(), act.data_ptr(), R, I2 // 2, K, bn, offsets.data_ptr(), tiles.data_ptr(), E,
-           status.data_ptr(), ops._stream())
+           *ops._clamp_args(clamp, E), status.data_ptr(), ops._stream())

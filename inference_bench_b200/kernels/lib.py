@@ -58,13 +58,29 @@ class AttnTail(C.Structure):
     ]
 
 
+class MemoryGates(C.Structure):
+    """Mirror of IbMemoryGates in csrc/gated_recurrence.cu."""
+    _fields_ = [
+        ("i_src", C.c_void_p),
+        ("f_src", C.c_void_p),
+        ("P", C.c_int),
+        ("row", C.c_int),
+        ("stride", C.c_size_t),
+        ("i_bias", C.c_void_p),
+        ("f_bias", C.c_void_p),
+        ("cap", C.c_float),
+        ("m_state", C.c_void_p),
+        ("m_stride", C.c_size_t),
+    ]
+
+
 _p, _i, _f, _ll = C.c_void_p, C.c_int, C.c_float, C.c_longlong
 
 _SIGNATURES = {
     "ib_embed": [_p, _i, _p, _p, _i, _i, _i, _p, _p],
     "ib_add_rmsnorm": [_p, _p, _i, _ll, _p, _p, _i, _p, _i, _i, _f, _i, _p],
-    "ib_rope_table": [_p, _p, _p, _p, _i, _i, _p],
-    "ib_silu_mul": [_p, _i, _ll, _p, _i, _i, _i, _p],
+    "ib_rope_table": [_p, _p, _p, _p, _i, _i, _f, _p],
+    "ib_silu_mul": [_p, _i, _ll, _p, _i, _i, _i, _p, _f, _p],
     "ib_qk_norm_rope_kv": [_p, _i, _ll, _p, _p, _f, _p, _p, _i, _p, _p, _p, _i, C.POINTER(KvView), _i, _i, _i, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p],
     "ib_attention_generic": [_p, _i, C.POINTER(KvView), _p, _p, _i, _f, _p, _i, _i, _p, _i, _i, _f, _i, _i, _p, _p, _i, _ll, _i, _f, _i, _i, _p],
     "ib_gemm_simt": [_p, _i, _p, _i, _p, _i, _i, _i, _p],

@@ -191,21 +191,40 @@ def add_rmsnorm(x: torch.Tensor, delta: Optional[torch.Tensor], w: torch.Tensor,
            float(eps), 0 if rows is not None else 1, _stream())
 
 
-def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> None:
+def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, amplitude: float = 1.0) -> None:
+    """cos[t, i], sin[t, i] = amplitude times the cosine and sine of positions[t] * inv_freq[i]."""
     T, half = positions.shape[0], inv_freq.shape[0]
     _check("positions", positions, torch.int32)
     _check("inv_freq", inv_freq, torch.float32)
     _check("cos", cos, torch.float32, (T, half))
     _check("sin", sin, torch.float32, (T, half))
-    L.call("ib_rope_table", positions.data_ptr(), inv_freq.data_ptr(), cos.data_ptr(), sin.data_ptr(), T, half, _stream())
+    L.call("ib_rope_table", positions.data_ptr(), inv_freq.data_ptr(), cos.data_ptr(), sin.data_ptr(), T, half, float(amplitude), _stream())
 
 
-def silu_mul(gate_up: torch.Tensor, act: torch.Tensor) -> None:
-    """act = silu(gate) * up with gate_up float32 [P, T, 2I] = [gate | up], partials summed first."""
+@dataclass(frozen=True)
+class Clamp:
+    """A gated pair with clamped halves in the place of silu(gate) * up: g sigmoid(slope g) (u + 1) with g = min(gate, limit) and u = up cut to
+    [-limit, limit]. limits: float32 [n] on the device (one for a single matrix, one an expert for grouped products)."""
+    limits: torch.Tensor
+    slope: float
+
+    def args(self, n: int) -> tuple:
+        _check("limits", self.limits, torch.float32)
+        if self.limits.numel() < n:
+            raise L.KernelError(f"{self.limits.numel()} limits for {n} matrices")
+        return self.limits.data_ptr(), float(self.slope)
+
+
+def _clamp_args(clamp: Optional[Clamp], n: int = 1) -> tuple:
+    return (None, 0.0) if clamp is None else clamp.args(n)
+
+
+def silu_mul(gate_up: torch.Tensor, act: torch.Tensor, clamp: Optional[Clamp] = None) -> None:
+    """act = silu(gate) * up (or the clamped pair) with gate_up float32 [P, T, 2I] = [gate | up], partials summed first."""
     _check("gate_up", gate_up, torch.float32)
     P, T, I2 = gate_up.shape
     _check("act", act, None, (T, I2 // 2))
-    L.call("ib_silu_mul", gate_up.data_ptr(), P, T * I2, act.data_ptr(), dtype_code(act.dtype), T, I2 // 2, _stream())
+    L.call("ib_silu_mul", gate_up.data_ptr(), P, T * I2, act.data_ptr(), dtype_code(act.dtype), T, I2 // 2, *_clamp_args(clamp), _stream())
 
 
 def qk_norm_rope_kv(qkv: torch.Tensor, q_norm_w: Optional[torch.Tensor], k_norm_w: Optional[torch.Tensor], eps: float,
@@ -349,7 +368,7 @@ def cast_rows(x: torch.Tensor, act: torch.Tensor) -> None:
 L.register("ib_latent_prepare", [L._p, L._i, L._ll, L._i, L._p, L._f, L._p, L._p, L._i, L._p, L._p, L._p, L._i, L._p, C.POINTER(L.KvView), L._i, L._i, L._i, L._i,
                                  L._i, L._i, L._p, L._p])
 L.register("ib_gemm_heads", [L._p, L._i, L._ll, L._ll, L._p, L._i, L._p, L._i, L._ll, L._ll, L._i, L._i, L._i, L._i, L._p, L._i, L._ll, L._i, L._p])
-L.register("ib_latent_attention", [L._p, C.POINTER(L.KvView), L._p, L._p, L._f, L._p, L._i, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p, L._i, L._p])
+L.register("ib_latent_attention", [L._p, C.POINTER(L.KvView), L._p, L._p, L._f, L._p, L._i, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p, L._i, L._p, L._p])
 L.register("ib_latent_down", [L._p, L._i, L._ll, L._i, L._i, L._p, L._p, L._i, L._p, L._f, L._p, L._p, L._i, L._p, L._p, C.POINTER(L.KvView), L._i, L._i, L._i, L._p, L._p])
 L.KERNELS_PER_CALL["ib_latent_attention"] = 1   # two with slices; counted by the caller
 
@@ -379,7 +398,7 @@ def latent_prepare(qd: torch.Tensor, c_norm_w: Optional[torch.Tensor], eps: floa
            rot, rank, status.data_ptr(), _stream())
 
 
-L.register("ib_gemm_grouped_mma", [L._p, L._p, L._p, L._p, L._i, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p])
+L.register("ib_gemm_grouped_mma", [L._p, L._p, L._p, L._p, L._i, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p, L._f, L._p])
 L.register("ib_gemm_heads_mma", [L._p, L._ll, L._ll, L._p, L._p, L._i, L._ll, L._ll, L._i, L._i, L._i, L._i, L._p, L._i, L._ll, L._i, L._p])
 
 
@@ -438,15 +457,17 @@ def gemm_heads(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n: int, tens
 
 
 def latent_attention(q_full: torch.Tensor, kv: KvLayerView, positions: torch.Tensor, seg_of_token: torch.Tensor, scale: float, out: torch.Tensor, rank: int,
-                     n_slices: int, slice_keys: int, scratch, status: torch.Tensor, window: Optional[int] = None) -> None:
+                     n_slices: int, slice_keys: int, scratch, status: torch.Tensor, window: Optional[int] = None, sink: Optional[torch.Tensor] = None) -> None:
     """q_full float32 [T, heads, row] against the cached rows [latent (rank) | key part]: out [T, heads, rank] = softmax-weighted sum of
     the latents of the keys a token sees (all up to its own position, or with `window` itself and the window - 1 before it; the slices
-    then cut that range). scratch: (part_o, part_ml) float32 when n_slices > 1."""
+    then cut that range). sink: float32 [heads], a score per head without key or value that the softmax's denominator holds as well. scratch: (part_o, part_ml) float32 when n_slices > 1."""
     T, heads, D = q_full.shape
     _check("q_full", q_full, torch.float32)
     _check("out", out, None, (T, heads, rank))
     _check("positions", positions, torch.int32, (T,))
     _check("seg_of_token", seg_of_token, torch.int32, (T,))
+    if sink is not None:
+        _check("sink", sink, torch.float32, (heads,))
     view = kv.c_view()
     if view.head_dim != D:
         raise L.KernelError(f"latent_attention: queries have {D} values, cache rows {view.head_dim}")
@@ -458,10 +479,10 @@ def latent_attention(q_full: torch.Tensor, kv: KvLayerView, positions: torch.Ten
             raise L.KernelError("latent_attention: the scratch for the slices is too small")
         L.launches += 1
     L.call("ib_latent_attention", q_full.data_ptr(), C.byref(view), positions.data_ptr(), seg_of_token.data_ptr(), float(scale), out.data_ptr(),
-           dtype_code(out.dtype), _ptr(part_o), _ptr(part_ml), T, heads, rank, n_slices, slice_keys, status.data_ptr(), int(window or 0), _stream())
+           dtype_code(out.dtype), _ptr(part_o), _ptr(part_ml), T, heads, rank, n_slices, slice_keys, status.data_ptr(), int(window or 0), _ptr(sink), _stream())
 
 
-L.register("ib_latent_attention_mma", [L._p, C.POINTER(L.KvView), L._p, L._p, L._p, L._i, L._i, L._f, L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p, L._i, L._p])
+L.register("ib_latent_attention_mma", [L._p, C.POINTER(L.KvView), L._p, L._p, L._p, L._i, L._i, L._f, L._p, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p, L._i, L._p, L._p])
 
 
 def latent_attention_mma_rows(rank: int, row: int, rows_wanted: int) -> int:
@@ -475,7 +496,7 @@ def latent_attention_mma_supports(rank: int, row: int) -> bool:
 
 def latent_attention_mma(q_full: torch.Tensor, kv: KvLayerView, positions: torch.Tensor, seg_of_token: torch.Tensor, units: Optional[torch.Tensor], scale: float,
                          out: torch.Tensor, rank: int, n_slices: int, slice_keys: int, scratch, status: torch.Tensor, rows: int = 16,
-                         window: Optional[int] = None) -> None:
+                         window: Optional[int] = None, sink: Optional[torch.Tensor] = None) -> None:
     """The same as `latent_attention` on the tensor cores (bfloat16 cache and output). rows: query rows a CTA holds (16, 32 or 64).
     units: None (a CTA per token) or int32 [n, 2] of (first token, tokens): runs of consecutive tokens of one request that share a
     CTA's rows (at most rows // heads tokens each)."""
@@ -484,6 +505,8 @@ def latent_attention_mma(q_full: torch.Tensor, kv: KvLayerView, positions: torch
     _check("out", out, torch.bfloat16, (T, heads, rank))
     _check("positions", positions, torch.int32, (T,))
     _check("seg_of_token", seg_of_token, torch.int32, (T,))
+    if sink is not None:
+        _check("sink", sink, torch.float32, (heads,))
     view = kv.c_view()
     if view.head_dim != D:
         raise L.KernelError(f"latent_attention_mma: queries have {D} values, cache rows {view.head_dim}")
@@ -497,14 +520,14 @@ def latent_attention_mma(q_full: torch.Tensor, kv: KvLayerView, positions: torch
             raise L.KernelError("latent_attention_mma: the scratch for the slices is too small")
         L.launches += 1
     L.call("ib_latent_attention_mma", q_full.data_ptr(), C.byref(view), positions.data_ptr(), seg_of_token.data_ptr(), _ptr(units), n_units, int(rows), float(scale),
-           out.data_ptr(), _ptr(part_o), _ptr(part_ml), T, heads, rank, n_slices, slice_keys, status.data_ptr(), int(window or 0), _stream())
+           out.data_ptr(), _ptr(part_o), _ptr(part_ml), T, heads, rank, n_slices, slice_keys, status.data_ptr(), int(window or 0), _ptr(sink), _stream())
 
 
 # ---------------------------------------------------------------- routed experts (csrc/moe.cu)
 L.register("ib_moe_route", [L._p, L._i, L._ll, L._i, L._i, L._i, L._i, L._i, L._f, L._i, L._p, L._p, L._i, L._p, L._i, L._i, L._p, L._i, L._i, L._p])
 L.register("ib_moe_route_sort", [L._p, L._i, L._ll, L._i, L._i, L._i, L._i, L._i, L._f, L._i, L._p, L._p, L._i, L._p, L._i, L._i, L._p, L._i, L._i, L._i, L._p, L._p, L._p, L._p, L._p])
 ROUTE_SCORES = {"softmax": 0, "sigmoid": 1, "chosen_softmax": 2}
-GROUPED_ACTS = {"none": 0, "swiglu": 1, "relu2": 2}
+GROUPED_ACTS = {"none": 0, "swiglu": 1, "relu2": 2, "clamped_swiglu": 3}
 L.register("ib_scatter_scaled_rows", [L._p, L._i, L._p, L._p, L._i, L._p, L._i, L._i, L._p])
 L.register("ib_moe_sort", [L._p, L._i, L._i, L._i, L._i, L._p, L._p, L._p, L._p, L._p])
 L.register("ib_gather_rows", [L._p, L._p, L._p, L._i, L._i, L._i, L._p])
@@ -524,7 +547,7 @@ def gather_rows(x: torch.Tensor, src_row: torch.Tensor, out: torch.Tensor) -> No
     if x.shape[1] != K:
         raise L.KernelError(f"gather_rows: x has {x.shape[1]} columns, out {K}")
     L.call("ib_gather_rows", x.data_ptr(), src_row.data_ptr(), out.data_ptr(), R, K, x.element_size(), _stream())
-L.register("ib_gemm_grouped", [L._p, L._i, L._p, L._p, L._i, L._p, L._i, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p])
+L.register("ib_gemm_grouped", [L._p, L._i, L._p, L._p, L._i, L._p, L._i, L._p, L._p, L._i, L._i, L._i, L._i, L._i, L._p, L._f, L._p])
 L.register("ib_moe_combine", [L._p, L._p, L._p, L._i, L._p, L._i, L._ll, L._p, L._i, L._i, L._p, L._i, L._ll, L._i, L._p])
 
 
@@ -580,13 +603,13 @@ def moe_sort(idx: torch.Tensor, n_experts: int, offsets: torch.Tensor, tile_star
 
 
 def gemm_grouped(x: torch.Tensor, src_row: Optional[torch.Tensor], w: torch.Tensor, out: torch.Tensor, offsets: torch.Tensor, tile_start: torch.Tensor,
-                 gated: bool, tensor_cores: bool = False, act: str = "none") -> None:
+                 gated: bool, tensor_cores: bool = False, act: str = "none", clamp: Optional[Clamp] = None) -> None:
     """out[r] = w[e(r)] x[src_row[r] or r] for the regrouped rows r (expert e's rows are offsets[e]..offsets[e+1]); w [E, N or 2N, K]; with
-    `gated`, w holds gate rows then up rows and out = silu(gate) * up; act "relu2" (not gated): out = max(product, 0)^2."""
+    `gated`, w holds gate rows then up rows and out = silu(gate) * up (with `clamp`, one limit an expert, the clamped pair); act "relu2" (not gated): out = max(product, 0)^2."""
     R, N = out.shape
     if act not in ("none", "relu2") or (gated and act != "none"):
         raise L.KernelError(f"gemm_grouped: activation {act!r} (none, relu2; a gated product has its own)")
-    code = GROUPED_ACTS["swiglu" if gated else act]
+    code = GROUPED_ACTS[("clamped_swiglu" if clamp is not None else "swiglu") if gated else act]
     E, rows_w, K = w.shape
     if rows_w != (2 * N if gated else N) or x.shape[1] != K:
         raise L.KernelError(f"gemm_grouped: w {tuple(w.shape)}, x {tuple(x.shape)}, out {tuple(out.shape)} do not fit (gated={gated})")
@@ -599,10 +622,10 @@ def gemm_grouped(x: torch.Tensor, src_row: Optional[torch.Tensor], w: torch.Tens
         if not rows_mma_fits(x, w):
             raise L.KernelError("gemm_grouped: the tensor-core kernel needs bfloat16 operands with an inner size that is a multiple of 8")
         L.call("ib_gemm_grouped_mma", x.data_ptr(), _ptr(src_row), w.data_ptr(), out.data_ptr(), dtype_code(out.dtype), offsets.data_ptr(), tile_start.data_ptr(), R, E,
-               N, K, code, _stream())
+               N, K, code, *_clamp_args(clamp, E), _stream())
         return
     L.call("ib_gemm_grouped", x.data_ptr(), dtype_code(x.dtype), _ptr(src_row), w.data_ptr(), dtype_code(w.dtype), out.data_ptr(), dtype_code(out.dtype),
-           offsets.data_ptr(), tile_start.data_ptr(), R, E, N, K, code, _stream())
+           offsets.data_ptr(), tile_start.data_ptr(), R, E, N, K, code, *_clamp_args(clamp, E), _stream())
 
 
 def scatter_scaled_rows(x: torch.Tensor, row_of_pair: torch.Tensor, wt: torch.Tensor, out: torch.Tensor) -> None:
@@ -645,7 +668,7 @@ def moe_combine(y: torch.Tensor, row_of_pair: torch.Tensor, wt: torch.Tensor, ba
 
 # ---------------------------------------------------------------- layer norm, input convolution, depth average (csrc/layernorm.cu)
 L.register("ib_add_layernorm", [L._p, L._p, L._i, L._ll, L._p, L._p, L._p, L._p, L._i, L._p, L._i, L._i, L._f, L._i, L._p, L._i, L._p, L._p, L._p, L._i, L._p, L._ll, L._p, L._f,
-                               L._i, L._p])
+                               L._i, L._p, L._i, L._ll, L._p])
 L.register("ib_softcap_values", [L._p, L._ll, L._f, L._p])
 L.register("ib_embed_layernorm", [L._p, L._i, L._p, L._p, L._p, L._f, L._p, L._i, L._i, L._i, L._p, L._p])
 L.register("ib_shift_mixes", [L._p, L._p, L._i, L._p, L._ll, L._p, L._p, L._p, L._p, L._i, L._i, L._i, L._p])
@@ -673,8 +696,9 @@ class ConvLayout:
 
 def add_layernorm(x: torch.Tensor, delta: Optional[torch.Tensor], w: torch.Tensor, out: torch.Tensor, eps: float, rows: Optional[torch.Tensor] = None,
                   delta_scale: Optional[torch.Tensor] = None, delta_bias: Optional[torch.Tensor] = None, x_copy: Optional[torch.Tensor] = None,
-                  layout: Optional[ConvLayout] = None, b: Optional[torch.Tensor] = None, delta_mult: float = 1.0, early: bool = True) -> None:
-    """v = x + delta_scale * (sum_p delta[p] + delta_bias) (x updated in place unless `rows` gathers); x_copy = v (optional);
+                  layout: Optional[ConvLayout] = None, b: Optional[torch.Tensor] = None, delta_mult: float = 1.0, early: bool = True,
+                  delta2: Optional[torch.Tensor] = None) -> None:
+    """delta2: a second contribution, float32 [P2, T, H], added after the first as it is. v = x + delta_scale * (sum_p delta[p] + delta_bias) (x updated in place unless `rows` gathers); x_copy = v (optional);
     out = w * (v - mean) / sqrt(var + eps) (+ b, float32 [H]). delta_mult: a constant in the place of delta_scale. early: whether the kernels that
     follow may be scheduled while this one runs. With `layout` out is float32 [T + halo * segments, H] in the layout of `ConvLayout`."""
     T, H = x.shape
@@ -698,10 +722,11 @@ def add_layernorm(x: torch.Tensor, delta: Optional[torch.Tensor], w: torch.Tenso
     if rows is not None:
         _check("rows", rows, torch.int32)
     lay = layout
+    d2_ptr, P2, stride2 = _delta(x, delta2)
     L.call("ib_add_layernorm", x.data_ptr(), _ptr(delta), P, stride, _ptr(delta_scale), _ptr(delta_bias), w.data_ptr(), out.data_ptr(), dtype_code(out.dtype),
            _ptr(rows), n_rows, H, float(eps), 0 if rows is not None else 1, _ptr(x_copy), lay.halo if lay else 0, _ptr(lay.seg_of_token) if lay else None,
            _ptr(lay.seg_start) if lay else None, _ptr(lay.seg_slot) if lay else None, lay.n_segments if lay else 0, _ptr(lay.state) if lay else None,
-           lay.slot_stride if lay else 0, _ptr(b), float(delta_mult), 1 if early else 0, _stream())
+           lay.slot_stride if lay else 0, _ptr(b), float(delta_mult), 1 if early else 0, d2_ptr, P2, stride2, _stream())
 
 
 def causal_conv_rows(ext: torch.Tensor, w: torch.Tensor, out: torch.Tensor, layout: ConvLayout) -> None:
@@ -955,6 +980,67 @@ def recurrence(form: str, q: Parts, k: Parts, v: Parts, head_param: torch.Tensor
     walk(m, None, chunks, chunk_state, chunk_decay, qa)
     L.call("ib_recurrence_chunks_finish", long_segs.data_ptr(), long_segs.shape[0], chunks.data_ptr(), m, seg_slot.data_ptr(), state.data_ptr(), heads * dim * vdim,
            chunk_state.data_ptr(), chunk_decay.data_ptr(), qa.data_ptr(), out.data_ptr(), heads, dim, vdim, _stream())
+
+
+L.register("ib_memory_walk", [L._p, L._p, L._p, L._i, L._ll, L._i, C.POINTER(L.MemoryGates), L._p, L._f, L._p, L._ll, L._p, L._p, L._i, L._p, L._i, L._i, L._i, L._p, L._p,
+                              L._p, L._p, L._p, L._p])
+L.register("ib_memory_gates", [C.POINTER(L.MemoryGates), L._p, L._p, L._i, L._p, L._p, L._i, L._p])
+L.register("ib_memory_out", [L._p, L._p, C.POINTER(L.MemoryGates), L._p, L._p, L._f, L._p, L._i, L._ll, L._i, L._p, L._i, L._i, L._i, L._i, L._p])
+
+
+def memory_recurrence(q: Parts, k: Parts, v: Parts, gate: Parts, i_gate: Parts, f_gate: Parts, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, state: torch.Tensor,
+                      m_state: torch.Tensor, seg_start: torch.Tensor, seg_slot: torch.Tensor, n_segments: int, norm_w: torch.Tensor, eps: float, out: torch.Tensor, heads: int,
+                      dim: int, vdim: int, single_tokens: bool, seg_list: Optional[torch.Tensor] = None, long_segs: Optional[torch.Tensor] = None,
+                      chunks: Optional[torch.Tensor] = None) -> None:
+    """The matrix memory with exponential gates over float32 partial sums of q, k (heads * dim columns), v, gate (heads * vdim) and the gates'
+    pre-activations (heads). With i = cap tanh((i_gate + i_bias) / cap), f = logsigmoid(cap tanh((f_gate + f_bias) / cap)), m = max(f + m, i):
+    S <- e^(f + m_old - m) S + e^(i - m) k [v | 1]^T, u = S^T q / sqrt(dim), o = u[:vdim] / (max(|u[vdim]|, e^(-m)) + 1e-6);
+    out [T, heads * vdim] = norm_w * o / rms(o) * sigmoid(gate). state float32 [slots, heads, dim, vdim + 1] and m_state float32 [slots, heads] are
+    advanced in place. single_tokens: every segment brings one token (two kernels instead of three). seg_list, long_segs, chunks: as for
+    `gated_recurrence`."""
+    T, V = out.shape[0], vdim
+    _check("out", out, None, (T, heads * V))
+    if len({(p.count, p.stride, p.row) for p in (q, k, v)}) != 1 or (i_gate.count, i_gate.stride, i_gate.row) != (f_gate.count, f_gate.stride, f_gate.row):
+        raise L.KernelError("memory_recurrence: q, k and v, and the two gates, must be laid out alike")
+    for name, p, n in (("q", q, heads * dim), ("k", k, heads * dim), ("v", v, heads * V), ("gate", gate, heads * V), ("i_gate", i_gate, heads), ("f_gate", f_gate, heads)):
+        _check(name, p.tensor, torch.float32)
+        if p.row < n or p.offset + (p.count - 1) * p.stride + (T - 1) * p.row + n > p.tensor.numel():
+            raise L.KernelError(f"memory_recurrence: {name} does not hold {T} rows of {n} entries in {p.count} partial sums")
+    _check("i_bias", i_bias, torch.float32, (heads,))
+    _check("f_bias", f_bias, torch.float32, (heads,))
+    _check("norm_w", norm_w, torch.float32, (heads * V,))
+    _check("state", state, torch.float32)
+    _check("m_state", m_state, torch.float32)
+    if tuple(state.shape[1:]) != (heads, dim, V + 1) or tuple(m_state.shape[1:]) != (heads,):
+        raise L.KernelError(f"memory_recurrence: the states must be [slots, {heads}, {dim}, {V + 1}] and [slots, {heads}], got {tuple(state.shape)} and {tuple(m_state.shape)}")
+    _check("seg_start", seg_start, torch.int32)
+    _check("seg_slot", seg_slot, torch.int32)
+    if single_tokens and n_segments != T:
+        raise L.KernelError(f"memory_recurrence: {T} rows in {n_segments} segments (every segment must bring one token)")
+    new = lambda *shape: torch.empty(shape, dtype=torch.float32, device=out.device)
+    g = L.MemoryGates(i_src=i_gate.ptr(), f_src=f_gate.ptr(), P=i_gate.count, row=i_gate.row, stride=i_gate.stride, i_bias=i_bias.data_ptr(), f_bias=f_bias.data_ptr(),
+                      cap=float(cap), m_state=m_state.data_ptr(), m_stride=m_state.stride(0))
+    o, gates, bound = new(T, heads, V + 1), None, None
+    if not single_tokens:
+        gates, bound = new(T, heads, 2), new(T, heads)
+        L.call("ib_memory_gates", C.byref(g), seg_start.data_ptr(), seg_slot.data_ptr(), n_segments, gates.data_ptr(), bound.data_ptr(), heads, _stream())
+
+    def walk(n, segs, table, chunk_state, chunk_decay, qa):
+        L.call("ib_memory_walk", q.ptr(), k.ptr(), v.ptr(), q.count, q.stride, q.row, C.byref(g), _ptr(gates), float(dim) ** -0.5, state.data_ptr(), heads * dim * (V + 1),
+               seg_start.data_ptr(), seg_slot.data_ptr(), n, o.data_ptr(), heads, dim, V, _ptr(segs), _ptr(table), _ptr(chunk_state), _ptr(chunk_decay), _ptr(qa), _stream())
+
+    if long_segs is None:
+        walk(n_segments if seg_list is None else seg_list.shape[0], seg_list, None, None, None, None)
+    else:
+        if seg_list is not None and seg_list.shape[0]:
+            walk(seg_list.shape[0], seg_list, None, None, None, None)
+        m = chunks.shape[0]
+        chunk_state, chunk_decay, qa = new(m, heads, dim, V + 1), new(m, heads, dim), new(T, heads, dim)
+        walk(m, None, chunks, chunk_state, chunk_decay, qa)
+        L.call("ib_recurrence_chunks_finish", long_segs.data_ptr(), long_segs.shape[0], chunks.data_ptr(), m, seg_slot.data_ptr(), state.data_ptr(), heads * dim * (V + 1),
+               chunk_state.data_ptr(), chunk_decay.data_ptr(), qa.data_ptr(), o.data_ptr(), heads, dim, V + 1, _stream())
+    L.call("ib_memory_out", o.data_ptr(), _ptr(bound), C.byref(g), seg_slot.data_ptr(), norm_w.data_ptr(), float(eps), gate.ptr(), gate.count, gate.stride, gate.row,
+           out.data_ptr(), dtype_code(out.dtype), T, heads, V, _stream())
 
 
 def decay_rows(low: torch.Tensor, w2: torch.Tensor, w0: torch.Tensor, decay: torch.Tensor) -> None:
@@ -1297,3 +1383,40 @@ def diff_combine(a: torch.Tensor, lam: float, eps: float, factor: float, out: to
     if n % v_dim:
         raise L.KernelError(f"diff_combine: rows of {n} entries are not whole heads of {v_dim}")
     L.call("ib_diff_combine", a.data_ptr(), dtype_code(a.dtype), float(lam), float(eps), float(factor), out.data_ptr(), T * (n // v_dim), v_dim, _stream())
+
+
+# ---------------------------------------------------------------- norms over whole query and key rows, mixed values (csrc/row_norm_qkv.cu)
+L.register("ib_row_norm_qkv", [L._p, L._i, L._ll, L._i, L._p, L._p, L._f, L._p, L._p, L._i, L._p, L._p, L._p, L._i, C.POINTER(L.KvView), L._i, L._i, L._i, L._i, L._p, L._p,
+                               L._p, L._p, L._p])
+
+
+def row_norm_qkv(proj: torch.Tensor, q_w: torch.Tensor, k_w: torch.Tensor, eps: float, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], positions: torch.Tensor,
+                 seg_of_token: torch.Tensor, q_out: torch.Tensor, kv: KvLayerView, heads: int, dim: int, v_dim: int, status: torch.Tensor, mix: Optional[torch.Tensor] = None,
+                 first: Optional[torch.Tensor] = None, keep: Optional[torch.Tensor] = None) -> None:
+    """proj float32 [P, T, R] = [heads x dim | kv_heads x dim | kv_heads x v_dim]: q and k divided by the root mean square of the token's whole query or
+    key row, times q_w [heads * dim] or k_w [kv_heads * dim], turned by cos and sin ([T, n]: entry i of a head with i + n; None: not); q_out
+    [T, heads * dim], keys and values into the paged cache. mix (float32 [1]): values (1 - mix) v + mix first, first float32 [T, kv_heads * v_dim];
+    keep float32 [T, kv_heads * v_dim]: receives the values as projected."""
+    _check("proj", proj, torch.float32)
+    P, T, R = proj.shape
+    view = kv.c_view()
+    G = view.kv_heads
+    if R != (heads + G) * dim + G * v_dim:
+        raise L.KernelError(f"row_norm_qkv: the projection has {R} columns, expected {(heads + G) * dim + G * v_dim}")
+    _check("q_w", q_w, torch.float32, (heads * dim,))
+    _check("k_w", k_w, torch.float32, (G * dim,))
+    _check("q_out", q_out, None, (T, heads * dim))
+    _check("positions", positions, torch.int32, (T,))
+    _check("seg_of_token", seg_of_token, torch.int32, (T,))
+    half = 0
+    if cos is not None:
+        half = cos.shape[1]
+        _check("cos", cos, torch.float32, (T, half))
+        _check("sin", sin, torch.float32, (T, half))
+    if mix is not None:
+        _check("mix", mix, torch.float32, (1,))
+        _check("first", first, torch.float32, (T, G * v_dim))
+    if keep is not None:
+        _check("keep", keep, torch.float32, (T, G * v_dim))
+    L.call("ib_row_norm_qkv", proj.data_ptr(), P, T * R, R, q_w.data_ptr(), k_w.data_ptr(), float(eps), _ptr(cos), _ptr(sin), half, positions.data_ptr(),
+           seg_of_token.data_ptr(), q_out.data_ptr(), dtype_code(q_out.dtype), C.byref(view), T, heads, dim, v_dim, _ptr(mix), _ptr(first), _ptr(keep), status.data_ptr(), _stream())

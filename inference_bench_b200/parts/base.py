@@ -31,6 +31,7 @@ class WeightSpec:
     "unit":   per-channel mixing weights, used in float32; random U(0, 1)
     "log_rate": logarithms of decay rates, used in float32; random log U(0.5, 8)
     "decay_bias": what a decay exp(-exp(z)) adds to z, used in float32; random U(-6, 0)
+    "keep_bias": what a forget gate's pre-activation gets added so that it mostly keeps, used in float32; random U(2, 6)
     "mix":    weights of an average over the n entries of the tensor's last axis, used in float32; random around 1 / n
     "table":  integer table, int32.
     `free` lists the axes whose size the checkpoint decides (the shape's entry there is what random weights are made with)."""
@@ -120,7 +121,16 @@ class ScaledDelta:
     scale: float
 
 
+@dataclass
+class SummedDelta:
+    """Two contributions to the residual stream that are added one after the other: what a block whose sublayers run side by side leaves for
+    the next norm; `Norm.takes_summed_delta` says whether a norm can add one."""
+    first: torch.Tensor     # float32 [P, T, H]
+    second: torch.Tensor    # float32 [P2, T, H]
+
+
 class Norm(Part):
+    takes_summed_delta = False   # True: `forward` takes a `SummedDelta` as delta
     takes_scaled_delta = False   # True: `forward` takes a `ScaledDelta` as delta
     takes_normed_delta = False   # True: `forward` takes a `NormedDelta` as delta
 

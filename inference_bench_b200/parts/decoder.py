@@ -86,6 +86,8 @@ class Decoder:
             return out + pending.norm.w * (y * torch.rsqrt((y * y).mean(-1, keepdim=True) + pending.norm.eps))
         if isinstance(pending, base.ScaledDelta):
             return out + pending.scale * pending.delta.sum(0).index_select(0, rows)
+        if isinstance(pending, base.SummedDelta):
+            return out + pending.first.sum(0).index_select(0, rows) + pending.second.sum(0).index_select(0, rows)
         if pending is not None:
             for p in range(pending.shape[0]):
                 out = out + pending[p].index_select(0, rows)

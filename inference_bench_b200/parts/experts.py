@@ -11,11 +11,15 @@ its n largest choice scores (experts of groups that do not stay cannot be chosen
 reads, out = sum_e down_e(silu(gate_e (weight_e h)) * up_e (weight_e h)), which is not the same thing for a gated expert.
 `score="chosen_softmax"`: the `top` experts with the largest logits are chosen and weighted by the softmax over the chosen logits alone;
 `router_bias` names a bias of the logits. `activation="relu2"`: experts and shared expert without a gate, down_e(max(up_e h, 0)^2).
+`activation="clamped_swiglu"` with clamp = (limit, slope): gated with clamped halves, g sigmoid(slope g) (u + 1) with g = min(gate, limit) and
+u = up cut to [-limit, limit]; the shared expert has a limit of its own (`shared_limit`).
 `shared_gate` names a vector (one row): the shared expert's output is multiplied by the sigmoid of its product with the token's row.
 The step's (token, expert) pairs are regrouped by expert on the device (no trip to the host, so the step can be captured),
 the experts' products run on the regrouped rows, and the weighted sum returns them to token order.
 """
 from __future__ import annotations
+
+from typing import Optional
 
 import torch
 
@@ -33,12 +37,17 @@ ROUTE_SORT_TOKENS = 32  # up to here the choice and the regrouping are one kerne
 class RoutedExperts(base.FeedForward):
     def __init__(self, prefix: str, hidden: int, expert_ff: int, experts: int, top: int, route_scale: float = 1.0, groups: int = 1, groups_keep: int = 1,
                  shared_ff: int = 0, renorm: bool = False, names: tuple = ("router", "e{}", "shared", "gate", "up", "down"), score: str = "softmax",
-                 weight_on: str = "output", correction: str = "", group_top: int = 1, activation: str = "swiglu", router_bias: str = "", shared_gate: str = ""):
+                 weight_on: str = "output", correction: str = "", group_top: int = 1, activation: str = "swiglu", router_bias: str = "", shared_gate: str = "",
+                 clamp: Optional[tuple] = None, shared_limit: float = 0.0):
         if not 0 < top <= experts or experts % groups or not 0 < groups_keep <= groups:
             raise ValueError(f"top {top} of {experts} experts in {groups} groups of which {groups_keep} stay")
-        if activation not in ("swiglu", "relu2"):
-            raise ValueError(f"activation {activation!r} is not known (swiglu, relu2)")
-        self.gated, self.router_bias, self.shared_gate = activation == "swiglu", router_bias, shared_gate if shared_ff else ""
+        if activation not in ("swiglu", "relu2", "clamped_swiglu"):
+            raise ValueError(f"activation {activation!r} is not known (swiglu, relu2, clamped_swiglu)")
+        if (clamp is not None) != (activation == "clamped_swiglu") or (clamp is not None and (not clamp[0] > 0 or (shared_ff and not shared_limit > 0))):
+            raise ValueError("the clamped activation, and no other, takes clamp = (limit, slope), and with a shared expert a limit for it")
+        self.gated, self.router_bias, self.shared_gate = activation != "relu2", router_bias, shared_gate if shared_ff else ""
+        self.clamp, self.shared_limit = clamp, float(shared_limit)
+        self.limits = self.shared_clamp = None      # `ops.Clamp` of the experts (then the shared expert's blocks), and of the shared expert alone
         self.b_router, self.blocks = None, 0
         if score not in ops.ROUTE_SCORES or weight_on not in ("output", "input"):
             raise ValueError(f"score {score!r} ({', '.join(ops.ROUTE_SCORES)}) or weight_on {weight_on!r} (output, input) is not known")
@@ -85,18 +94,29 @@ class RoutedExperts(base.FeedForward):
         # [experts, gate rows then up rows, width] and [experts, width, inner]: one tensor each, so a tile of the grouped product finds its expert by an offset
         front = (0, 1) if self.gated else (1,)
         S, F = self.shared_ff, self.expert_ff
-        self.blocks = S // F if S and S % F == 0 and not self.gated and self.weight_on == "output" else 0
+        self.blocks = S // F if S and S % F == 0 and (not self.gated or self.clamp is not None) and self.weight_on == "output" else 0
         gu = [torch.cat([weights[self._expert(k, i)] for i in front], dim=0) for k in range(self.experts)]
         down = [weights[self._expert(k, 2)] for k in range(self.experts)]
         if S:
             shared_gu, shared_d = torch.cat([weights[self._shared(i)] for i in front], dim=0), weights[self._shared(2)]
             # the shared expert's inner channels in blocks of a routed expert's size, behind the routed experts
-            gu += list(shared_gu.split(F)) if self.blocks else []
+            if self.blocks and self.gated:
+                gate, up = shared_gu.split(S)
+                gu += [torch.cat([gate[b:b + F], up[b:b + F]], dim=0) for b in range(0, S, F)]
+            elif self.blocks:
+                gu += list(shared_gu.split(F))
             down += list(shared_d.split(F, dim=1)) if self.blocks else []
         self.w_gu, self.w_d = rt.upload(torch.stack(gu), rt.act_dtype), rt.upload(torch.stack(down), rt.act_dtype)
         if S:
-            self.shared_gu = rt.matrix(self.w_gu[self.experts:].reshape(S, self.hidden) if self.blocks else shared_gu)   # (a view where the blocks hold it)
+            # (a view where the blocks hold it as it is: a gated one in several blocks has its gate and up rows elsewhere)
+            whole = self.blocks and (not self.gated or self.blocks == 1)
+            self.shared_gu = rt.matrix(self.w_gu[self.experts:].reshape(-1, self.hidden) if whole else shared_gu)
             self.shared_d = rt.matrix(self.w_d[self.experts] if self.blocks == 1 else shared_d)
+        if self.clamp is not None:
+            limit, slope = self.clamp
+            self.limits = ops.Clamp(rt.upload(torch.tensor([limit] * self.experts + [self.shared_limit] * self.blocks, dtype=torch.float32)), slope)
+            if S:
+                self.shared_clamp = ops.Clamp(rt.upload(torch.tensor([self.shared_limit], dtype=torch.float32)), slope)
 
     def forward(self, ctx, h):
         rt, T, E, top = ctx.rt, ctx.n_tokens, self.experts, self.top
@@ -131,7 +151,10 @@ class RoutedExperts(base.FeedForward):
                 ops.scatter_scaled_rows(h, row_of_pair, wt, xs)
             else:
                 ops.gather_rows(h, token_of_row, xs)
-            (G.gemm_grouped_swiglu if self.gated else G.gemm_grouped_relu2)(xs, w_gu, act, bn, offsets, tile_start, rt.status)
+            if self.gated:
+                G.gemm_grouped_swiglu(xs, w_gu, act, bn, offsets, tile_start, rt.status, clamp=self.limits)
+            else:
+                G.gemm_grouped_relu2(xs, w_gu, act, bn, offsets, tile_start, rt.status)
             G.gemm_grouped(act, w_d, y, bn, offsets, tile_start, rt.status)
         else:
             tc = how != "simt"
@@ -140,11 +163,11 @@ class RoutedExperts(base.FeedForward):
                 src, rows = rt.empty((R, self.hidden)), None
                 ops.scatter_scaled_rows(h, row_of_pair, wt, src)
             ops.gemm_grouped(src, rows, w_gu, act, offsets, tile_start, gated=self.gated, tensor_cores=tc and ops.rows_mma_fits(src, w_gu),
-                             act="none" if self.gated else "relu2")
+                             act="none" if self.gated else "relu2", clamp=self.limits)
             ops.gemm_grouped(act, None, w_d, y, offsets, tile_start, gated=False, tensor_cores=tc and ops.rows_mma_fits(act, w_d))
         shared = None
         if self.shared_ff and not always:
-            shared = rt.linear(rt.gate_up_act(h, self.shared_gu) if self.gated else rt.up_act(h, self.shared_gu, "relu2"), self.shared_d)
+            shared = rt.linear(rt.gate_up_act(h, self.shared_gu, self.shared_clamp) if self.gated else rt.up_act(h, self.shared_gu, "relu2"), self.shared_d)
         out = rt.empty((1, T, self.hidden), torch.float32)
         ops.moe_combine(y, row_of_pair, wt, shared, out[0], weighted=not on_input, gate=(logits, E) if self.shared_gate and shared is not None else None)
         return out

@@ -16,7 +16,8 @@ Variants, each a constructor parameter. `q_rank` n: the queries go through a lat
 q = Wuq c_q; the layer's first product is then [Wdq | Wdkv] h and a second one makes the heads' queries. `window` W: a position sees
 itself and the W - 1 positions before it (the cache then keeps only those pages). `gate`: head a's output is multiplied by
 sigmoid(Wg h)_a, one number a head from the layer's input (its rows ride in the first product; the sigmoid sits in the epilogue of the
-per-head product with Wuv). rot_dim 0: no rotated part at all (the position encoding is then "none").
+per-head product with Wuv). `sink`: a learned number per head whose exponential the softmax's denominator holds as well (no key, no value, not
+scaled). rot_dim 0: no rotated part at all (the position encoding is then "none").
 """
 from __future__ import annotations
 
@@ -34,7 +35,8 @@ from .base import PagedRows, WeightSpec
 class LatentAttention(base.Mixer):
     def __init__(self, prefix: str, hidden: int, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, scale: float, norm_eps: float,
                  position: base.PositionEncoding, own_kv: bool = True, window: Optional[int] = None,
-                 names: tuple = ("q", "dkv", "dkv.norm", "uk", "uv", "o", "dq", "dq.norm", "uq", "g"), q_rank: Optional[int] = None, gate: bool = False):
+                 names: tuple = ("q", "dkv", "dkv.norm", "uk", "uv", "o", "dq", "dq.norm", "uq", "g", "sink"), q_rank: Optional[int] = None, gate: bool = False,
+                 sink: bool = False):
         if getattr(position, "pairing", "interleaved") != "interleaved":
             raise ValueError("latent attention turns entry 2i with 2i + 1: it needs a position encoding with pairing=\"interleaved\" (or none)")
         if window is not None and (window <= 0 or not own_kv):
@@ -43,6 +45,7 @@ class LatentAttention(base.Mixer):
             raise ValueError("a query latent must have a positive size, and is built for layers that keep their own latent")
         self.window, self.q_rank, self.gate = window, q_rank, bool(gate)
         self.w_uq = self.q_norm = None
+        self.sink, self.sink_dev = bool(sink), None
         self.prefix, self.hidden, self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank = prefix, hidden, heads, dim, rot_dim, vdim, kv_rank
         self.scale, self.norm_eps, self.position, self.own_kv, self.names = scale, norm_eps, position, own_kv, tuple(names)
         self.w_in = self.wuk_t = self.wuv = self.wo = self.c_norm = None
@@ -63,6 +66,8 @@ class LatentAttention(base.Mixer):
                       WeightSpec(self._name(8), (H * (self.dim + self.rot_dim), self.q_rank))]
         if self.gate:
             specs.append(WeightSpec(self._name(9), (H, self.hidden)))
+        if self.sink:
+            specs.append(WeightSpec(self._name(10), (H,), std=1.0))
         if self.own_kv:
             specs += [WeightSpec(self._name(1), (r + self.rot_dim, self.hidden)), WeightSpec(self._name(2), (r,), role="norm")]
         return specs
@@ -81,6 +86,8 @@ class LatentAttention(base.Mixer):
         self.wuk_t = rt.upload(weights[self._name(3)].view(H, self.dim, r).transpose(1, 2), rt.act_dtype)   # [H, rank, dim]: q_n -> rank values
         self.wuv = rt.upload(weights[self._name(4)].view(H, self.vdim, r), rt.act_dtype)                    # [H, vdim, rank]
         self.wo = rt.matrix(weights[self._name(5)])
+        if self.sink:
+            self.sink_dev = rt.vector(weights[self._name(10)])
         self.position.bind(weights, rt)
 
     def _slices(self, ctx, view) -> tuple[int, int]:
@@ -131,7 +138,9 @@ class LatentAttention(base.Mixer):
             raise ValueError(f"latent_attention = \"mma\" needs a latent and a rotated part that are multiples of 16 (up to 512 and 576 together), got {self.kv_rank} and {self.rot_dim}")
         return fits
 
-    def forward(self, ctx, h, cache):
+    adds_to_residual = True   # the output projection may add to the residual stream in its epilogue
+
+    def forward(self, ctx, h, cache, residual=None):
         rt, T, H, r, rot = ctx.rt, ctx.n_tokens, self.heads, self.kv_rank, self.rot_dim
         cos, sin = self.position.tables(ctx)
         qd = rt.linear(h, self.w_in)
@@ -162,9 +171,9 @@ class LatentAttention(base.Mixer):
         u = rt.empty((T, H, r))
         if self._tensor_cores(rt):
             rows, units = self._rows_and_units(ctx)
-            ops.latent_attention_mma(q_full, cache, ctx.positions, ctx.seg_of_token, units, self.scale, u, r, n_slices, slice_keys, scratch, rt.status, rows, window=self.window)
+            ops.latent_attention_mma(q_full, cache, ctx.positions, ctx.seg_of_token, units, self.scale, u, r, n_slices, slice_keys, scratch, rt.status, rows, window=self.window, sink=self.sink_dev)
         else:
-            ops.latent_attention(q_full, cache, ctx.positions, ctx.seg_of_token, self.scale, u, r, n_slices, slice_keys, scratch, rt.status, window=self.window)
+            ops.latent_attention(q_full, cache, ctx.positions, ctx.seg_of_token, self.scale, u, r, n_slices, slice_keys, scratch, rt.status, window=self.window, sink=self.sink_dev)
         v = rt.empty((T, H, self.vdim))
         ops.gemm_heads(u, self.wuv, v, self.vdim, tensor_cores=tc and ops.rows_mma_fits(u, self.wuv), gate=gate)
-        return rt.linear(v.view(T, H * self.vdim), self.wo)
+        return rt.linear(v.view(T, H * self.vdim), self.wo, add_to=residual)

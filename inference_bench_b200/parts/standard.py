@@ -74,7 +74,7 @@ class LayerNorm(base.Norm):
 
     takes_layout = True   # `forward` takes the extras named above (what a block with input convolutions asks of its norms)
 
-    takes_scaled_delta = True
+    takes_scaled_delta = takes_summed_delta = True
 
     def __init__(self, name: str, size: int, eps: float, bias: Optional[str] = None):
         """bias: None, or the bias tensor's name as a pattern of the weight's ("{}.b")."""
@@ -114,6 +114,10 @@ class LayerNorm(base.Norm):
         ops.shift_mixes(h, mu, state, ctx.seg_of_token, ctx.seg_start, ctx.seg_slot, out)
 
     def forward(self, ctx, x, delta, rows=None, delta_scale=None, delta_bias=None, x_copy=None, layout=None):
+        if isinstance(delta, base.SummedDelta):
+            out = ctx.rt.empty((x.shape[0] if rows is None else rows.shape[0], self.size))
+            ops.add_layernorm(x, delta.first, self.w, out, self.eps, rows, b=self.b, early=self._early(ctx), delta2=delta.second)
+            return out
         if isinstance(delta, base.ScaledDelta):
             out = ctx.rt.empty((x.shape[0] if rows is None else rows.shape[0], self.size))
             ops.add_layernorm(x, delta.delta, self.w, out, self.eps, rows, b=self.b, delta_mult=delta.scale, early=self._early(ctx))
@@ -133,12 +137,21 @@ class RotaryEmbedding(base.PositionEncoding):
     inv_freq_i = theta^(-2i/rotary_dim), angle = float(pos) * inv_freq_i in float32
     (crates/kir/tests/golden/attention/RopeKvWrite_bf16x2_sm120.cu:32-35, 200-206)."""
 
-    def __init__(self, rotary_dim: int, theta: float, pairing: str = "half", scaling: Optional[tuple] = None):
+    def __init__(self, rotary_dim: int, theta: float, pairing: str = "half", scaling: Optional[tuple] = None, yarn: Optional[tuple] = None):
         """pairing: which entries a mixer turns together with these angles: "half" pairs entry i with i + rotary_dim/2,
         "interleaved" pairs entry 2i with 2i + 1. The tables are the same; the mixer's kernel does the pairing.
         scaling: None or (factor, low, high, original): frequencies are rescaled by wavelength l = 2 pi / f in three bands. Where
         l < original / high the frequency stays; where l > original / low it becomes f / factor; between the two it is
-        (1 - s) f / factor + s f with s = (original / l - low) / (high - low)."""
+        (1 - s) f / factor + s f with s = (original / l - low) / (high - low).
+        yarn: None or (factor, original, fast, slow): pair i keeps its frequency f below a ramp of pairs, has f / factor above it and a blend
+        between; the ramp runs from the pair that turns `fast` times over `original` positions (rounded down, at least 0) to the one that
+        turns `slow` times (rounded up, at most rotary_dim - 1). Cosines and sines are then multiplied by 0.1 ln(factor) + 1."""
+        if yarn is not None:
+            yarn = tuple(float(v) for v in yarn)
+            if len(yarn) != 4 or min(yarn) <= 0 or theta <= 0 or theta == 1.0 or scaling is not None:
+                raise ValueError(f"yarn must be four positive numbers (factor, original, fast, slow), alone and with a base other than 1, got {yarn}")
+        self.yarn = yarn
+        self.amplitude = 1.0 if yarn is None else 0.1 * math.log(yarn[0]) + 1.0
         if scaling is not None:
             scaling = tuple(float(v) for v in scaling)
             if len(scaling) != 4 or scaling[0] <= 0 or scaling[2] == scaling[1] or scaling[3] <= 0:
@@ -160,15 +173,21 @@ class RotaryEmbedding(base.PositionEncoding):
             blend = (original / wavelength - low) / (high - low)
             mid = (1.0 - blend) * f / factor + blend * f
             f = torch.where(wavelength < original / high, f, torch.where(wavelength > original / low, f / factor, mid))
+        if self.yarn is not None:
+            factor, original, fast, slow = self.yarn
+            pair_of = lambda turns: self.rotary_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.theta))
+            lo, hi = max(math.floor(pair_of(fast)), 0), min(math.ceil(pair_of(slow)), self.rotary_dim - 1)
+            ramp = ((torch.arange(f.shape[0], dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+            f = f / factor * ramp + f * (1.0 - ramp)
         self.inv_freq = rt.upload(f.to(torch.float32))
 
     def tables(self, ctx):
-        key = ("rope", self.rotary_dim, self.theta, self.scaling)
+        key = ("rope", self.rotary_dim, self.theta, self.scaling, self.yarn)
         if key not in ctx.memo:
             half = self.rotary_dim // 2
             cos = ctx.rt.empty((ctx.n_tokens, half), torch.float32)
             sin = ctx.rt.empty((ctx.n_tokens, half), torch.float32)
-            ops.rope_table(ctx.positions, self.inv_freq, cos, sin)
+            ops.rope_table(ctx.positions, self.inv_freq, cos, sin, self.amplitude)
             ctx.memo[key] = (cos, sin)
         return ctx.memo[key]
 
@@ -311,8 +330,12 @@ class SwiGLU(base.FeedForward):
     (crates/kir/src/cuda/prelude.cu:125-133; gate and up fused into one product at load,
     crates/specrt/src/weights.rs:1049-1062)."""
 
-    def __init__(self, prefix: str, hidden: int, intermediate: int, names: tuple = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")):
-        """names: what the gate, up and down matrices are called under `prefix`."""
+    def __init__(self, prefix: str, hidden: int, intermediate: int, names: tuple = ("gate_proj.weight", "up_proj.weight", "down_proj.weight"), clamp: Optional[tuple] = None):
+        """names: what the gate, up and down matrices are called under `prefix`. clamp: None, or (limit, slope): the halves are clamped and the
+        activation is g sigmoid(slope g) (u + 1) with g = min(gate, limit), u = up cut to [-limit, limit]."""
+        if clamp is not None and not clamp[0] > 0:
+            raise ValueError(f"a limit must be positive, got {clamp[0]}")
+        self.clamp, self.clamp_dev = clamp, None
         self.prefix, self.hidden, self.intermediate, self.names = prefix, hidden, intermediate, tuple(names)
         self.wgu = self.wd = None
 
@@ -325,12 +348,14 @@ class SwiGLU(base.FeedForward):
         p, (g, u, d) = self.prefix, self.names
         self.wgu = rt.matrix(torch.cat([weights[f"{p}.{g}"], weights[f"{p}.{u}"]], dim=0))
         self.wd = rt.matrix(weights[f"{p}.{d}"])
+        if self.clamp is not None:
+            self.clamp_dev = ops.Clamp(rt.upload(torch.tensor([self.clamp[0]], dtype=torch.float32)), self.clamp[1])
 
     adds_to_residual = True   # the down projection may add to the residual stream in its epilogue
 
     def forward(self, ctx, h, residual=None):
         rt = ctx.rt
-        return rt.linear(rt.gate_up_act(h, self.wgu), self.wd, add_to=residual)
+        return rt.linear(rt.gate_up_act(h, self.wgu, self.clamp_dev), self.wd, add_to=residual)
 
 
 @base.register_feed_forward("dense_xielu")
@@ -468,6 +493,36 @@ class PreNormBlock(base.Block):
         h = self.feed_forward_norm.forward(ctx, x, a)
         f = self.feed_forward.forward(ctx, h, residual=x) if self.feed_forward.adds_to_residual and plain else self.feed_forward.forward(ctx, h)
         return f if plain else base.ScaledDelta(f, self.residual_mult)
+
+
+@base.register_block("parallel_sublayers")
+class ParallelBlock(base.Block):
+    """x += mixer(h) + feed_forward(h) with h = norm(x): one norm in front of both sublayers, which read the same rows. Both contributions are
+    left to the next norm, which adds them in one kernel (a `SummedDelta`); a product that can add to the stream in its epilogue may do so at
+    any time, since neither sublayer reads the stream. A layer without a feed-forward has the mixer alone."""
+
+    def __init__(self, mixer_norm, mixer, feed_forward_norm, feed_forward):
+        super().__init__(mixer_norm, mixer, feed_forward_norm, feed_forward)
+        self.has_ff = not isinstance(feed_forward, NoFeedForward)
+        if not mixer_norm.takes_summed_delta or not mixer_norm.takes_scaled_delta:
+            raise ValueError(f"this arrangement needs a norm that adds two contributions, which {type(mixer_norm).__name__} does not")
+        if getattr(mixer, "bias", False) or mixer.runs_norm:
+            raise ValueError("this arrangement takes neither a mixer's output bias nor a mixer that runs its own norm")
+
+    def forward(self, ctx, x, pending, cache):
+        if pending is None:
+            ctx.rt.next_in_order(ctx)
+        h = self.mixer_norm.forward(ctx, x, pending)
+        run = lambda part, *args: part.forward(ctx, h, *args, residual=x) if part.adds_to_residual else part.forward(ctx, h, *args)
+        f = None
+        if self.has_ff:
+            f = run(self.feed_forward)
+            ctx.rt.next_in_order(ctx)
+        a = run(self.mixer, cache)
+        left = [d for d in (a, f) if d is not None]
+        if len(left) == 2:
+            return base.SummedDelta(*left)
+        return base.ScaledDelta(left[0], 1.0) if left else None
 
 
 @base.register_block("outnorm")

@@ -41,6 +41,8 @@ def random_tensor(spec: WeightSpec, seed: int, device="cpu", dtype=torch.bfloat1
         t = torch.log(0.5 + 7.5 * torch.rand(spec.shape, generator=g, device=device, dtype=torch.float32))
     elif spec.role == "decay_bias":    # z of a decay exp(-exp(z)): decays between 0.37 and 0.998
         t = torch.rand(spec.shape, generator=g, device=device, dtype=torch.float32) * 6.0 - 6.0
+    elif spec.role == "keep_bias":     # forget gates sigmoid(z) between 0.88 and 0.998
+        t = torch.rand(spec.shape, generator=g, device=device, dtype=torch.float32) * 4.0 + 2.0
     elif spec.role == "matrix":
         t = torch.randn(spec.shape, generator=g, device=device, dtype=torch.float32) * (spec.std if std is None else std)
     else:
