@@ -662,6 +662,65 @@ def fedipel_work(z: dict, layers: int, T: int, ctx: int, batch: int) -> tuple:
     return work, lin
 
 
+# Gokosun at layer sizes that resemble small hybrid models: a matrix memory with heads of 128 x 128, grouped attention with heads of 128, latent attention
+# with a query latent and a rotated part; routed feed-forwards beside a shared expert, a dense one of the same active size every fourth layer. Beside
+# it Fedipel (recurrence, grouped attention, layer norms, experts with a shared one) and, for the latent attention and gated experts, Ditalorn, at
+# equal width, heads, cache rows, experts and choices.
+GOKOSUN_SIZES = {name: dict(FEDIPEL_SIZES[name], att_dim=128, lat_heads=d["heads"], lat_dim=d["dim"], lat_rot=d["rot"], lat_vdim=d["vdim"], rank=d["rank"], q_rank=d["q_rank"],
+                            dense_ff=FEDIPEL_SIZES[name]["top"] * FEDIPEL_SIZES[name]["expert_ff"] + FEDIPEL_SIZES[name]["shared_ff"], ditalorn=d)
+                 for name, d in (("small", DITALORN_SIZES["small"]), ("mid", DITALORN_SIZES["lite"]))}
+DESIGN_KINDS["gokosun"] = {
+    "attention": ["ib_attention_generic", "ib_attention_decode", "ib_attention_decode_stream", "ib_attention_prefill_ws", "ib_attention_prefill_tc"],
+    "latent": ["ib_latent_attention", "ib_latent_attention_mma"], "heads": ["ib_gemm_heads", "ib_gemm_heads_mma"],
+    "recurrence": ["ib_memory_gates", "ib_memory_walk", "ib_recurrence_chunks_finish", "ib_memory_out"],
+    "experts": ["ib_gemm_grouped", "ib_gemm_grouped_mma", "ib_gemm_grouped_tcgen05", "ib_gemm_grouped_swiglu_tcgen05", "ib_gather_rows"],
+    "route": ["ib_moe_route", "ib_moe_sort", "ib_moe_route_sort", "ib_moe_combine"],
+    "norm": ["ib_add_layernorm", "ib_row_norm_qkv", "ib_latent_down", "ib_latent_prepare"], "gemm": LEAVE_OUT["gemm"]}
+
+
+def gokosun_config(z: dict, layers: int) -> dict:
+    att = {"heads": z["att_heads"], "kv_heads": z["att_kv_heads"], "dim": z["att_dim"], "vdim": z["att_vdim"], "scale": z["att_dim"] ** -0.5, "v_mix": True,
+           "rot": {"base": 500000.0, "dims": z["att_dim"]}}
+    mem = {"heads": z["rec_heads"], "dim": z["rec_dim"], "vdim": z["rec_vdim"], "gate_cap": 15.0}
+    lat = {"heads": z["lat_heads"], "dim": z["lat_dim"], "rot_dim": z["lat_rot"], "vdim": z["lat_vdim"], "kv_rank": z["rank"], "q_rank": z["q_rank"],
+           "scale": (z["lat_dim"] + z["lat_rot"]) ** -0.5,
+           "rot": {"base": 10000.0, "dims": z["lat_rot"], "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"], "limit": 7.0}, "router": {"experts": z["experts"], "top": z["top"], "scale": 2.0},
+           "shared": {"ff": z["shared_ff"], "limit": 7.0}}
+    four = [("mlstm", mem, moe), ("attention", att, moe), ("latent_attention", lat, moe), ("attention", att, {"kind": "dense", "ff": z["dense_ff"], "limit": 7.0})]
+    ls = [dict(zip(("type", "mixer", "mlp"), four[i % 4])) for i in range(layers)]
+    return {"architecture": "Gokosun", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "layers": ls}
+
+
+def gokosun_work(z: dict, layers: int, T: int, ctx: int, batch: int) -> tuple:
+    """As `lulenex_work`: the memory's walk is float32 FMAs, its floor the bytes it must move."""
+    n_mem, n_lat = (sum(1 for i in range(layers) if i % 4 == k) for k in (0, 2))
+    n_att, n_dense = layers - n_mem - n_lat, sum(1 for i in range(layers) if i % 4 == 3)
+    n_moe = layers - n_dense
+    W, H, G, D, V = z["width"], z["att_heads"], z["att_kv_heads"], z["att_dim"], z["att_vdim"]
+    LH, LD, LR, LV, K, Q = z["lat_heads"], z["lat_dim"], z["lat_rot"], z["lat_vdim"], z["rank"], z["q_rank"]
+    rh, rd, rv, F, S, E, top = z["rec_heads"], z["rec_dim"], z["rec_vdim"], z["expert_ff"], z["shared_ff"], z["experts"], z["top"]
+    pairs = T * (T + 1) / 2
+    mem_row = rh * (4.0 * (2 * rd + rv) + 4.0 * rv + 10.0 * rv)          # q, k, v in; o out; o and the gate in, the gated norm out
+    norm_row = layers * W * (4.0 * 4 + 2) + n_att * (6.0 * (H * D + G * (D + V)) + 4.0 * G * V) + n_lat * (6.0 * (Q + K + LR) + 6.0 * LH * (LD + LR))
+    lin = n_mem * (2 * rh * rd + 3 * rh * rv + 2 * rh) * W + n_att * (H * D + G * (D + V) + H * V) * W + \
+        n_lat * ((Q + K + LR) * W + LH * (LD + LR) * Q + LH * LV * W) + n_moe * (E + 3 * S) * W + n_dense * 3 * z["dense_ff"] * W + z["vocab"] * W
+    used = min(batch * top, E)
+    work = {
+        "prefill": {"attention": {"flops": n_att * 2.0 * H * (D + V) * pairs}, "latent": {"flops": n_lat * 2.0 * LH * pairs * (2 * K + LR)},
+                    "heads": {"flops": n_lat * 2.0 * T * LH * K * (LD + LV)}, "recurrence": {"flops": 0.0, "bytes": n_mem * T * mem_row},
+                    "experts": {"flops": n_moe * 2.0 * T * top * 3 * F * W}, "norm": {"flops": 0.0, "bytes": T * norm_row}},
+        # (up to 64 tokens the shared expert's products run among the experts')
+        "decode": {"attention": {"flops": n_att * 2.0 * H * (D + V) * batch * ctx, "bytes": n_att * 2.0 * batch * ctx * G * (D + V)},
+                   "latent": {"flops": n_lat * 2.0 * LH * batch * ctx * (2 * K + LR), "bytes": n_lat * 2.0 * batch * ctx * (K + LR)},
+                   "heads": {"flops": n_lat * 2.0 * batch * LH * K * (LD + LV), "bytes": n_lat * 2.0 * LH * K * (LD + LV)},
+                   "recurrence": {"flops": 0.0, "bytes": n_mem * batch * (mem_row + rh * 8.0 * rd * (rv + 1))},
+                   "experts": {"flops": n_moe * 2.0 * batch * 3 * (top * F + S) * W, "bytes": n_moe * 2.0 * 3 * (used * F + S) * W},
+                   "norm": {"flops": 0.0, "bytes": batch * norm_row}},
+    }
+    return work, lin
+
+
 def kernel_times(engine, entries) -> dict:
     """Milliseconds per library entry point in one step run outside a graph: every call stands between two CUDA events, and a
     long idle kernel goes first so that the whole step is queued before its first kernel starts (the events then measure the
@@ -753,7 +812,7 @@ def run_design(args) -> dict:
     layers = args.layers or 4
     steps, warmup = min(args.steps, 32), max(args.warmup, 3)
     out = {"design": args.design, "layers": layers, "peaks": pk_src, "sizes": {}}
-    sizes = {"busadra": BUSADRA_SIZES, "lulenex": LULENEX_SIZES, "ditalorn": DITALORN_SIZES, "fedipel": FEDIPEL_SIZES}.get(args.design, DESIGN_SIZES)
+    sizes = {"busadra": BUSADRA_SIZES, "lulenex": LULENEX_SIZES, "ditalorn": DITALORN_SIZES, "fedipel": FEDIPEL_SIZES, "gokosun": GOKOSUN_SIZES}.get(args.design, DESIGN_SIZES)
     for name in (args.size.split(",") if args.size else list(sizes)):
         z = sizes[name] if name in sizes or args.design != "lulenex" else LULENEX_EXTRA_SIZES[name]
         report = {}
@@ -766,6 +825,9 @@ def run_design(args) -> dict:
         elif args.design == "fedipel":
             zb = z
             pair = (("fedipel", fedipel_config(z, layers)), ("busadra", busadra_config(z, layers)))
+        elif args.design == "gokosun":
+            zb = z
+            pair = (("gokosun", gokosun_config(z, layers)), ("fedipel", fedipel_config(z, layers)), ("ditalorn", ditalorn_config(z["ditalorn"], layers)))
         elif args.design == "ditalorn":
             pair = (("ditalorn", ditalorn_config(z, layers)), ("zabonex", zabonex_config(z, layers)))
         else:
@@ -780,10 +842,12 @@ def run_design(args) -> dict:
                     3 * z["dense_ff"] * z["width"] + (layers - 1) * (3 * z["shared_ff"] + z["experts"]) * z["width"] + vocab * z["width"]
             elif arch == "lulenex":
                 work, lin = lulenex_work(z, layers, PROMPT, PROMPT, 8)
+            elif arch == "gokosun":
+                work, lin = gokosun_work(z, layers, PROMPT, PROMPT, 8)
             elif arch == "fedipel":
                 work, lin = fedipel_work(z, layers, PROMPT, PROMPT, 8)
             elif arch == "ditalorn":
-                work, lin = ditalorn_work(z, layers, PROMPT, PROMPT, 8)
+                work, lin = ditalorn_work(z.get("ditalorn", z), layers, PROMPT, PROMPT, 8)
             elif arch == "busadra":
                 work = busadra_work(zb, layers, PROMPT, PROMPT, 8)
                 n_att = sum(1 for i in range(layers) if i % 4 in (0, 3))
@@ -856,9 +920,9 @@ def main() -> int:
     ap.add_argument("--leave-out", default="", help="with --only decode or prefill: also time the step without each of these kinds of kernel (comma separated; "
                     "a+b leaves both out): " + ", ".join(sorted(LEAVE_OUT)))
     ap.add_argument("--only", default="", choices=["", "prefill", "decode", "mixed"], help="run one part alone (for profiling); prints a short report")
-    ap.add_argument("--design", default="", choices=["", "zabonex", "busadra", "lulenex", "ditalorn", "fedipel"],
-                    help="measure another design beside the closest existing one at equal size (Qwen3; for lulenex and fedipel, Busadra; for ditalorn, Zabonex) instead of the benchmark (prints its own report)")
-    ap.add_argument("--size", default="", help="with --design: which of its sizes (comma separated; default all): " + ", ".join(DESIGN_SIZES) + " (zabonex); " + ", ".join(BUSADRA_SIZES) + " (busadra); " + ", ".join(LULENEX_SIZES) + " (lulenex); " + ", ".join(DITALORN_SIZES) + " (ditalorn); " + ", ".join(FEDIPEL_SIZES) + " (fedipel)")
+    ap.add_argument("--design", default="", choices=["", "zabonex", "busadra", "lulenex", "ditalorn", "fedipel", "gokosun"],
+                    help="measure another design beside the closest existing one at equal size (Qwen3; for lulenex and fedipel, Busadra; for ditalorn, Zabonex; for gokosun, Fedipel and Ditalorn) instead of the benchmark (prints its own report)")
+    ap.add_argument("--size", default="", help="with --design: which of its sizes (comma separated; default all): " + ", ".join(DESIGN_SIZES) + " (zabonex); " + ", ".join(BUSADRA_SIZES) + " (busadra); " + ", ".join(LULENEX_SIZES) + " (lulenex); " + ", ".join(DITALORN_SIZES) + " (ditalorn); " + ", ".join(FEDIPEL_SIZES) + " (fedipel); " + ", ".join(GOKOSUN_SIZES) + " (gokosun)")
     ap.add_argument("--kernels", action="store_true", help="with --design: also list every library entry point's time in one prefill and one decode step")
     args = ap.parse_args()
     if args.design:

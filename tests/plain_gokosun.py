@@ -217,8 +217,12 @@ def experts_ff(h, w, p, f):
 # ------------------------------------------------------------------------------------------ the model
 def hidden_states(cfg, w, tokens):
     """The residual stream after every layer, [layers, T, W]."""
+    return hidden_from(cfg, w, d(w["embed"])[torch.as_tensor(tokens, dtype=torch.long)])
+
+
+def hidden_from(cfg, w, x):
+    """The same from the stream in front of the first layer."""
     eps = float(cfg["norm"]["eps"])
-    x = d(w["embed"])[torch.as_tensor(tokens, dtype=torch.long)]
     out, first = [], None
     for i, l in enumerate(cfg["layers"]):
         p, m, f = f"l{i}.mix", l["mixer"], l.get("mlp")
