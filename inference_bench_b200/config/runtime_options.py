@@ -36,6 +36,7 @@ class RuntimeOptions:
     # ---- launches
     graphs: bool = True                # replay steps of decoded tokens as CUDA graphs
     pdl: bool = True                   # programmatic dependent launch: a kernel's set-up overlaps the tail of the one before
+    side_stream: bool = True           # sublayers that read the same rows run side by side in captured steps of decoded tokens (the feed-forward on a stream of its own)
     pipeline: bool = True              # keep decode steps one ahead of the host
     # ---- fusion
     fuse: bool = True                  # master switch: False turns every fused form below off

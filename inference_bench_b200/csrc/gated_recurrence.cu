@@ -100,6 +100,7 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && RPT == 8 ? 3 : 1) gated_r
   const int a = blockIdx.y, j0 = blockIdx.z * kCols;
   const int tid = threadIdx.x, ds = tid % DS, col = 2 * (tid / DS), j = j0 + col;   // columns j and j + 1, rows ds * RPT .. ds * RPT + RPT - 1
   const int d0 = ds * RPT;
+  const bool live = j0 + 2 * ((tid & ~31) / DS) < V;   // (a warp whose columns all lie beyond V only helps to prepare the tokens)
   const bool d4 = D % 4 == 0;
   int t0, t1;
   float* S;
@@ -321,7 +322,7 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && RPT == 8 ? 3 : 1) gated_r
     // Eight tokens at a time: their sixteen sums per thread are reduced over the DS threads of the column pair together, each exchange halving
     // what a lane still holds (15 shuffles for eight tokens and DS = 16 instead of 64; the pairs that are added, and so the bits, are those of
     // the token-by-token reduction).
-    for (; tt + kGroup <= n; tt += kGroup) {
+    for (; live && tt + kGroup <= n; tt += kGroup) {
       float acc[2 * kGroup];
 #pragma unroll
       for (int k = 0; k < kGroup; k++) advance(tt + k, acc[2 * k], acc[2 * k + 1]);
@@ -349,7 +350,7 @@ __global__ void __launch_bounds__(MAXT, MAXT == 256 && RPT == 8 ? 3 : 1) gated_r
         }
       }
     }
-    for (; tt < n; tt++) {
+    for (; live && tt < n; tt++) {
       float acc0, acc1;
       advance(tt, acc0, acc1);
       for (int o = DS >> 1; o > 0; o >>= 1) {

@@ -50,6 +50,7 @@ class Runtime:
         self.mode = self.options.dtype
         self.act_dtype = MODES[self.mode]
         self.gemm = self.options.gemm  # "auto" | "simt" | "tcgen05"
+        self._side: Optional[torch.cuda.Stream] = None
         self.status = torch.zeros(1, dtype=torch.int32, device=self.device)
         self.activate()
 
@@ -60,6 +61,17 @@ class Runtime:
         ops._device_index = self.device_index
         self.lib.ib_set_pdl(1 if self.options.pdl else 0)
         self.lib.ib_set_wait_limit_ms(int(self.options.wait_limit_ms))
+
+    def side_stream(self, ctx) -> Optional[torch.cuda.Stream]:
+        """A second stream for work of a captured step that does not depend on what the current stream does meanwhile, or None where the step
+        runs on one stream (a step with prompt portions fills the GPU by itself, and its order is kept). Whoever uses it makes it wait for the
+        current stream first and the current stream for it before anything reads the results, and holds every tensor both streams touch
+        until then."""
+        if not ctx.fixed_shape or not self.options.side_stream:
+            return None
+        if self._side is None:
+            self._side = torch.cuda.Stream(device=self.device)
+        return self._side
 
     def next_in_order(self, ctx) -> None:
         """In a step with prompt portions: the next kernel starts only when everything before it is done. For a place where a third kernel in a

@@ -499,7 +499,7 @@ class PreNormBlock(base.Block):
 class ParallelBlock(base.Block):
     """x += mixer(h) + feed_forward(h) with h = norm(x): one norm in front of both sublayers, which read the same rows. Both contributions are
     left to the next norm, which adds them in one kernel (a `SummedDelta`); a product that can add to the stream in its epilogue may do so at
-    any time, since neither sublayer reads the stream. A layer without a feed-forward has the mixer alone."""
+    any time, since neither sublayer reads the stream. In captured steps of decoded tokens the two run on streams of their own. A layer without a feed-forward has the mixer alone."""
 
     def __init__(self, mixer_norm, mixer, feed_forward_norm, feed_forward):
         super().__init__(mixer_norm, mixer, feed_forward_norm, feed_forward)
@@ -513,12 +513,20 @@ class ParallelBlock(base.Block):
         if pending is None:
             ctx.rt.next_in_order(ctx)
         h = self.mixer_norm.forward(ctx, x, pending)
-        run = lambda part, *args: part.forward(ctx, h, *args, residual=x) if part.adds_to_residual else part.forward(ctx, h, *args)
-        f = None
-        if self.has_ff:
-            f = run(self.feed_forward)
-            ctx.rt.next_in_order(ctx)
-        a = run(self.mixer, cache)
+        run = lambda part, *args, **kw: part.forward(ctx, h, *args, **(kw if part.adds_to_residual else {}))
+        f, side = None, ctx.rt.side_stream(ctx) if self.has_ff else None
+        if side is not None:
+            main = torch.cuda.current_stream(ctx.rt.device)
+            side.wait_stream(main)
+            with torch.cuda.stream(side):   # (neither adds to the stream itself here: they run at the same time)
+                f = run(self.feed_forward)
+            a = run(self.mixer, cache)
+            main.wait_stream(side)
+        else:
+            if self.has_ff:
+                f = run(self.feed_forward, residual=x)
+                ctx.rt.next_in_order(ctx)
+            a = run(self.mixer, cache, residual=x)
         left = [d for d in (a, f) if d is not None]
         if len(left) == 2:
             return base.SummedDelta(*left)

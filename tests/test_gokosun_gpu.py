@@ -582,6 +582,22 @@ def test_greedy_generation_through_the_engine(gdirs, name, graphs):
     assert one.tokens == want[1]
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_sublayers_on_two_streams_give_the_bits_of_one(gdirs, dtype):
+    """Captured decode steps with the feed-forward on a stream of its own: the logits of every step have the bits of the steps on one stream, for
+    one request and for five (padded rows beside them)."""
+    from inference_bench_b200 import Engine
+    vocab = tg.CONFIGS["C"]["config"]["vocab"]
+    prompts = [traces.prompt(30 + i, n, vocab) for i, n in enumerate((9, 40, 3, 70, 17))]
+    out = []
+    for side in (True, False):
+        eng = Engine(gdirs["C"], dtype=dtype, max_ctx=256, page_size=16, options={"side_stream": side})
+        tokens = [r.tokens for r in eng.generate(prompts, max_tokens=24)] + [eng.generate(prompts[1], max_tokens=24).tokens]
+        out.append((tokens, eng.executor.last_logits.clone() if eng.executor.last_logits is not None else None))
+    assert out[0][0] == out[1][0]
+    assert out[0][1] is None or torch.equal(out[0][1], out[1][1])
+
+
 def test_generation_in_bfloat16_runs_and_long_decoding_stays_close(gdirs):
     from inference_bench_b200 import Engine
     name = "C"
