@@ -1,5 +1,5 @@
-// Queries, keys and values of an attention whose norms run over a token's whole query and key rows (all heads at once, before they are split
-// into heads) and whose values may be mixed with another layer's.
+// Queries, keys and values of an attention whose norms run over a token's whole query and key rows (all heads at once, not head by
+// head) and whose values may be mixed with another layer's.
 //
 //  * row_norm_qkv: a CTA per token adds the partial sums of its projection row [heads x D | kv_heads x D | kv_heads x V] once (several loads in
 //    flight) into shared memory, takes the two sums of squares as block sums, and writes: q = w_q q / sqrt(mean(q^2) + eps) and k likewise, both

@@ -126,7 +126,8 @@ class LayerNorm(base.Norm):
             out = ctx.rt.empty((layout.rows(x.shape[0]), self.size), torch.float32)
         else:
             out = ctx.rt.empty((x.shape[0] if rows is None else rows.shape[0], self.size))
-        ops.add_layernorm(x, delta, self.w, out, self.eps, rows, delta_scale, delta_bias, x_copy, layout, b=self.b)
+        # (no contribution left to add: products added theirs to the stream themselves, right before this kernel)
+        ops.add_layernorm(x, delta, self.w, out, self.eps, rows, delta_scale, delta_bias, x_copy, layout, b=self.b, early=delta is not None or self._early(ctx))
         return out
 
 
@@ -499,7 +500,8 @@ class PreNormBlock(base.Block):
 class ParallelBlock(base.Block):
     """x += mixer(h) + feed_forward(h) with h = norm(x): one norm in front of both sublayers, which read the same rows. Both contributions are
     left to the next norm, which adds them in one kernel (a `SummedDelta`); a product that can add to the stream in its epilogue may do so at
-    any time, since neither sublayer reads the stream. In captured steps of decoded tokens the two run on streams of their own. A layer without a feed-forward has the mixer alone."""
+    any time, since neither sublayer reads the stream. In captured steps of decoded tokens the two run on streams of their own. A layer
+    without a feed-forward has the mixer alone."""
 
     def __init__(self, mixer_norm, mixer, feed_forward_norm, feed_forward):
         super().__init__(mixer_norm, mixer, feed_forward_norm, feed_forward)
@@ -510,8 +512,6 @@ class ParallelBlock(base.Block):
             raise ValueError("this arrangement takes neither a mixer's output bias nor a mixer that runs its own norm")
 
     def forward(self, ctx, x, pending, cache):
-        if pending is None:
-            ctx.rt.next_in_order(ctx)
         h = self.mixer_norm.forward(ctx, x, pending)
         run = lambda part, *args, **kw: part.forward(ctx, h, *args, **(kw if part.adds_to_residual else {}))
         f, side = None, ctx.rt.side_stream(ctx) if self.has_ff else None
